@@ -105,6 +105,8 @@ int md_set_gemm_mode(md_ctx* ctx, int mode);
  *   "pdl"           1 = launch the GEMV kernels with programmatic dependent launch: a kernel starts
  *                   streaming its weights while its predecessor on the stream drains.  Only for streams
  *                   on which no earlier kernel writes the weight matrices (registered weights).
+ *   "stack_trace"   1 = md_text_step of a layer-stack model keeps the residual stream after every layer for
+ *                   md_text_layer_stream (and is not recorded into a graph), 0 (default) = it does not
  *   "fused_decode"  1 (default) = a decode layer runs as three fused kernels, 0 = one kernel per reference op
  *   "dualk_variant" 0..4 = (warps, unroll) of the out-proj + fc2 kernel of the fused decode layer
  *   "decode_cluster" 1 = merge the key splits of the decode attention through the shared memory of a 16-CTA cluster;

@@ -72,7 +72,7 @@ int md_text_forward(md_text_model* model, md_text_request* req, const uint16_t* 
  *   tokens_out   host u32 [n_steps]: the token produced by each step
  *   forced       optional host u32 [n_steps]: teacher forcing — step i consumes forced[i-1] instead of
  *                its own previous output (step 0 consumes `first`)
- *   logits_out   optional host f16 [n_steps, vocab] */
+ *   logits_out   optional host f16 [n_steps, vocab] (layer-stack models: f32, passed through the same pointer) */
 int md_text_generate(md_text_model* model, md_text_request* req, uint32_t first, size_t n_steps,
                      uint32_t* tokens_out, const uint32_t* forced, uint16_t* logits_out);
 
@@ -88,6 +88,77 @@ int md_text_generate_batch(md_text_model* model, md_text_request* const* reqs, s
  * produced.  For parity checks of batched decoding against a reference that generated the forced tokens. */
 int md_text_generate_batch_forced(md_text_model* model, md_text_request* const* reqs, size_t batch, const uint32_t* first,
                                   size_t n_steps, uint32_t* tokens_out, const uint32_t* forced);
+
+/* ---- layer-stack text decoders --------------------------------------------------------------
+ *
+ * Decoder-only language models described layer by layer: every layer names its mixer (with the mixer's sizes), its
+ * feed-forward, and carries its own weights.  md_stack_model_create returns an ordinary md_text_model: requests, resets,
+ * md_text_step, md_text_generate and the batched forms work on it as on the Phi-style decoder above.
+ *
+ * One layer, x being the f32 residual stream and m = residual_mult:
+ *   u = rms(x; norm1);  u += causal_conv(u; conv1);  x += m * rms(mixer(u); norm1b)
+ *   u = rms(x; norm2);  u += causal_conv(u; conv2);  x += m * rms(ff(u);    norm2b)      (ff != MD_FF_NONE)
+ *
+ * Mixers
+ *   MD_MIXER_WINDOW_ATTENTION  grouped-query softmax attention whose values are its keys; score(i, j) =
+ *       scale * q.k - r1[h] * ln(1 + r2[h] * (i - j)); key j is visible to query i iff j <= i and (i - j < window or
+ *       j < keep_first); head h's output is multiplied by logistic(g_h).  w_in rows: q | k | g.
+ *   MD_MIXER_LIGHTNING         linear attention: S_t = decay[h] S_(t-1) + k_t v_t^T, o_t = S_t^T q_t with q, k, v = silu
+ *       of their projections; rms over all heads with mix_norm, times logistic(g).  w_in rows: q | k | v | g.
+ * Feed-forward
+ *   MD_FF_DENSE  w_down (act(w_gate u) * (w_up u));  MD_FF_MOE  `top` of `experts` such layers chosen by the largest
+ *       logistic(router u) and weighted with those scores.
+ *
+ * dtype MD_DTYPE_BF16: matrices and activations bfloat16, f32 accumulation.  MD_DTYPE_F32: everything f32, no
+ * reduced-precision product.  Matrices marked T below have that type; vectors are always f32.  All pointers are device
+ * pointers that stay valid as long as the model. */
+enum { MD_DTYPE_F16 = 0, MD_DTYPE_BF16 = 1, MD_DTYPE_F32 = 2 };
+enum { MD_MIXER_WINDOW_ATTENTION = 1, MD_MIXER_LIGHTNING = 2 };
+enum { MD_FF_NONE = 0, MD_FF_DENSE = 1, MD_FF_MOE = 2 };
+enum { MD_ACT_GELU_TANH = 1, MD_ACT_SILU = 2 };
+
+typedef struct md_stack_layer {
+    int mixer, ff;
+    size_t heads, kv_heads, dim, vdim;     /* kv_heads: attention only */
+    size_t window, keep_first;             /* attention; window 0 = unlimited */
+    float scale;                           /* attention */
+    const float* r1; const float* r2;      /* attention, [heads] */
+    const float* decay;                    /* lightning, [heads] */
+    const float* mix_norm;                 /* lightning, [heads * vdim] */
+    const void* w_in;                      /* T [in_rows, width]; in_rows: the rows named above, rounded up to 8 with zeros */
+    const float* b_in;                     /* [in_rows] or NULL */
+    size_t in_rows;
+    const void* w_out;                     /* T [width, heads * vdim] */
+    const float* norm1; const float* norm1b; const float* norm2; const float* norm2b;   /* [width] */
+    const float* conv1; const float* conv2;                                             /* [taps, width] */
+    int act;                               /* MD_ACT_* of the feed-forward */
+    size_t ff_dim, ff_pad;                 /* ff_pad: ff_dim rounded up to a multiple of 32 */
+    const void* w_gate_up;                 /* T [(experts,) 2 * ff_pad, width]: blocks of 32 gate rows and 32 up rows in turn */
+    const void* w_down;                    /* T [(experts,) width, ff_pad] */
+    const void* router;                    /* T [experts, width] */
+    size_t experts, top;
+} md_stack_layer;
+
+typedef struct md_stack_weights {
+    int dtype;
+    size_t n_layers, width, vocab, max_seq, taps;
+    float eps, residual_mult;
+    const md_stack_layer* layers;          /* host array, copied */
+    const void* embed;                     /* T [vocab, width] */
+    const void* head;                      /* T [vocab, width] */
+    const float* final_norm;               /* [width] */
+} md_stack_weights;
+
+int md_stack_model_create(md_ctx* ctx, const md_stack_weights* w, md_text_model** out);
+
+/* Run the next n >= 1 tokens of one request (any portion of a prompt, or one decoded token) from the state earlier calls
+ * left.  Optional outputs: the logits at the n_want places `want` (indices into tokens, ascending) as f32
+ * [n_want, vocab], host or device; token_out = argmax of the last row's logits.  Works for every md_text_model. */
+int md_text_step(md_text_model* model, md_text_request* req, const uint32_t* tokens, size_t n, const uint32_t* want,
+                 size_t n_want, float* logits_out, uint64_t* token_out);
+/* Copy the residual stream after layer `layer` of the last md_text_step (f32 [rows, width], layer-stack models with
+ * md_set_option("stack_trace", 1) at that step) to the host. */
+int md_text_layer_stream(md_text_request* req, size_t layer, float* out, size_t rows);
 
 /* ---- vision encoder (SigLIP-style ViT, vision_model.zig) --------------------------------- */
 

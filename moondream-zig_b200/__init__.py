@@ -44,15 +44,18 @@ class MdError(RuntimeError):
             self.zig_error = "error." + message.split(":", 1)[0]
 
 
-def build(force: bool = False) -> str:
-    """Compile the CUDA library in-tree (nvcc, sm_100a) if it is missing or stale."""
+def build(force: bool = False, static: bool = True) -> str:
+    """Compile the CUDA library in-tree (nvcc, sm_100a) if it is missing or stale.  static=False: only the shared library
+    this package loads, not the archive for native hosts."""
     csrc = os.path.join(_HERE, "csrc")
     srcs = [os.path.join(csrc, f) for f in os.listdir(csrc) if f.endswith((".cu", ".cuh"))] + [HEADER_PATH]
     inc = os.path.dirname(HEADER_PATH)
     srcs += [os.path.join(inc, f) for f in os.listdir(inc) if f.endswith(".h")]
     stale = (not os.path.exists(LIB_PATH)) or any(os.path.getmtime(s) > os.path.getmtime(LIB_PATH) for s in srcs)
     if force or stale:
-        subprocess.check_call(["make", "-C", csrc, "-j8"] + (["-B"] if force else []), stdout=subprocess.DEVNULL)
+        target = "all" if static else os.path.join("..", os.path.basename(LIB_PATH))
+        subprocess.check_call(["make", "-C", csrc, f"-j{max(8, os.cpu_count() or 8)}", target] + (["-B"] if force else []),
+                              stdout=subprocess.DEVNULL)
     return LIB_PATH
 
 
@@ -186,6 +189,11 @@ class Context:
         b = DevBuf(self, p.value, arr.nbytes, arr.shape, arr.dtype)
         self._owned.append(b)
         return b
+
+    def release(self, buf: DevBuf):
+        """Free an allocation of this context before the context goes."""
+        self._owned = [b for b in self._owned if b is not buf]
+        buf.free()
 
     @staticmethod
     def _ptr(x):

@@ -393,6 +393,7 @@ int md_set_option(md_ctx* ctx, const char* key, long value) {
     if (!strcmp(key, "decode_split_ln")) { ctx->decode_split_ln = (int)value; return MD_OK; }
     if (!strcmp(key, "fused_decode")) { ctx->fused_decode = value ? 1 : 0; return MD_OK; }
     if (!strcmp(key, "pdl")) { ctx->pdl = value ? 1 : 0; return MD_OK; }
+    if (!strcmp(key, "stack_trace")) { ctx->stack_trace = value ? 1 : 0; return MD_OK; }
     if (!strcmp(key, "prefill_fork")) { ctx->prefill_fork = value ? 1 : 0; return MD_OK; }
     if (!strcmp(key, "decode_fork")) { ctx->decode_fork = value ? 1 : 0; return MD_OK; }
     if (!strcmp(key, "push_tma")) { ctx->push_tma = value ? 1 : 0; return MD_OK; }

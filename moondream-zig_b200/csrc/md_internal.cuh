@@ -93,6 +93,7 @@ struct md_ctx {
     int decode_cluster_ok = -1;    // -1 unknown, 0/1: 16-CTA clusters usable for the decode attention merge
     int decode_cluster_mode = -1;  // md_set_option("decode_cluster"): 0 forces the scratch-based merge
     int dualk_variant = 0;   // md_set_option("dualk_variant"): (warps, unroll) of gemv_dual_k_kernel
+    int stack_trace = 0;     // md_set_option("stack_trace"): md_text_step keeps the residual stream after every layer
     int fused_decode = 1;    // md_set_option("fused_decode"): decode layers as 3 fused kernels
     int pdl = 0;             // md_set_option("pdl"): programmatic dependent launch for the GEMV kernels
     int prefill_fork = 1;       // md_set_option("prefill_fork"): prefill layers run the MLP beside the attention

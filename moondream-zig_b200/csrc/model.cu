@@ -1,13 +1,13 @@
 // Device-resident restatement of the reference's model control flow on top of the hot-path
-// kernels: text_model.zig:106-345 (text_encoder, text_decoder, lm_head, KVCache) and
+// kernels (and, for models described layer by layer, of stack.cu): text_model.zig:106-345 (text_encoder, text_decoder, lm_head, KVCache) and
 // vision_model.zig:160-387 (normalise, patchify, vision_encoder, encode_mlp), plus the greedy
 // generation loop of moondream.zig:323-368.  Host code + a few tiny kernels; every matmul goes
 // through md_gemm_dispatch (GEMV for <= 8 rows, tcgen05 GEMM otherwise) with the reference's
 // glue fused into the epilogue at the reference's rounding points.
-#include "md_internal.cuh"
+#include "stack.cuh"
+#include "text_model.cuh"
 
-#include "../../include/moondream_b200_model.h"
-
+#include <algorithm>
 #include <cstring>
 
 extern "C" int md_gemm_dispatch(md_ctx* ctx, const __half* a, const __half* b, __half* c, size_t M, size_t N, size_t K,
@@ -54,6 +54,7 @@ advance_kernel(unsigned long long* cur_tokens, unsigned long long* sampled, int 
     }
     __syncthreads();
     if (b == 0) *step = s + 1;
+    if (!wte) return;   // the next step gathers its embedding rows itself
     // the embedding rows of the next tokens; 16 bytes per thread where the rows allow it, all rows requested at once
     if ((dim & 7) == 0 && ((reinterpret_cast<uintptr_t>(wte) | reinterpret_cast<uintptr_t>(hidden)) & 15) == 0) {
         const int vec = dim >> 3;
@@ -70,33 +71,17 @@ advance_kernel(unsigned long long* cur_tokens, unsigned long long* sampled, int 
     }
 }
 
-__global__ void copy_logits_kernel(const __half* __restrict__ logits, __half* __restrict__ all, int vocab,
-                                   const int* step) {
-    __half* dst = all + (size_t)(*step) * vocab;
+template <class T>
+__global__ void copy_logits_kernel(const T* __restrict__ logits, T* __restrict__ all, int vocab, const int* step) {
+    T* dst = all + (size_t)(*step) * vocab;
     for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < vocab; i += gridDim.x * blockDim.x) dst[i] = logits[i];
 }
 
 __global__ void set_int_kernel(int* p, int v) { *p = v; }
-
-struct DevPtr {
-    void* p = nullptr;
-    size_t cap = 0;
-    ~DevPtr() { if (p) cudaFree(p); }
-    int ensure(md_ctx* ctx, size_t bytes) {
-        if (cap >= bytes) return MD_OK;
-        if (ctx->capturing) return md_fail(ctx, MD_ERR_UNSUPPORTED, "buffer growth during graph capture");
-        if (p) {
-            MD_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
-            MD_CUDA(ctx, cudaFree(p));
-            p = nullptr;
-            cap = 0;
-        }
-        MD_CUDA(ctx, cudaMalloc(&p, bytes));
-        cap = bytes;
-        return MD_OK;
-    }
-    template <class T> T* as() const { return reinterpret_cast<T*>(p); }
-};
+__global__ void add_int_kernel(int* p, int v) { *p += v; }
+__global__ void widen_kernel(const __half* __restrict__ x, float* __restrict__ y, int n) {
+    for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < n; i += gridDim.x * blockDim.x) y[i] = __half2float(x[i]);
+}
 
 template <class T> std::vector<T> copy_ptrs(const T* src, size_t n) { return std::vector<T>(src, src + n); }
 
@@ -111,42 +96,7 @@ int copy_out(md_ctx* ctx, void* user, const void* dev, size_t bytes) {
 
 // ------------------------------------------------------------------------------------ text
 
-struct md_text_model {
-    md_ctx* ctx;
-    md_text_weights w;
-    std::vector<const uint16_t*> ln_w, ln_b, wqkv, bqkv, wout, bout, wfc1, bfc1, wfc2, bfc2;
-};
-
-struct md_text_request {
-    md_text_model* model;
-    std::vector<__half*> kc, vc;  // per layer [n_heads][max_seq][head_dim]
-    size_t pos = 0;               // host mirror of *pos_dev
-    int* pos_dev = nullptr;
-    // activations of one forward over `rows` rows
-    DevPtr hidden, ln, qkv, attn, attn_out, fc1, logits, ln_last;
-    DevPtr mlp_part;  // up to four f32 [8, dim] partial products of fc2 (the decode layer whose MLP runs as two half-width chains)
-    // device-side generation state
-    DevPtr cur_token, sampled, tokens_out, forced, step, logits_all, pos_ptrs;
-    md_graph* graph = nullptr;
-    uint64_t graph_gen = 0, prefill_graph_gen = 0;  // md_ctx::generation the graphs were captured under
-    size_t graph_steps = 0;
-    bool graph_forced = false, graph_logits = false;
-    // a prefill of the same shape at the same position seen twice is captured and replayed
-    md_graph* prefill_graph = nullptr;
-    size_t prefill_S = 0, prefill_pos = 0, seen_S = 0, seen_pos = ~(size_t)0;
-};
-
 namespace {
-
-// While alive, the kernels that implement the programmatic-dependent-launch protocol (GEMV, tcgen05 GEMM and
-// attention, LayerNorm, rope) are launched dependent on their predecessor: each starts its set-up while the
-// previous one drains and waits (griddepcontrol.wait) before touching global memory.
-struct PdlScope {
-    md_ctx* c;
-    int old;
-    explicit PdlScope(md_ctx* cc) : c(cc), old(cc->pdl) { c->pdl = 1; }
-    ~PdlScope() { c->pdl = old; }
-};
 
 // Overrides the automatic (warps, unroll) choice of the GEMV kernel for a scope, unless the caller fixed one.
 struct GemvVariantScope {
@@ -403,6 +353,34 @@ int text_lm_head(md_text_model* m, const __half* hidden_rows, size_t rows, __hal
     return MD_OK;
 }
 
+// Run `body` (a forward over S rows at pos0 into the request's buffers).  The second forward of a shape is recorded and
+// replayed from then on: the ~170 launches are host-bound when issued one by one.
+template <class F>
+int run_captured(md_text_request* req, size_t S, size_t pos0, F&& body) {
+    md_ctx* ctx = req->model->ctx;
+    if (req->prefill_graph && req->prefill_S == S && req->prefill_pos == pos0 && req->prefill_graph_gen == ctx->generation)
+        return md_graph_launch(ctx, req->prefill_graph);
+    MD_TRY(body());
+    if (!ctx->capturing && req->seen_S == S && req->seen_pos == pos0) {
+        if (req->prefill_graph) { md_graph_destroy(ctx, req->prefill_graph); req->prefill_graph = nullptr; }
+        MD_TRY(md_graph_begin(ctx));
+        const int st = body();
+        md_graph* g = nullptr;
+        const int st2 = md_graph_end(ctx, &g);
+        if (st == MD_OK && st2 == MD_OK) {
+            req->prefill_graph = g;
+            req->prefill_graph_gen = ctx->generation;
+            req->prefill_S = S;
+            req->prefill_pos = pos0;
+        } else if (g) {
+            md_graph_destroy(ctx, g);
+        }
+    }
+    req->seen_S = S;
+    req->seen_pos = pos0;
+    return MD_OK;
+}
+
 }  // namespace
 
 extern "C" {
@@ -427,6 +405,7 @@ int md_text_model_create(md_ctx* ctx, const md_text_weights* w, md_text_model** 
 }
 
 int md_text_model_destroy(md_text_model* model) {
+    if (model && model->stack) md_stack_destroy(model->stack);
     delete model;
     return MD_OK;
 }
@@ -438,7 +417,14 @@ int md_text_request_create(md_text_model* model, md_text_request** out) {
     md_text_request* r = new md_text_request();
     r->model = model;
     const size_t cache_bytes = w.n_heads * w.max_seq * w.head_dim * 2;
-    for (size_t l = 0; l < w.n_layers; ++l) {
+    if (model->stack) {
+        const int st = md_stack_request_create(r);
+        if (st != MD_OK) {
+            md_text_request_destroy(r);
+            return st;
+        }
+    }
+    for (size_t l = 0; l < w.n_layers && !model->stack; ++l) {
         void *k = nullptr, *v = nullptr;
         if (cudaMalloc(&k, cache_bytes) != cudaSuccess || cudaMalloc(&v, cache_bytes) != cudaSuccess) {
             cudaGetLastError();
@@ -454,7 +440,7 @@ int md_text_request_create(md_text_model* model, md_text_request** out) {
         return md_fail(ctx, MD_ERR_OOM, "request state allocation failed");
     }
     cudaMemsetAsync(r->pos_dev, 0, sizeof(int), ctx->stream);
-    int st = ensure_rows(r, 8);
+    int st = model->stack ? r->logits.ensure(ctx, 8 * w.vocab * sizeof(float)) : ensure_rows(r, 8);
     if (st == MD_OK) st = r->cur_token.ensure(ctx, 8 * sizeof(unsigned long long));
     if (st == MD_OK) st = r->sampled.ensure(ctx, 8 * sizeof(unsigned long long));
     if (st == MD_OK) st = r->step.ensure(ctx, sizeof(int));
@@ -475,6 +461,7 @@ int md_text_request_destroy(md_text_request* req) {
     for (auto p : req->kc) cudaFree(p);
     for (auto p : req->vc) cudaFree(p);
     if (req->pos_dev) cudaFree(req->pos_dev);
+    if (req->stack) md_stack_request_destroy(req);
     delete req;
     return MD_OK;
 }
@@ -484,7 +471,7 @@ int md_text_request_reset(md_text_request* req) {
     md_ctx* ctx = req->model->ctx;
     req->pos = 0;
     MD_CUDA(ctx, cudaMemsetAsync(req->pos_dev, 0, sizeof(int), ctx->stream));
-    return MD_OK;
+    return req->stack ? md_stack_request_reset(req) : MD_OK;
 }
 
 int md_text_request_len(const md_text_request* req, size_t* len_out) {
@@ -497,6 +484,7 @@ int md_text_encoder(md_text_model* model, const uint32_t* ids, size_t n, uint16_
     if (!model) return MD_ERR_INVALID_ARG;
     md_ctx* ctx = model->ctx;
     if (!ids || !out) return md_fail(ctx, MD_ERR_INVALID_ARG, "text_encoder: null pointer");
+    if (model->stack) return md_fail(ctx, MD_ERR_UNSUPPORTED, "text_encoder: this model reads token ids (md_text_step)");
     const md_text_weights& w = model->w;
     if (n > w.max_seq) return md_fail(ctx, MD_ERR_SEQUENCE_TOO_LONG, "text_encoder: %zu ids > %zu", n, w.max_seq);
     std::vector<unsigned long long> wide(n);
@@ -526,6 +514,7 @@ int md_text_forward(md_text_model* model, md_text_request* req, const uint16_t* 
     md_ctx* ctx = model->ctx;
     const md_text_weights& w = model->w;
     if (!embeds || S == 0) return md_fail(ctx, MD_ERR_INVALID_ARG, "text_forward: no input rows");
+    if (model->stack) return md_fail(ctx, MD_ERR_UNSUPPORTED, "text_forward: this model reads token ids (md_text_step)");
     if (req->pos + S > w.max_seq)
         return md_fail(ctx, MD_ERR_SEQUENCE_TOO_LONG, "text_forward: %zu cached + %zu new tokens exceed %zu", req->pos, S,
                        w.max_seq);
@@ -543,30 +532,8 @@ int md_text_forward(md_text_model* model, md_text_request* req, const uint16_t* 
         MD_LAUNCH_CHECK(ctx, "set_int_kernel");
         return MD_OK;
     };
-    if (S > 1 && req->prefill_graph && req->prefill_S == S && req->prefill_pos == pos0 &&
-        req->prefill_graph_gen == ctx->generation) {
-        MD_TRY(md_graph_launch(ctx, req->prefill_graph));
-    } else {
-        MD_TRY(body());
-        if (S > 1 && !ctx->capturing && req->seen_S == S && req->seen_pos == pos0) {
-            // second prefill of this shape: record it (the ~170 launches are host-bound when issued one by one)
-            if (req->prefill_graph) { md_graph_destroy(ctx, req->prefill_graph); req->prefill_graph = nullptr; }
-            MD_TRY(md_graph_begin(ctx));
-            const int st = body();
-            md_graph* g = nullptr;
-            const int st2 = md_graph_end(ctx, &g);
-            if (st == MD_OK && st2 == MD_OK) {
-                req->prefill_graph = g;
-                req->prefill_graph_gen = ctx->generation;
-                req->prefill_S = S;
-                req->prefill_pos = pos0;
-            } else if (g) {
-                md_graph_destroy(ctx, g);
-            }
-        }
-        req->seen_S = S;
-        req->seen_pos = pos0;
-    }
+    if (S > 1) MD_TRY(run_captured(req, S, pos0, body));
+    else MD_TRY(body());
     req->pos = pos0 + S;
     MD_TRY(copy_out(ctx, hidden_out, req->hidden.p, S * w.dim * 2));
     if (logits_out || token_out) {
@@ -578,6 +545,86 @@ int md_text_forward(md_text_model* model, md_text_request* req, const uint16_t* 
     return md_check_flags(ctx);
 }
 
+int md_text_step(md_text_model* model, md_text_request* req, const uint32_t* tokens, size_t n, const uint32_t* want,
+                 size_t n_want, float* logits_out, uint64_t* token_out) {
+    if (!model || !req) return MD_ERR_INVALID_ARG;
+    md_ctx* ctx = model->ctx;
+    const md_text_weights& w = model->w;
+    if (req->model != model) return md_fail(ctx, MD_ERR_INVALID_ARG, "text_step: foreign request");
+    if (!tokens || n == 0) return md_fail(ctx, MD_ERR_INVALID_ARG, "text_step: no tokens");
+    if (n_want && (!want || !logits_out)) return md_fail(ctx, MD_ERR_INVALID_ARG, "text_step: null pointer");
+    if (req->pos + n > w.max_seq)
+        return md_fail(ctx, MD_ERR_SEQUENCE_TOO_LONG, "text_step: %zu cached + %zu new tokens exceed %zu", req->pos, n, w.max_seq);
+    // the rows whose logits are computed: the wanted ones, and the last one if its sample is asked for
+    std::vector<int> rows(want, want + n_want);
+    for (int r : rows)
+        if ((size_t)r >= n) return md_fail(ctx, MD_ERR_INVALID_ARG, "text_step: wanted row %d of %zu", r, n);
+    if (n_want > n) return md_fail(ctx, MD_ERR_INVALID_ARG, "text_step: %zu wanted rows of %zu", n_want, n);
+    if (token_out) rows.push_back((int)n - 1);
+    std::vector<unsigned long long> ids(n);
+    for (size_t i = 0; i < n; ++i) {
+        if (tokens[i] >= w.vocab) return md_fail(ctx, MD_ERR_INVALID_ARG, "text_step: token id %u out of bounds", tokens[i]);
+        ids[i] = tokens[i];
+    }
+    const size_t pos0 = req->pos, rows_cap = std::max<size_t>(n + 1, 8), n_rows = rows.size();
+    if (model->stack) MD_TRY(md_stack_reserve(req, rows_cap));
+    else MD_TRY(ensure_rows(req, rows_cap));
+    const size_t ids_bytes = (rows_cap * sizeof(ids[0]) + 255) & ~(size_t)255;
+    if (req->cur_token.cap < ids_bytes + rows_cap * sizeof(int)) {   // moves: recorded steps are stale
+        if (req->graph) { md_graph_destroy(ctx, req->graph); req->graph = nullptr; }
+        if (req->prefill_graph) { md_graph_destroy(ctx, req->prefill_graph); req->prefill_graph = nullptr; }
+        MD_TRY(req->cur_token.ensure(ctx, ids_bytes + 2 * rows_cap * sizeof(int)));
+    }
+    unsigned long long* ids_dev = req->cur_token.as<unsigned long long>();
+    MD_CUDA(ctx, cudaMemcpyAsync(ids_dev, ids.data(), n * sizeof(ids[0]), cudaMemcpyHostToDevice, ctx->stream));
+    auto body = [&]() -> int {
+        PdlScope pdl_scope(ctx);
+        if (model->stack) {
+            MD_TRY(md_stack_layers(model, &req, 1, n, ids_dev, n == 1, pos0));
+        } else {
+            embed_kernel<<<(unsigned)n, 256, 0, ctx->stream>>>(H(w.wte), ids_dev, req->hidden.as<__half>(), (int)w.dim, (int)w.vocab);
+            MD_LAUNCH_CHECK(ctx, "embed_kernel");
+            const LayerIO io = io_of(req);
+            for (size_t l = 0; l < w.n_layers; ++l) MD_TRY(text_layer(model, l, io, n, n == 1, &req, pos0));
+        }
+        add_int_kernel<<<1, 1, 0, ctx->stream>>>(req->pos_dev, (int)n);
+        MD_LAUNCH_CHECK(ctx, "add_int_kernel");
+        return MD_OK;
+    };
+    // a decoded token finds its position in device memory, so one recording serves every position
+    if (ctx->stack_trace) MD_TRY(body());
+    else MD_TRY(run_captured(req, n, n == 1 ? 0 : pos0, body));
+    req->pos = pos0 + n;
+    if (n_rows) {
+        PdlScope pdl_scope(ctx);
+        if (req->logits_all.cap < n_rows * w.vocab * sizeof(float)) MD_TRY(req->logits_all.ensure(ctx, n_rows * w.vocab * sizeof(float)));
+        float* logits = req->logits_all.as<float>();
+        if (model->stack) {
+            int* rows_dev = reinterpret_cast<int*>(req->cur_token.as<char>() + ids_bytes);
+            MD_CUDA(ctx, cudaMemcpyAsync(rows_dev, rows.data(), n_rows * sizeof(int), cudaMemcpyHostToDevice, ctx->stream));
+            MD_TRY(md_stack_head(model, req, n, rows_dev, n_rows, logits));
+        } else {
+            for (size_t i = 0; i < n_rows; ++i) {
+                MD_TRY(text_lm_head(model, req->hidden.as<__half>() + (size_t)rows[i] * w.dim, 1, req->ln_last.as<__half>(),
+                                    req->logits.as<__half>(), req->sampled.as<unsigned long long>()));
+                widen_kernel<<<64, 256, 0, ctx->stream>>>(req->logits.as<__half>(), logits + i * w.vocab, (int)w.vocab);
+                MD_LAUNCH_CHECK(ctx, "widen_kernel");
+            }
+        }
+        if (token_out)
+            MD_TRY(md_launch_argmax_f32(ctx, logits + (n_rows - 1) * w.vocab, w.vocab, w.vocab, 1, req->sampled.as<unsigned long long>()));
+        MD_TRY(copy_out(ctx, logits_out, logits, n_want * w.vocab * sizeof(float)));
+        if (token_out) MD_TRY(copy_out(ctx, token_out, req->sampled.p, sizeof(uint64_t)));
+    }
+    return md_check_flags(ctx);
+}
+
+int md_text_layer_stream(md_text_request* req, size_t layer, float* out, size_t rows) {
+    if (!req) return MD_ERR_INVALID_ARG;
+    if (!req->stack) return md_fail(req->model->ctx, MD_ERR_UNSUPPORTED, "md_text_layer_stream: layer-stack models only");
+    return md_stack_copy_stream(req, layer, out, rows);
+}
+
 // Enqueue one decode step for `batch` requests that share the activation buffers of reqs[0].
 static int enqueue_decode_step(md_text_model* model, md_text_request* const* reqs, size_t batch, size_t n_steps,
                                bool forced, bool keep_logits) {
@@ -586,6 +633,22 @@ static int enqueue_decode_step(md_text_model* model, md_text_request* const* req
     md_text_request* r0 = reqs[0];
     // registered weights are never written on this stream: the GEMVs may overlap their predecessors' tails
     PdlScope pdl_scope(ctx);
+    if (model->stack) {
+        float* logits = r0->logits.as<float>();
+        MD_TRY(md_stack_layers(model, reqs, batch, 1, r0->cur_token.as<unsigned long long>(), true, 0));
+        MD_TRY(md_stack_head(model, r0, batch, nullptr, batch, logits));
+        MD_TRY(md_launch_argmax_f32(ctx, logits, w.vocab, w.vocab, batch, r0->sampled.as<unsigned long long>()));
+        if (keep_logits) {
+            copy_logits_kernel<float><<<32, 256, 0, ctx->stream>>>(logits, r0->logits_all.as<float>(), (int)w.vocab, r0->step.as<int>());
+            MD_LAUNCH_CHECK(ctx, "copy_logits_kernel");
+        }
+        advance_kernel<<<1, 256, 0, ctx->stream>>>(r0->cur_token.as<unsigned long long>(), r0->sampled.as<unsigned long long>(), 0,
+                                                   (int)batch, r0->tokens_out.as<unsigned int>(), (int)n_steps,
+                                                   forced ? r0->forced.as<unsigned int>() : nullptr, r0->step.as<int>(),
+                                                   r0->pos_ptrs.as<int*>(), nullptr, nullptr, (int)w.dim, (int)w.vocab);
+        MD_LAUNCH_CHECK(ctx, "advance_kernel");
+        return MD_OK;
+    }
     // hidden already holds the embeddings of the current tokens (generate_impl / the previous advance_kernel)
     const LayerIO io = io_of(r0);
     const bool ln_once = ctx->decode_split_ln > 0 && batch >= (size_t)ctx->decode_split_ln;
@@ -605,7 +668,7 @@ static int enqueue_decode_step(md_text_model* model, md_text_request* const* req
                             r0->sampled.as<unsigned long long>()));
     }
     if (keep_logits) {
-        copy_logits_kernel<<<32, 256, 0, ctx->stream>>>(r0->logits.as<__half>(), r0->logits_all.as<__half>(),
+        copy_logits_kernel<__half><<<32, 256, 0, ctx->stream>>>(r0->logits.as<__half>(), r0->logits_all.as<__half>(),
                                                         (int)w.vocab, r0->step.as<int>());
         MD_LAUNCH_CHECK(ctx, "copy_logits_kernel");
     }
@@ -634,10 +697,11 @@ static int generate_impl(md_text_model* model, md_text_request* const* reqs, siz
         if (first[b] >= w.vocab) return md_fail(ctx, MD_ERR_INVALID_ARG, "generate: token id %u out of bounds", first[b]);
     }
     md_text_request* r0 = reqs[0];
-    MD_TRY(ensure_rows(r0, 8));
+    const size_t logit_bytes = model->stack ? sizeof(float) : sizeof(__half);
+    if (!model->stack) MD_TRY(ensure_rows(r0, 8));
     MD_TRY(r0->tokens_out.ensure(ctx, batch * n_steps * sizeof(unsigned int)));
     if (forced) MD_TRY(r0->forced.ensure(ctx, batch * n_steps * sizeof(unsigned int)));
-    if (logits_out) MD_TRY(r0->logits_all.ensure(ctx, n_steps * w.vocab * 2));
+    if (logits_out) MD_TRY(r0->logits_all.ensure(ctx, n_steps * w.vocab * logit_bytes));
     MD_TRY(r0->pos_ptrs.ensure(ctx, 8 * sizeof(int*)));
     // device-side state of the loop
     unsigned long long cur[8] = {0};
@@ -650,9 +714,11 @@ static int generate_impl(md_text_model* model, md_text_request* const* reqs, siz
     MD_CUDA(ctx, cudaMemcpyAsync(r0->pos_ptrs.p, pos_ptrs, sizeof(pos_ptrs), cudaMemcpyHostToDevice, ctx->stream));
     MD_CUDA(ctx, cudaMemsetAsync(r0->step.p, 0, sizeof(int), ctx->stream));
     MD_CUDA(ctx, cudaMemsetAsync(r0->sampled.p, 0, 8 * sizeof(unsigned long long), ctx->stream));
-    embed_kernel<<<(unsigned)batch, 256, 0, ctx->stream>>>(H(w.wte), r0->cur_token.as<unsigned long long>(),
-                                                           r0->hidden.as<__half>(), (int)w.dim, (int)w.vocab);
-    MD_LAUNCH_CHECK(ctx, "embed_kernel");
+    if (!model->stack) {
+        embed_kernel<<<(unsigned)batch, 256, 0, ctx->stream>>>(H(w.wte), r0->cur_token.as<unsigned long long>(),
+                                                               r0->hidden.as<__half>(), (int)w.dim, (int)w.vocab);
+        MD_LAUNCH_CHECK(ctx, "embed_kernel");
+    }
     if (forced)
         MD_CUDA(ctx, cudaMemcpyAsync(r0->forced.p, forced, batch * n_steps * sizeof(unsigned int), cudaMemcpyHostToDevice,
                                      ctx->stream));
@@ -692,7 +758,7 @@ static int generate_impl(md_text_model* model, md_text_request* const* reqs, siz
     MD_CUDA(ctx, cudaMemcpyAsync(tokens_out, r0->tokens_out.p, batch * n_steps * sizeof(unsigned int),
                                  cudaMemcpyDeviceToHost, ctx->stream));
     if (logits_out)
-        MD_CUDA(ctx, cudaMemcpyAsync(logits_out, r0->logits_all.p, n_steps * w.vocab * 2, cudaMemcpyDeviceToHost,
+        MD_CUDA(ctx, cudaMemcpyAsync(logits_out, r0->logits_all.p, n_steps * w.vocab * logit_bytes, cudaMemcpyDeviceToHost,
                                      ctx->stream));
     const int st = md_check_flags(ctx);
     if (graph && batch != 1) md_graph_destroy(ctx, graph);

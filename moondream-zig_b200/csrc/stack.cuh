@@ -1,0 +1,166 @@
+// Internal declarations of the layer-stack decoders: text models described layer by layer (md_stack_weights of
+// moondream_b200_model.h) instead of by one fixed layout.  The kernels are generic over the element type of weights and
+// activations, T = __nv_bfloat16 (served) or float (every product in true 32-bit); the residual stream, norms, attention
+// scores, recurrent states and routers are f32 in both.
+#pragma once
+
+#include <cuda_bf16.h>
+
+#include "md_internal.cuh"
+
+#include "../../include/moondream_b200_model.h"
+
+constexpr int MD_STACK_MAX_SEQS = 8;     // requests advanced together by one step
+constexpr int MD_STACK_MAX_TAPS = 8;
+constexpr int MD_GROUP_ROWS = 128;       // an expert's rows in the sorted buffers start at a multiple of this
+
+// ---- linear layers: C[M,N] = act(A[M,K] . W[N,K]^T + bias) --------------------------------------------------
+struct md_lin {
+    const float* bias = nullptr;     // [N] or null
+    int silu_cols = 0;               // columns < silu_cols go through silu
+    int sigmoid_from = 1 << 30;      // columns >= sigmoid_from go through the logistic function
+    // glu != 0: W's rows are gate and up rows in alternating blocks of 32 (MD_GLU_BLOCK) and C[M, N/2] = act(gate) * up
+    int glu = 0;                     // MD_ACT_*
+    float* out_f32 = nullptr;        // write f32 sums here instead of T to C
+    // rows sorted by expert: row block b (128 rows) belongs to expert tile_expert[b], whose matrix is W + e * N * K;
+    // only the first *n_blocks blocks are computed
+    const int* tile_expert = nullptr;
+    const int* n_blocks = nullptr;
+    int n_experts = 0;
+};
+constexpr int MD_GLU_BLOCK = 32;
+int md_linear(md_ctx* ctx, int dtype, const void* a, const void* w, void* c, size_t M, size_t N, size_t K, const md_lin& ep);
+
+// ---- residual + norms + causal convolution ---------------------------------------------------------------
+// For every row t of a sequence:
+//   x_out[t] = x[t] + mult * rms_norm(y[t]; w_post)             (y == null: x_out = x; tokens != null: x = embed[token])
+//   n[t]     = rms_norm(x_out[t]; w_pre)
+//   out[t]   = n[t] + sum_j conv[j] * n[t - taps + 1 + j]       (conv == null: out = n)
+// The convolution's last taps - 1 inputs live in `state` ([taps - 1][width] f32) between calls.
+struct md_glue {
+    int width = 0, rows = 0, taps = 0;      // rows per sequence
+    float eps = 0.f, mult = 0.f;
+    const float* x = nullptr;               // [seqs * rows, width]
+    float* x_out = nullptr;                 // must differ from x when rows > 1
+    const void* embed = nullptr;            // [vocab, width] T
+    const unsigned long long* tokens = nullptr;
+    int vocab = 0;
+    // the sublayer's output, one of: f32 rows, T rows, or T rows of the expert-sorted buffer
+    const float* y_f32 = nullptr;
+    const void* y = nullptr;
+    const float* w_post = nullptr;
+    // y is scaled per row by 1 / sqrt(sum(ssq) / ssq_n + eps) (the norm ahead of the output projection, applied after it)
+    const float* ssq = nullptr;             // [rows, ssq_parts]
+    int ssq_parts = 0, ssq_n = 0;
+    // mixture of experts: y of row t = sum_k score[t][k] * y[slot[t][k]]
+    const int* slot = nullptr;              // [rows, top]
+    const float* score = nullptr;
+    int top = 0;
+    const float* w_pre = nullptr;
+    const float* conv = nullptr;            // [taps][width]
+    void* out = nullptr;                    // [seqs * rows, width] T
+    const int* gather = nullptr;            // rows to take (final norm of the wanted rows): x row = gather[i], no x_out
+    int seqs = 1;
+    float* state[MD_STACK_MAX_SEQS] = {};
+};
+int md_launch_glue(md_ctx* ctx, int dtype, const md_glue& g);
+
+// ---- attention: distance bias, sliding window with kept first keys, values = keys, gated heads -------------
+struct md_win_attn {
+    int heads = 0, kv_heads = 0, dim = 0;
+    float scale = 0.f;
+    int window = 0, keep_first = 0;         // window <= 0: unlimited
+    const float *r1 = nullptr, *r2 = nullptr;
+    const void* qkg = nullptr;              // rows [q: heads * dim | k: kv_heads * dim | gate: heads (logistic applied)]
+    int row_stride = 0;
+    void* out = nullptr;                    // [rows, heads * dim] T
+    int rows = 0;                           // per sequence
+    size_t max_seq = 0;
+    int seqs = 1;
+    void* kc[MD_STACK_MAX_SEQS] = {};       // [kv_heads][max_seq][dim] T
+    const int* pos_dev[MD_STACK_MAX_SEQS] = {};   // decode: position of the new token
+    int pos0 = 0;                           // prefill: position of row 0
+};
+int md_launch_window_attention(md_ctx* ctx, int dtype, const md_win_attn& a, bool decode);
+
+// ---- linear attention with per-head decay ----------------------------------------------------------------
+struct md_lightning {
+    int heads = 0, dim = 0, vdim = 0;
+    const float* decay = nullptr;           // [heads] device
+    const float* norm_w = nullptr;          // [heads * vdim]
+    const void* qkvg = nullptr;             // rows [q | k | v (all through silu) | g (logistic applied)]
+    int row_stride = 0;
+    void* out = nullptr;                    // [rows, heads * vdim] T: o * norm_w * gate, not yet divided by its rms
+    float* ssq = nullptr;                   // [rows, ssq_parts]: sums of o^2
+    int ssq_parts = 0;
+    int rows = 0, seqs = 1;
+    float* state[MD_STACK_MAX_SEQS] = {};   // [heads][dim][vdim] f32
+};
+// number of ssq entries a row has for these sizes
+int md_lightning_ssq_parts(int heads, int vdim);
+int md_launch_lightning(md_ctx* ctx, int dtype, const md_lightning& l, bool decode);
+
+// ---- mixture of experts --------------------------------------------------------------------------------------
+struct md_moe {
+    int width = 0, experts = 0, top = 0, ff = 0, ff_pad = 0, act = 0;
+    const void *router = nullptr, *w_gu = nullptr, *w_down = nullptr;   // [E, W], [E, 2 ff_pad, W], [E, W, ff_pad]
+};
+struct md_moe_buffers {
+    float* score = nullptr;       // [rows, top]
+    int *sel = nullptr, *rank = nullptr, *slot = nullptr;     // [rows, top]
+    int *count = nullptr;         // [experts]
+    int *tile_expert = nullptr, *n_blocks = nullptr;
+    void *xs = nullptr, *act = nullptr, *ys = nullptr;        // sorted rows
+    float* y_f32 = nullptr;       // [rows, width] (decode)
+};
+size_t md_moe_sorted_rows(size_t rows, int experts, int top);   // capacity of the sorted buffers
+// true: md_launch_moe leaves a token's outputs in the sorted rows (slot, score, ys); false: their sum in y_f32
+bool md_moe_sorted(int dtype, size_t rows);
+int md_launch_moe(md_ctx* ctx, int dtype, const md_moe& m, const void* h, size_t rows, const md_moe_buffers& b);
+
+int md_launch_argmax_f32(md_ctx* ctx, const float* x, size_t n, size_t stride, size_t rows, unsigned long long* idx_dev);
+
+#ifdef __CUDACC__
+template <class T> struct md_elem;
+template <> struct md_elem<__nv_bfloat16> {
+    static __device__ __forceinline__ float get(__nv_bfloat16 v) { return __bfloat162float(v); }
+    static __device__ __forceinline__ __nv_bfloat16 put(float v) { return __float2bfloat16_rn(v); }
+};
+template <> struct md_elem<float> {
+    static __device__ __forceinline__ float get(float v) { return v; }
+    static __device__ __forceinline__ float put(float v) { return v; }
+};
+__device__ __forceinline__ float md_logistic(float z) { return 1.f / (1.f + expf(-z)); }
+__device__ __forceinline__ float md_silu(float z) { return z / (1.f + expf(-z)); }
+__device__ __forceinline__ float md_gelu_tanh(float z) {
+    return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+}
+__device__ __forceinline__ float md_act(int act, float z) { return act == MD_ACT_SILU ? md_silu(z) : md_gelu_tanh(z); }
+// column activation of md_lin
+__device__ __forceinline__ float md_lin_col(float v, int n, int silu_cols, int sigmoid_from) {
+    if (n < silu_cols) return md_silu(v);
+    if (n >= sigmoid_from) return md_logistic(v);
+    return v;
+}
+template <class T> __device__ __forceinline__ void md_load4(const T* p, float (&f)[4]);
+template <> __device__ __forceinline__ void md_load4<float>(const float* p, float (&f)[4]) {
+    const float4 v = __ldcg(reinterpret_cast<const float4*>(p));
+    f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
+}
+template <> __device__ __forceinline__ void md_load4<__nv_bfloat16>(const __nv_bfloat16* p, float (&f)[4]) {
+    const uint2 u = __ldcg(reinterpret_cast<const uint2*>(p));
+    f[0] = __uint_as_float(u.x << 16); f[1] = __uint_as_float(u.x & 0xffff0000u);
+    f[2] = __uint_as_float(u.y << 16); f[3] = __uint_as_float(u.y & 0xffff0000u);
+}
+__device__ __forceinline__ uint32_t md_pack_bf16(float lo, float hi) {
+    const __nv_bfloat162 h = __floats2bfloat162_rn(lo, hi);
+    return *reinterpret_cast<const uint32_t*>(&h);
+}
+template <class T> __device__ __forceinline__ void md_store4(T* p, const float (&f)[4]);
+template <> __device__ __forceinline__ void md_store4<float>(float* p, const float (&f)[4]) {
+    *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+}
+template <> __device__ __forceinline__ void md_store4<__nv_bfloat16>(__nv_bfloat16* p, const float (&f)[4]) {
+    *reinterpret_cast<uint2*>(p) = make_uint2(md_pack_bf16(f[0], f[1]), md_pack_bf16(f[2], f[3]));
+}
+#endif

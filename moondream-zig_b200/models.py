@@ -1,10 +1,16 @@
-"""ctypes binding of include/moondream_b200_model.h: the device-resident text decoder and
+"""ctypes binding of include/moondream_b200_model.h: the device-resident text decoders and
 vision encoder built on the hot-path kernels.  Weights are numpy f16 arrays laid out as the
 reference holds them (text matrices [out,in], vision matrices [in,out]); they are uploaded
-once at construction."""
+once at construction.
+
+``load_model`` opens a model folder: a config.json names the design in "architecture" and its registered builder reads
+model.safetensors; a folder with a moondream.bin gives the Phi-style TextModel.  StackModel is the binding of the
+layer-stack decoders (md_stack_weights), which share TextModel's requests, steps and generation."""
 from __future__ import annotations
 
 import ctypes as C
+import json
+import os
 
 import numpy as np
 
@@ -73,6 +79,8 @@ class TextRequest:
 
 
 class TextModel:
+    logits_dtype = np.float16    # of generate(want_logits=True)
+
     def __init__(self, ctx, weights: dict, n_heads: int = 32, max_seq: int = 2048, rot_dim: int | None = None,
                  theta: float = 10000.0, eps=np.float16(1e-5)):
         self.ctx, self.lib = ctx, ctx.lib
@@ -141,11 +149,23 @@ class TextModel:
             C.c_void_p(tok.ctypes.data)))
         return hidden, logits, int(tok[0])
 
+    def step(self, req: TextRequest, tokens, want=(), want_token: bool = False):
+        """md_text_step: run the next tokens of a request from the state it holds.  Returns (float32 logits
+        [len(want), vocab] at the wanted places, argmax of the last row or None)."""
+        tokens = np.ascontiguousarray(tokens, np.uint32)
+        want = np.ascontiguousarray(want, np.uint32)
+        logits = np.empty((want.size, self.vocab), np.float32)
+        tok = np.zeros(1, np.uint64)
+        self.ctx._check(self.lib.md_text_step(
+            self.h, req.h, C.c_void_p(tokens.ctypes.data), _sz(tokens.size), C.c_void_p(want.ctypes.data), _sz(want.size),
+            C.c_void_p(logits.ctypes.data if want.size else 0), C.c_void_p(tok.ctypes.data if want_token else 0)))
+        return logits, (int(tok[0]) if want_token else None)
+
     def generate(self, req: TextRequest, first: int, n_steps: int, forced=None, want_logits=False):
         """Greedy decode loop on the device (moondream.zig:323-368)."""
         toks = np.zeros(n_steps, np.uint32)
         f = np.ascontiguousarray(forced, np.uint32) if forced is not None else None
-        logits = np.empty((n_steps, self.vocab), np.float16) if want_logits else None
+        logits = np.empty((n_steps, self.vocab), self.logits_dtype) if want_logits else None
         self.ctx._check(self.lib.md_text_generate(
             self.h, req.h, C.c_uint32(int(first)), _sz(n_steps), C.c_void_p(toks.ctypes.data),
             C.c_void_p(f.ctypes.data if f is not None else 0), C.c_void_p(logits.ctypes.data if want_logits else 0)))
@@ -172,6 +192,175 @@ class TextModel:
         if getattr(self, "h", None):
             self.lib.md_text_model_destroy(self.h)
             self.h = None
+
+
+# ---------------------------------------------------------------- layer-stack decoders
+
+DTYPES = {"bfloat16": 1, "float32": 2}
+MIXER_WINDOW_ATTENTION, MIXER_LIGHTNING = 1, 2
+FF_NONE, FF_DENSE, FF_MOE = 0, 1, 2
+ACT_GELU_TANH, ACT_SILU = 1, 2
+
+
+class _StackLayer(C.Structure):
+    _fields_ = ([(n, C.c_int) for n in ("mixer", "ff")] +
+                [(n, C.c_size_t) for n in ("heads", "kv_heads", "dim", "vdim", "window", "keep_first")] +
+                [("scale", C.c_float)] + [(n, C.c_void_p) for n in ("r1", "r2", "decay", "mix_norm", "w_in", "b_in")] +
+                [("in_rows", C.c_size_t)] +
+                [(n, C.c_void_p) for n in ("w_out", "norm1", "norm1b", "norm2", "norm2b", "conv1", "conv2")] +
+                [("act", C.c_int), ("ff_dim", C.c_size_t), ("ff_pad", C.c_size_t)] +
+                [(n, C.c_void_p) for n in ("w_gate_up", "w_down", "router")] +
+                [("experts", C.c_size_t), ("top", C.c_size_t)])
+
+
+class _StackW(C.Structure):
+    _fields_ = ([("dtype", C.c_int)] + [(n, C.c_size_t) for n in ("n_layers", "width", "vocab", "max_seq", "taps")] +
+                [("eps", C.c_float), ("residual_mult", C.c_float)] +
+                [(n, C.c_void_p) for n in ("layers", "embed", "head", "final_norm")])
+
+
+class StackModel(TextModel):
+    """A text model described layer by layer (md_stack_model_create).  `layers`: one dict per layer with the fields of
+    md_stack_layer; arrays may be numpy (uint16 = bfloat16 bits, or floats) or CUDA torch tensors already of the model's
+    type, which are used in place."""
+    logits_dtype = np.float32
+    VECTORS = ("r1", "r2", "decay", "mix_norm", "b_in", "norm1", "norm1b", "norm2", "norm2b", "conv1", "conv2")
+    MATRICES = ("w_in", "w_out", "w_gate_up", "w_down", "router")
+
+    def __init__(self, ctx, layers: list, embed, head, final_norm, eps: float, residual_mult: float, taps: int,
+                 dtype: str = "bfloat16", max_seq: int = 2048):
+        if dtype not in DTYPES:
+            raise ValueError(f"dtype {dtype!r}: expected one of {sorted(DTYPES)}")
+        self.ctx, self.lib, self.dtype = ctx, ctx.lib, dtype
+        self.dev, self._keep, self._bufs = {}, [], []
+        table = (_StackLayer * len(layers))()
+        for s, d in zip(table, layers):
+            for n in ("mixer", "ff", "heads", "dim", "vdim"):
+                setattr(s, n, int(d[n]))
+            for n in ("kv_heads", "window", "keep_first", "act", "ff_dim", "experts", "top"):
+                setattr(s, n, int(d.get(n) or 0))
+            s.scale = float(d.get("scale") or 0.0)
+            s.in_rows = d["w_in"].shape[0]
+            if d["ff"] != FF_NONE:
+                s.ff_pad = d["w_down"].shape[-1]
+            for n in self.VECTORS:
+                if d.get(n) is not None:
+                    setattr(s, n, self._vector(d[n].T if n.startswith("conv") else d[n]))
+            for n in self.MATRICES:
+                if d.get(n) is not None:
+                    setattr(s, n, self._matrix(d[n]))
+        w = _StackW()
+        w.dtype, w.n_layers, w.width, w.vocab, w.max_seq, w.taps = (DTYPES[dtype], len(layers), embed.shape[1],
+                                                                    embed.shape[0], max_seq, taps)
+        w.eps, w.residual_mult = eps, residual_mult
+        w.layers = C.cast(table, C.c_void_p)
+        w.embed, w.head, w.final_norm = self._matrix(embed), self._matrix(head), self._vector(final_norm)
+        self.s = w
+        self.dim, self.vocab, self.n_layers = int(w.width), int(w.vocab), int(w.n_layers)
+        h = C.c_void_p()
+        ctx._check(self.lib.md_stack_model_create(ctx.h, C.byref(w), C.byref(h)))
+        self.h = h
+
+    @staticmethod
+    def widen(a: np.ndarray) -> np.ndarray:
+        """bfloat16 bits (uint16) or floats -> float32."""
+        a = np.ascontiguousarray(a)
+        if a.dtype == np.uint16:
+            return (a.astype(np.uint32) << 16).view(np.float32)
+        return a.astype(np.float32)
+
+    @staticmethod
+    def narrow(a: np.ndarray) -> np.ndarray:
+        """bfloat16 bits as they are, floats rounded to nearest even."""
+        a = np.ascontiguousarray(a)
+        if a.dtype == np.uint16:
+            return a
+        u = a.astype(np.float32).view(np.uint32)
+        return ((u + 0x7FFF + ((u >> 16) & 1)) >> 16).astype(np.uint16)
+
+    def _upload(self, a):
+        if hasattr(a, "data_ptr"):
+            assert a.is_cuda and a.is_contiguous()
+            b = _TorchBuf(a)
+        else:
+            b = self.ctx.upload(a)
+        self._bufs.append(b)
+        return b.ptr
+
+    def _matrix(self, a):
+        if hasattr(a, "data_ptr"):
+            assert a.element_size() == (4 if self.dtype == "float32" else 2)
+            return self._upload(a)
+        return self._upload(self.widen(a) if self.dtype == "float32" else self.narrow(a))
+
+    def _vector(self, a):
+        if hasattr(a, "data_ptr"):
+            return self._upload(a.float().contiguous())
+        return self._upload(self.widen(a))
+
+    def layer_stream(self, req: TextRequest, layer: int, rows: int) -> np.ndarray:
+        """Residual stream after `layer` of the last step (set the option "stack_trace" before it)."""
+        out = np.empty((rows, self.dim), np.float32)
+        self.ctx._check(self.lib.md_text_layer_stream(req.h, _sz(layer), C.c_void_p(out.ctypes.data), _sz(rows)))
+        return out
+
+    def close(self):
+        super().close()
+        for b in self._bufs:
+            if not isinstance(b, _TorchBuf):
+                self.ctx.release(b)
+        self._bufs = []
+
+
+# architecture name of a config.json -> builder(ctx, config, tensors, dtype=, max_seq=)
+MODELS: dict = {}
+
+
+def register_model(name: str):
+    def add(fn):
+        MODELS[name] = fn
+        return fn
+    return add
+
+
+def load_model(ctx, folder: str, dtype: str = "bfloat16", max_seq: int = 2048):
+    """The text model of a folder: config.json + model.safetensors of a registered architecture, or moondream.bin."""
+    from . import korupel, weights  # noqa: F401  (registers its architecture)
+    path = os.path.join(folder, "config.json")
+    if not os.path.exists(path) and os.path.exists(os.path.join(folder, "moondream.bin")):
+        return weights.WeightFile(os.path.join(folder, "moondream.bin")).upload(ctx).text_model()
+    with open(path) as f:
+        cfg = json.load(f)
+    name = cfg.get("architecture")
+    if name not in MODELS:
+        raise ValueError(f"architecture {name!r} is not one of {sorted(MODELS)}")
+    with weights.SafetensorsFile(os.path.join(folder, "model.safetensors")) as tensors:
+        return MODELS[name](ctx, cfg, tensors, dtype=dtype, max_seq=max_seq)
+
+
+class RequestPool:
+    """Requests of one model that are reused: a finished request's caches and states serve the next one."""
+
+    def __init__(self, model: TextModel):
+        self.model, self.free, self.live = model, [], {}
+
+    def get(self, key) -> TextRequest:
+        if key not in self.live:
+            if self.free:
+                r = self.free.pop()
+                r.reset()
+            else:
+                r = self.model.request()
+            self.live[key] = r
+        return self.live[key]
+
+    def end(self, key):
+        self.free.append(self.live.pop(key))
+
+    def close(self):
+        for r in self.free + list(self.live.values()):
+            r.close()
+        self.free, self.live = [], {}
 
 
 class VisionModel:

@@ -4,10 +4,13 @@ bytes as the reference's converter (weights.py:82-135: header, name, u64 dims, r
 
 The writer takes the two weight dictionaries the model classes use (per-layer lists of [out,in] text
 matrices and [in,out] vision matrices) and stacks the per-layer tensors on a leading axis, as
-weights.py:137-154 does."""
+weights.py:137-154 does.
+
+SafetensorsFile reads the tensors of the designs that come as config.json + model.safetensors."""
 from __future__ import annotations
 
 import ctypes as C
+import json
 import struct
 
 import numpy as np
@@ -93,6 +96,50 @@ def write_weight_file(path: str, text: dict, vision: dict) -> None:
             if name == "v_pos_embedding" and a.ndim == 2:
                 a = a[None]  # the file holds [1, tokens, dim] (weights.zig:455)
             write_tensor(f, name, a)
+
+
+class SafetensorsFile:
+    """Read-only mapping name -> array over a safetensors file (u64 header length, JSON header, data).  bfloat16 tensors
+    come as their uint16 bits, the other types as numpy arrays; the data stays in the mapped file until it is used."""
+
+    DTYPES = {"BF16": np.uint16, "F16": np.float16, "F32": np.float32, "F64": np.float64, "I32": np.int32, "I64": np.int64,
+              "U8": np.uint8}
+
+    def __init__(self, path: str):
+        self.path = path
+        self.data = np.memmap(path, np.uint8, "r")
+        if self.data.size < 8:
+            raise ValueError(f"{path}: no safetensors header")
+        n = int(self.data[:8].view("<u8")[0])
+        if n > self.data.size - 8:
+            raise ValueError(f"{path}: the header of {n} bytes does not fit the file")
+        self.header = json.loads(bytes(self.data[8:8 + n]))
+        self.header.pop("__metadata__", None)
+        self.base = 8 + n
+
+    def __enter__(self):
+        return self
+
+    def __exit__(self, *exc):
+        self.data = None
+
+    def __contains__(self, name):
+        return name in self.header
+
+    def keys(self):
+        return self.header.keys()
+
+    def __getitem__(self, name: str) -> np.ndarray:
+        if name not in self.header:
+            raise KeyError(f"{self.path} holds no tensor {name!r}")
+        e = self.header[name]
+        if e["dtype"] not in self.DTYPES:
+            raise ValueError(f"{name}: dtype {e['dtype']} is not supported")
+        dt, (lo, hi) = np.dtype(self.DTYPES[e["dtype"]]), e["data_offsets"]
+        count = int(np.prod(e["shape"], dtype=np.int64))
+        if hi - lo != count * dt.itemsize or lo < 0 or self.base + hi > self.data.size:
+            raise ValueError(f"{name}: data offsets {lo}..{hi} do not hold {e['shape']} of {e['dtype']}")
+        return np.frombuffer(self.data, dt, count, self.base + lo).reshape(e["shape"])
 
 
 class WeightFile:
