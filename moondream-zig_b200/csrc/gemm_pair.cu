@@ -92,11 +92,12 @@ __device__ __forceinline__ void pair_tile_coords(int tile, int tiles_m, int tile
 // PUSH = the column-split form: eight more warps per CTA copy every finished tile (this CTA's 128 rows of it) from
 // this GPU's C into the peers' C, as in the single-CTA kernel (its own instantiation, so that the plain kernel keeps
 // the register budget of 320 threads).
-template <bool B_MN_MAJOR, bool PUSH>
+// BF16 = bfloat16 operands and output with the glue of md_lin, as in the single-CTA kernel.
+template <bool B_MN_MAJOR, bool PUSH, bool BF16>
 __global__ void __launch_bounds__(PUSH ? NUM_THREADS_PUSH : NUM_THREADS, 1)
 gemm_pair_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant__ CUtensorMap tm_b,
                  const __grid_constant__ CUtensorMap tm_c, int M, int N, int K, int tiles_m, int num_tiles,
-                 md_epilogue ep, md_push push, md_devflags* flags, const __grid_constant__ md_peer_maps pm) {
+                 md_epilogue ep, md_push push, md_devflags* flags, const __grid_constant__ md_peer_maps pm, md_lin lin) {
     extern __shared__ uint8_t smem_raw[];
     const uint32_t raw = smem_u32(smem_raw);
     const uint32_t base = (raw + 1023u) & ~1023u;
@@ -191,7 +192,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant
         // ------------------------------------------------------------ MMA issuer (leader only)
         if (lane == 0 && rank == 0) {
             // M = 256 over the pair (128 rows per CTA), N = 256, f32 accumulators
-            const uint32_t idesc = (1u << 4) | ((B_MN_MAJOR ? 1u : 0u) << 16) | ((uint32_t)(BLOCK_N >> 3) << 17) |
+            const uint32_t idesc = (1u << 4) | idesc_format<BF16>() | ((B_MN_MAJOR ? 1u : 0u) << 16) | ((uint32_t)(BLOCK_N >> 3) << 17) |
                                    ((uint32_t)((2 * BLOCK_M) >> 4) << 24);
             constexpr uint32_t A_KSTEP = (UMMA_K * 2) >> 4, B_KSTEP = (B_MN_MAJOR ? UMMA_K * 128 : UMMA_K * 2) >> 4;
             const uint32_t a_hi = desc_hi(1024, 2), b_hi = desc_hi(1024, 2);
@@ -250,8 +251,23 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant
                 if (lane == 0) tma_store_wait_read<0>();
                 __syncwarp();
                 uint8_t* out_row = my_epi_ptr + lane * 128;
+                const bool glu = BF16 && lin.glu;
+                if (glu) {
+                    uint32_t g[32], u[32];
+                    tc_ld_32x32(t_row + (uint32_t)(c * 64), g);
+                    tc_ld_32x32(t_row + (uint32_t)(c * 64 + 32), u);
+                    tc_wait_ld();
+#pragma unroll
+                    for (int q = 0; q < 4; ++q) {
+                        uint32_t pk[4];
+                        glu_glue8(g + 8 * q, u + 8 * q, lin.glu, pk);
+                        const int chunk = q ^ ((lane >> 1) & 3);   // 64-byte swizzle
+                        *reinterpret_cast<uint4*>(my_epi_ptr + lane * 64 + chunk * 16) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
+                    }
+                }
 #pragma unroll
                 for (int h = 0; h < 2; ++h) {
+                    if (glu) break;
                     uint32_t r[32];
                     tc_ld_32x32(t_row + (uint32_t)(c * 64 + h * 32), r);
                     tc_wait_ld();
@@ -260,7 +276,8 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant
                     for (int q = 0; q < 4; ++q) {
                         const int cq = col0 + 8 * q;
                         uint32_t pk[4];
-                        epilogue_glue8(r + 8 * q, ep, row, cq, N, any_glue && row < M && cq < N, pk);
+                        if constexpr (BF16) lin_glue8(r + 8 * q, lin, cq, N, pk);
+                        else epilogue_glue8(r + 8 * q, ep, row, cq, N, any_glue && row < M && cq < N, pk);
                         const int chunk = (h * 4 + q) ^ (lane & 7);  // 128-byte swizzle, matches the store map
                         *reinterpret_cast<uint4*>(out_row + chunk * 16) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
                     }
@@ -274,7 +291,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant
                 fence_async_smem();
                 __syncwarp();
                 if (lane == 0) {
-                    tma_store_2d(&tm_c, my_epi, n0 + c * 64, mrow0);
+                    tma_store_2d(&tm_c, my_epi, glu ? (n0 + c * 64) / 2 : n0 + c * 64, mrow0);
                     if (PUSH && push.tma) {
                         // the same staged chunk into every peer's C, starting with a different peer in every CTA
                         for (int pi = 0; pi < push.n; ++pi) {
@@ -347,33 +364,19 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant
 
 }  // namespace
 
-int md_make_map_2d(md_ctx* ctx, CUtensorMap* map, const void* ptr, uint64_t inner, uint64_t outer, uint32_t box_inner,
-                   uint32_t box_outer, uint64_t ld);
+namespace {
 
-// C[M,N] = A . B (+ fused glue) on CTA pairs.  Same operand rules as the single-CTA kernel (K % 8 == 0, N % 8 == 0,
-// 16-byte aligned pointers, C with row stride ldc); the caller decides when the shape is large enough to pay for the
-// pairing.  push.n > 0: the column-split form (every tile also stored into the peers' C).
-int md_launch_gemm_pair(md_ctx* ctx, const __half* a, const __half* b, __half* c, size_t M, size_t N, size_t K, int b_layout,
-                        const md_epilogue& ep, size_t ldc, const md_push& push) {
-    const bool mn = (b_layout == 0), with_push = push.n > 0;
-    CUtensorMap tm_a, tm_b, tm_c;
-    MD_TRY(md_make_map_2d(ctx, &tm_a, a, K, M, BLOCK_K, BLOCK_M, 0));
-    if (mn) MD_TRY(md_make_map_2d(ctx, &tm_b, b, N, K, 64, BLOCK_K, 0));
-    else MD_TRY(md_make_map_2d(ctx, &tm_b, b, K, N, BLOCK_K, HALF_N, 0));
-    MD_TRY(md_make_map_2d(ctx, &tm_c, c, N, M, 64, 32, ldc));
+typedef void (*pair_fn)(CUtensorMap, CUtensorMap, CUtensorMap, int, int, int, int, int, md_epilogue, md_push, md_devflags*,
+                        md_peer_maps, md_lin);
+
+int launch_pairs(md_ctx* ctx, pair_fn kern, uint32_t cfg_bit, const CUtensorMap& tm_a, const CUtensorMap& tm_b,
+                 const CUtensorMap& tm_c, size_t M, size_t N, size_t K, const md_epilogue& ep, const md_push& push,
+                 const md_peer_maps& pm, const md_lin& lin) {
+    const bool with_push = push.n > 0;
     const int tiles_m = (int)((M + 2 * BLOCK_M - 1) / (2 * BLOCK_M)), tiles_n = (int)((N + BLOCK_N - 1) / BLOCK_N);
     const int num_tiles = tiles_m * tiles_n;
     const int max_pairs = ctx->sm_count / 2;
     const int pairs = num_tiles < max_pairs ? num_tiles : max_pairs;
-    md_peer_maps pm;
-    memset(&pm, 0, sizeof(pm));
-    if (with_push && push.tma)
-        for (int i = 0; i < push.n; ++i) MD_TRY(md_make_map_2d(ctx, &pm.m[i], push.base[i], N, M, 64, 32, ldc));
-    void (*kern)(CUtensorMap, CUtensorMap, CUtensorMap, int, int, int, int, int, md_epilogue, md_push, md_devflags*,
-                 md_peer_maps) =
-        with_push ? (mn ? gemm_pair_kernel<true, true> : gemm_pair_kernel<false, true>)
-                  : (mn ? gemm_pair_kernel<true, false> : gemm_pair_kernel<false, false>);
-    const uint32_t cfg_bit = 1u << ((mn ? 1 : 0) + (with_push ? 2 : 0));
     if (!(ctx->pair_configured & cfg_bit)) {
         MD_CUDA(ctx, cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES));
         ctx->pair_configured |= cfg_bit;
@@ -394,8 +397,46 @@ int md_launch_gemm_pair(md_ctx* ctx, const __half* a, const __half* b, __half* c
     cfg.numAttrs = ctx->pdl ? 2 : 1;
     ctx->last_tc_tile = 2256;   // md_get_option("last_tc_tile"): 2256 = a 256 x 256 tile on a CTA pair
     const int Mi = (int)M, Ni = (int)N, Ki = (int)K;
-    const cudaError_t e = cudaLaunchKernelEx(&cfg, kern, tm_a, tm_b, tm_c, Mi, Ni, Ki, tiles_m, num_tiles, ep, push, ctx->flags, pm);
+    const cudaError_t e = cudaLaunchKernelEx(&cfg, kern, tm_a, tm_b, tm_c, Mi, Ni, Ki, tiles_m, num_tiles, ep, push, ctx->flags, pm, lin);
     if (e != cudaSuccess) return md_fail(ctx, MD_ERR_CUDA, "launch of gemm_pair_kernel failed: %s", cudaGetErrorString(e));
     ctx->launches++;
     return MD_OK;
+}
+
+}  // namespace
+
+int md_make_map_2d(md_ctx* ctx, CUtensorMap* map, const void* ptr, uint64_t inner, uint64_t outer, uint32_t box_inner,
+                   uint32_t box_outer, uint64_t ld);
+
+// C[M,N] = A . B (+ fused glue) on CTA pairs.  Same operand rules as the single-CTA kernel (K % 8 == 0, N % 8 == 0,
+// 16-byte aligned pointers, C with row stride ldc); the caller decides when the shape is large enough to pay for the
+// pairing.  push.n > 0: the column-split form (every tile also stored into the peers' C).
+int md_launch_gemm_pair(md_ctx* ctx, const __half* a, const __half* b, __half* c, size_t M, size_t N, size_t K, int b_layout,
+                        const md_epilogue& ep, size_t ldc, const md_push& push) {
+    const bool mn = (b_layout == 0), with_push = push.n > 0;
+    CUtensorMap tm_a, tm_b, tm_c;
+    MD_TRY(md_make_map_2d(ctx, &tm_a, a, K, M, BLOCK_K, BLOCK_M, 0));
+    if (mn) MD_TRY(md_make_map_2d(ctx, &tm_b, b, N, K, 64, BLOCK_K, 0));
+    else MD_TRY(md_make_map_2d(ctx, &tm_b, b, K, N, BLOCK_K, HALF_N, 0));
+    MD_TRY(md_make_map_2d(ctx, &tm_c, c, N, M, 64, 32, ldc));
+    md_peer_maps pm;
+    memset(&pm, 0, sizeof(pm));
+    if (with_push && push.tma)
+        for (int i = 0; i < push.n; ++i) MD_TRY(md_make_map_2d(ctx, &pm.m[i], push.base[i], N, M, 64, 32, ldc));
+    void (*kern)(CUtensorMap, CUtensorMap, CUtensorMap, int, int, int, int, int, md_epilogue, md_push, md_devflags*,
+                 md_peer_maps, md_lin) =
+        with_push ? (mn ? gemm_pair_kernel<true, true, false> : gemm_pair_kernel<false, true, false>)
+                  : (mn ? gemm_pair_kernel<true, false, false> : gemm_pair_kernel<false, false, false>);
+    return launch_pairs(ctx, kern, 1u << ((mn ? 1 : 0) + (with_push ? 2 : 0)), tm_a, tm_b, tm_c, M, N, K, ep, push, pm, md_lin());
+}
+
+int md_launch_gemm_pair_lin(md_ctx* ctx, const void* a, const void* b, void* c, size_t M, size_t N, size_t K, const md_lin& lin) {
+    CUtensorMap tm_a, tm_b, tm_c;
+    MD_TRY(md_make_map_2d_bf16(ctx, &tm_a, a, K, M, BLOCK_K, BLOCK_M, false));
+    MD_TRY(md_make_map_2d_bf16(ctx, &tm_b, b, K, N, BLOCK_K, HALF_N, false));
+    if (lin.glu) MD_TRY(md_make_map_2d_bf16(ctx, &tm_c, c, N / 2, M, 32, 32, true));
+    else MD_TRY(md_make_map_2d_bf16(ctx, &tm_c, c, N, M, 64, 32, false));
+    md_peer_maps pm;
+    memset(&pm, 0, sizeof(pm));
+    return launch_pairs(ctx, gemm_pair_kernel<false, false, true>, 1u << 4, tm_a, tm_b, tm_c, M, N, K, md_epilogue(), md_push(), pm, lin);
 }

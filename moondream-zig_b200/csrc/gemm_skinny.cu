@@ -20,6 +20,7 @@
 // TMEM), warps 2..5 epilogue: tcgen05.ld of the transposed tile (TMEM lane = output column) into shared memory as
 // [row][128 columns], then 16-byte pieces of rows go to the workspace or, through the glue, to C.
 // Every mbarrier wait is bounded as in the general kernel.
+// BF16: bfloat16 operands and output with the glue of md_lin (a gated product combines columns c and c + 32 of a tile).
 #include "md_internal.cuh"
 #include "tc_common.cuh"
 
@@ -39,10 +40,10 @@ constexpr int SMEM_BYTES = 1024 + STAGES * STAGE_BYTES + 256;
 constexpr uint32_t TMEM_COLS = 64;
 constexpr int MAX_SPLITS = 8;          // portable cluster size
 
-template <bool W_MN_MAJOR>
+template <bool W_MN_MAJOR, bool BF16>
 __global__ void __launch_bounds__(THREADS, 2)
 gemm_skinny_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__ CUtensorMap tm_x, __half* C, int M,
-                   int N, int K, int kb_per_split, int splits, md_epilogue ep, md_devflags* flags) {
+                   int N, int K, int kb_per_split, int splits, md_epilogue ep, md_devflags* flags, md_lin lin) {
     extern __shared__ uint8_t smem_raw[];
     const uint32_t raw = smem_u32(smem_raw);
     const uint32_t base = (raw + 1023u) & ~1023u;
@@ -128,7 +129,7 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_consta
         if (lane == 0) {
             // D[128 weight rows, 64 activation rows] (f32), A = weights (K-major, or MN-major for the [K,N] layout),
             // B = activations (K-major)
-            const uint32_t idesc = (1u << 4) | ((W_MN_MAJOR ? 1u : 0u) << 15) | ((uint32_t)(XN >> 3) << 17) |
+            const uint32_t idesc = (1u << 4) | idesc_format<BF16>() | ((W_MN_MAJOR ? 1u : 0u) << 15) | ((uint32_t)(XN >> 3) << 17) |
                                    ((uint32_t)(TILE_N >> 4) << 24);
             constexpr uint32_t W_KSTEP = (W_MN_MAJOR ? UMMA_K * 128 : UMMA_K * 2) >> 4, X_KSTEP = (UMMA_K * 2) >> 4;
             const uint32_t hi = desc_hi(1024, 2);
@@ -190,6 +191,30 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_consta
         const int c4 = (et & 31) * 4, n = n0 + c4;
         const uint32_t tile_addr = base;   // shared-memory address of tile_f32 (same offset in every CTA of the cluster)
         auto finish = [&](int m, const float4& acc) {
+            if constexpr (BF16) {
+                __nv_bfloat16* Cb = reinterpret_cast<__nv_bfloat16*>(C);
+                float f[4] = {acc.x, acc.y, acc.z, acc.w};
+                if (lin.glu) {
+                    // gate columns sit in lanes whose bit 3 is clear, the up columns 32 further in the lanes 8 above
+                    float u[4];
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) u[j] = __shfl_down_sync(0xffffffffu, f[j], 8);
+                    if ((et & 8) || n >= N || m >= M) return;
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) f[j] = fast_act(lin.glu, f[j]) * u[j];
+                    md_store4<__nv_bfloat16>(Cb + (size_t)m * (N / 2) + (n & ~63) / 2 + (n & 31), f);
+                    return;
+                }
+                if (n >= N || m >= M) return;
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    if (lin.bias) f[j] += lin.bias[n + j];
+                    if (n + j < lin.silu_cols) f[j] = fast_silu(f[j]);
+                    else if (n + j >= lin.sigmoid_from) f[j] = fast_logistic(f[j]);
+                }
+                md_store4<__nv_bfloat16>(Cb + (size_t)m * N + n, f);
+                return;
+            }
             if (n >= N || m >= M) return;   // N % 8 == 0: a piece of four columns is inside or outside C
             const __half2 lo = __floats2half2_rn(md_epilogue_value(ep, acc.x, m, n, N), md_epilogue_value(ep, acc.y, m, n + 1, N));
             const __half2 hi = __floats2half2_rn(md_epilogue_value(ep, acc.z, m, n + 2, N), md_epilogue_value(ep, acc.w, m, n + 3, N));
@@ -255,15 +280,12 @@ bool md_gemm_skinny_supported(const void* a, const void* b, const void* c, size_
     return N <= (1u << 30) && K <= (1u << 30);
 }
 
-int md_launch_gemm_skinny(md_ctx* ctx, const __half* a, const __half* b, __half* c, size_t M, size_t N, size_t K,
-                          int b_layout, const md_epilogue& ep) {
-    if (!md_gemm_skinny_supported(a, b, c, M, N, K))
-        return md_fail(ctx, MD_ERR_UNSUPPORTED, "skinny GEMM needs 8 < M <= 64, K %% 8 == 0, N %% 8 == 0 and 16-byte aligned operands");
-    const bool mn = (b_layout == 0);
-    CUtensorMap tm_w, tm_x;
-    if (mn) MD_TRY(md_make_map_2d(ctx, &tm_w, b, N, K, 64, BLOCK_K, 0));
-    else MD_TRY(md_make_map_2d(ctx, &tm_w, b, K, N, BLOCK_K, TILE_N, 0));
-    MD_TRY(md_make_map_2d(ctx, &tm_x, a, K, M, BLOCK_K, XN, 0));
+namespace {
+
+typedef void (*skinny_fn)(CUtensorMap, CUtensorMap, __half*, int, int, int, int, int, md_epilogue, md_devflags*, md_lin);
+
+int launch_splits(md_ctx* ctx, skinny_fn kern, uint32_t cfg_bit, const CUtensorMap& tm_w, const CUtensorMap& tm_x, __half* c, size_t M,
+                  size_t N, size_t K, const md_epilogue& ep, const md_lin& lin) {
     const int tiles = (int)((N + TILE_N - 1) / TILE_N);
     const int num_kb = (int)((K + BLOCK_K - 1) / BLOCK_K);
     // splits of K = CTAs per cluster: about two CTAs per SM in one wave, a power of two up to the portable cluster
@@ -273,10 +295,8 @@ int md_launch_gemm_skinny(md_ctx* ctx, const __half* a, const __half* b, __half*
     int splits = 1;
     while (splits * 2 <= want && splits * 2 <= MAX_SPLITS) splits *= 2;
     const int kb_per_split = (num_kb + splits - 1) / splits;
-    const uint32_t cfg_bit = 1u << (mn ? 14 : 13);
     if (!(ctx->tc_configured & cfg_bit)) {
-        if (mn) MD_CUDA(ctx, cudaFuncSetAttribute(gemm_skinny_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES));
-        else MD_CUDA(ctx, cudaFuncSetAttribute(gemm_skinny_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES));
+        MD_CUDA(ctx, cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES));
         ctx->tc_configured |= cfg_bit;
     }
     ctx->last_tc_tile = 1000 + splits;   // md_get_option("last_tc_tile"): 1000 + S = the skinny kernel with S splits
@@ -302,9 +322,33 @@ int md_launch_gemm_skinny(md_ctx* ctx, const __half* a, const __half* b, __half*
     cfg.attrs = attr;
     cfg.numAttrs = na;
     const int Mi = (int)M, Ni = (int)N, Ki = (int)K;
-    const cudaError_t e = mn ? cudaLaunchKernelEx(&cfg, gemm_skinny_kernel<true>, tm_w, tm_x, c, Mi, Ni, Ki, kb_per_split, splits, ep, ctx->flags)
-                             : cudaLaunchKernelEx(&cfg, gemm_skinny_kernel<false>, tm_w, tm_x, c, Mi, Ni, Ki, kb_per_split, splits, ep, ctx->flags);
+    const cudaError_t e = cudaLaunchKernelEx(&cfg, kern, tm_w, tm_x, c, Mi, Ni, Ki, kb_per_split, splits, ep, ctx->flags, lin);
     if (e != cudaSuccess) return md_fail(ctx, MD_ERR_CUDA, "launch of gemm_skinny_kernel failed: %s", cudaGetErrorString(e));
     ctx->launches++;
     return MD_OK;
+}
+
+}  // namespace
+
+int md_launch_gemm_skinny(md_ctx* ctx, const __half* a, const __half* b, __half* c, size_t M, size_t N, size_t K,
+                          int b_layout, const md_epilogue& ep) {
+    if (!md_gemm_skinny_supported(a, b, c, M, N, K))
+        return md_fail(ctx, MD_ERR_UNSUPPORTED, "skinny GEMM needs 8 < M <= 64, K %% 8 == 0, N %% 8 == 0 and 16-byte aligned operands");
+    const bool mn = (b_layout == 0);
+    CUtensorMap tm_w, tm_x;
+    if (mn) MD_TRY(md_make_map_2d(ctx, &tm_w, b, N, K, 64, BLOCK_K, 0));
+    else MD_TRY(md_make_map_2d(ctx, &tm_w, b, K, N, BLOCK_K, TILE_N, 0));
+    MD_TRY(md_make_map_2d(ctx, &tm_x, a, K, M, BLOCK_K, XN, 0));
+    return launch_splits(ctx, mn ? gemm_skinny_kernel<true, false> : gemm_skinny_kernel<false, false>, 1u << (mn ? 14 : 13), tm_w, tm_x,
+                         c, M, N, K, ep, md_lin());
+}
+
+int md_launch_gemm_skinny_lin(md_ctx* ctx, const void* a, const void* b, void* c, size_t M, size_t N, size_t K, const md_lin& lin) {
+    if (!md_gemm_skinny_supported(a, b, c, M, N, K) || lin.tile_expert || lin.out_f32)
+        return md_fail(ctx, MD_ERR_UNSUPPORTED, "skinny GEMM needs 8 < M <= 64, K %% 8 == 0, N %% 8 == 0 and 16-byte aligned operands");
+    CUtensorMap tm_w, tm_x;
+    MD_TRY(md_make_map_2d_bf16(ctx, &tm_w, b, K, N, BLOCK_K, TILE_N, false));
+    MD_TRY(md_make_map_2d_bf16(ctx, &tm_x, a, K, M, BLOCK_K, XN, false));
+    return launch_splits(ctx, gemm_skinny_kernel<false, true>, 1u << 15, tm_w, tm_x, reinterpret_cast<__half*>(c), M, N, K,
+                         md_epilogue(), lin);
 }

@@ -27,6 +27,12 @@
 // Tails: TMA zero-fills out-of-bounds loads and clips out-of-bounds stores, so any M, N, K
 // with 16-byte-aligned row strides is accepted.
 //
+// bfloat16 form (BF16; md_lin in stack.cuh): the same structure with bfloat16 operands and output, an f32 bias, column
+// activations, or a gated product: B's rows are gate and up rows in blocks of 32, so a 64-column chunk of the
+// accumulators gives 32 finished columns (64-byte rows in the staging buffer, 64-byte swizzle).  With rows sorted by
+// expert (tile_expert) the row block picks the matrix: B is the stack of all experts' matrices as one tall one, and the
+// number of row blocks is read from device memory.
+//
 // Every mbarrier wait is bounded (about a second); a wait that gives up records an error
 // in the context's device flag word, raises a CTA-wide abort flag that makes all later
 // waits return at once, and the kernel still runs to its end, frees its TMEM and exits.
@@ -78,12 +84,12 @@ __device__ __forceinline__ void epi_sync() { asm volatile("bar.sync 1, %0;" ::"n
 // register budget of 320 threads)
 // SPLITK = the form that may split K over several CTAs per tile (its own instantiation: the others compile with one
 // range per tile and carry none of its code).
-template <int BLOCK_N, bool B_MN_MAJOR, int MT, bool PUSH, bool SPLITK>
+template <int BLOCK_N, bool B_MN_MAJOR, int MT, bool PUSH, bool SPLITK, bool BF16>
 __global__ void __launch_bounds__(PUSH ? NUM_THREADS_PUSH : NUM_THREADS, 1)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant__ CUtensorMap tm_b,
                const __grid_constant__ CUtensorMap tm_c, int M, int N, int K, int tiles_m, int num_tiles,
                md_epilogue ep, md_push push, md_devflags* flags, int splits_arg, float* part, unsigned* tickets,
-               const __grid_constant__ md_peer_maps pm) {
+               const __grid_constant__ md_peer_maps pm, md_lin lin) {
     const int splits = SPLITK ? splits_arg : 1;
     // splits > 1 (MT == 1, no peers): a work unit is one of `splits` ranges of k-blocks of a tile.  Every unit leaves
     // its f32 accumulators in `part` ([unit][column][row]); the unit that arrives last at the tile's ticket adds the
@@ -121,7 +127,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant__
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int num_kb = (K + BLOCK_K - 1) / BLOCK_K;
     const int tiles_n = num_tiles / tiles_m;
-    const int num_units = num_tiles * splits, kb_per = (num_kb + splits - 1) / splits;
+    int num_units = num_tiles * splits;
+    const int kb_per = (num_kb + splits - 1) / splits;
     volatile int* last_flag = reinterpret_cast<volatile int*>(bars_ptr + 16 * STAGES + 40 + 4 * EPI_WARPS);
 
     // programmatic dependent launch: the successor may start its own set-up now; this kernel sets up its
@@ -156,6 +163,11 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant__
     tc_fence_after();
     const uint32_t tmem_base = *tmem_slot;
     md_pdl_wait();
+    const bool grouped = BF16 && MT == 1 && lin.tile_expert != nullptr;
+    if (grouped) {
+        tiles_m = min(tiles_m, *lin.n_blocks);
+        num_units = tiles_m * tiles_n;
+    }
 
     if (warp == 0) {
         // ------------------------------------------------------------ TMA producer
@@ -166,7 +178,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant__
                 const int tile = unit / splits, kb0 = (unit - tile * splits) * kb_per, kb1 = min(num_kb, kb0 + kb_per);
                 int tm, tn;
                 tile_coords(tile, tiles_m, tiles_n, tm, tn);
-                const int m0 = tm * TILE_M, n0 = tn * BLOCK_N;
+                const int m0 = tm * TILE_M, n0 = tn * BLOCK_N + (grouped ? lin.tile_expert[tm] * N : 0);
                 for (int kb = kb0; kb < kb1; ++kb) {
                     mbar_wait(bar_empty + 8 * stage, phase ^ 1u, abort_flag, flags, 1);
                     const uint32_t full = bar_full + 8 * stage;
@@ -196,7 +208,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant__
     } else if (warp == 1) {
         // ------------------------------------------------------------ MMA issuer
         if (lane == 0) {
-            const uint32_t idesc = (1u << 4) | ((B_MN_MAJOR ? 1u : 0u) << 16) | ((uint32_t)(BLOCK_N >> 3) << 17) |
+            const uint32_t idesc = (1u << 4) | idesc_format<BF16>() | ((B_MN_MAJOR ? 1u : 0u) << 16) | ((uint32_t)(BLOCK_N >> 3) << 17) |
                                    ((uint32_t)(BLOCK_M >> 4) << 24);
             // descriptors as 32-bit halves: constant high words, low words advanced by adds (tc_common.cuh)
             // K-major operand: 16 k = 32 B further along the swizzled row; MN-major B: 16 k-rows = 2048 B
@@ -299,8 +311,23 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant__
                 if (lane == 0) tma_store_wait_read<0>();
                 __syncwarp();
                 uint8_t* out_row = my_epi_ptr + lane * 128;
+                const bool glu = BF16 && lin.glu;
+                if (glu) {
+                    uint32_t g[32], u[32];
+                    tc_ld_32x32(t_row + (uint32_t)(c * 64), g);
+                    tc_ld_32x32(t_row + (uint32_t)(c * 64 + 32), u);
+                    tc_wait_ld();
+#pragma unroll
+                    for (int q = 0; q < 4; ++q) {
+                        uint32_t pk[4];
+                        glu_glue8(g + 8 * q, u + 8 * q, lin.glu, pk);
+                        const int chunk = q ^ ((lane >> 1) & 3);   // 64-byte swizzle: 16-byte piece ^ address bits 7-8
+                        *reinterpret_cast<uint4*>(my_epi_ptr + lane * 64 + chunk * 16) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
+                    }
+                }
 #pragma unroll
                 for (int h = 0; h < 2; ++h) {
+                    if (glu) break;
                     uint32_t r[32];
                     if (from_part) {
                         // the k ranges added up in their order, whichever unit got here last; a range's 32 loads are
@@ -330,7 +357,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant__
                     for (int q = 0; q < 4; ++q) {
                         const int cq = col0 + 8 * q;
                         uint32_t pk[4];
-                        epilogue_glue8(r + 8 * q, ep, row, cq, N, any_glue && row < M && cq < N, pk);
+                        if constexpr (BF16) lin_glue8(r + 8 * q, lin, cq, N, pk);
+                        else epilogue_glue8(r + 8 * q, ep, row, cq, N, any_glue && row < M && cq < N, pk);
                         const int chunk = (h * 4 + q) ^ (lane & 7);  // 128-byte swizzle, matches the store map
                         *reinterpret_cast<uint4*>(out_row + chunk * 16) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
                     }
@@ -344,7 +372,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant__
                 fence_async_smem();
                 __syncwarp();
                 if (lane == 0) {
-                    tma_store_2d(&tm_c, my_epi, n0 + c * 64, mrow0);
+                    tma_store_2d(&tm_c, my_epi, glu ? (n0 + c * 64) / 2 : n0 + c * 64, mrow0);
                     if (PUSH && push.tma) {
                         // the same staged chunk into every peer's C, starting with a different peer in every CTA;
                         // the staging buffer is reused once all of these stores have read it
@@ -444,15 +472,16 @@ int resolve_encode_tiled(md_ctx* ctx) {
 }
 
 int make_map_2d(md_ctx* ctx, CUtensorMap* map, const void* ptr, uint64_t inner, uint64_t outer, uint32_t box_inner,
-                uint32_t box_outer, uint64_t ld = 0) {
+                uint32_t box_outer, uint64_t ld = 0, bool bf16 = false, bool swizzle_64 = false) {
     MD_TRY(resolve_encode_tiled(ctx));
     const cuuint64_t dims[2] = {inner, outer};
     const cuuint64_t strides[1] = {(ld ? ld : inner) * 2};
     const cuuint32_t box[2] = {box_inner, box_outer};
     const cuuint32_t elem[2] = {1, 1};
     CUresult r = reinterpret_cast<encode_tiled_fn>(ctx->encode_tiled)(
-        map, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 2, const_cast<void*>(ptr), dims, strides, box, elem,
-        CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+        map, bf16 ? CU_TENSOR_MAP_DATA_TYPE_BFLOAT16 : CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 2, const_cast<void*>(ptr), dims,
+        strides, box, elem, CU_TENSOR_MAP_INTERLEAVE_NONE,
+        swizzle_64 ? CU_TENSOR_MAP_SWIZZLE_64B : CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
         CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
     if (r != CUDA_SUCCESS) return md_fail(ctx, MD_ERR_CUDA, "cuTensorMapEncodeTiled failed with CUresult %d", (int)r);
     return MD_OK;
@@ -487,8 +516,8 @@ int launch_as(md_ctx* ctx, const __half* a, const __half* b, __half* c, size_t M
     const int grid = units < ctx->sm_count ? units : ctx->sm_count;
     // the split-K instantiation exists for single 128-row tiles of 256 columns without peers only
     constexpr bool CAN_SPLIT = MT == 1 && !PUSH && BLOCK_N == 256;
-    auto kern = (CAN_SPLIT && splits > 1) ? gemm_tc_kernel<BLOCK_N, B_MN_MAJOR, MT, PUSH, CAN_SPLIT>
-                                          : gemm_tc_kernel<BLOCK_N, B_MN_MAJOR, MT, PUSH, false>;
+    auto kern = (CAN_SPLIT && splits > 1) ? gemm_tc_kernel<BLOCK_N, B_MN_MAJOR, MT, PUSH, CAN_SPLIT, false>
+                                          : gemm_tc_kernel<BLOCK_N, B_MN_MAJOR, MT, PUSH, false, false>;
     constexpr int smem = smem_bytes(BLOCK_N, MT);
     const uint32_t cfg_bit = (CAN_SPLIT && splits > 1)
                                  ? 1u << (B_MN_MAJOR ? 7 : 6)
@@ -502,7 +531,32 @@ int launch_as(md_ctx* ctx, const __half* a, const __half* b, __half* c, size_t M
     ctx->last_tc_tile = (MT == 2 ? 512 : BLOCK_N) + (splits > 1 ? 10000 * splits : 0);   // 30256 = 128 x 256 tiles, K in 3
     return md_launch_ex(ctx, kern, dim3((unsigned)grid), dim3(PUSH ? NUM_THREADS_PUSH : NUM_THREADS), smem,
                         "gemm_tc_kernel", tm_a, tm_b, tm_c, (int)M, (int)N, (int)K, tiles_m, num_tiles, ep, push, ctx->flags,
-                        splits, part, tickets, pm);
+                        splits, part, tickets, pm, md_lin());
+}
+
+// The bfloat16 form: C[M, N] (N / 2 columns for a gated product) = md_lin of A[M, K] and B[N, K].
+template <int BLOCK_N, int MT>
+int launch_lin(md_ctx* ctx, const void* a, const void* b, void* c, size_t M, size_t N, size_t K, const md_lin& lin) {
+    CUtensorMap tm_a, tm_b, tm_c;
+    const size_t b_rows = lin.tile_expert ? N * (size_t)lin.n_experts : N;
+    MD_TRY(make_map_2d(ctx, &tm_a, a, K, M, BLOCK_K, BLOCK_M, 0, true));
+    MD_TRY(make_map_2d(ctx, &tm_b, b, K, b_rows, BLOCK_K, BLOCK_N, 0, true));
+    if (lin.glu) MD_TRY(make_map_2d(ctx, &tm_c, c, N / 2, M, 32, 32, 0, true, true));
+    else MD_TRY(make_map_2d(ctx, &tm_c, c, N, M, 64, 32, 0, true));
+    const int tiles_m = (int)((M + MT * BLOCK_M - 1) / (MT * BLOCK_M)), tiles_n = (int)((N + BLOCK_N - 1) / BLOCK_N);
+    const int num_tiles = tiles_m * tiles_n, grid = num_tiles < ctx->sm_count ? num_tiles : ctx->sm_count;
+    auto kern = gemm_tc_kernel<BLOCK_N, false, MT, false, false, true>;
+    constexpr int smem = smem_bytes(BLOCK_N, MT);
+    const uint32_t bit = 1u << (MT == 2 ? 3 : BLOCK_N == 256 ? 0 : BLOCK_N == 128 ? 1 : 2);
+    if (!(ctx->lin_configured & bit)) {
+        MD_CUDA(ctx, cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+        ctx->lin_configured |= bit;
+    }
+    md_peer_maps pm;
+    memset(&pm, 0, sizeof(pm));
+    ctx->last_tc_tile = MT == 2 ? 512 : BLOCK_N;
+    return md_launch_ex(ctx, kern, dim3((unsigned)grid), dim3(NUM_THREADS), smem, "gemm_tc_kernel", tm_a, tm_b, tm_c, (int)M, (int)N,
+                        (int)K, tiles_m, num_tiles, md_epilogue(), md_push(), ctx->flags, 1, (float*)nullptr, (unsigned*)nullptr, pm, lin);
 }
 
 template <int BLOCK_N, bool B_MN_MAJOR, int MT = 1>
@@ -528,6 +582,35 @@ int md_launch_gemm_tc(md_ctx* ctx, const __half* a, const __half* b, __half* c, 
                       int b_layout, const md_epilogue& ep) {
     md_push none;
     return md_launch_gemm_tc_ex(ctx, a, b, c, M, N, K, b_layout, ep, N, none);
+}
+
+int md_launch_gemm_tc_lin(md_ctx* ctx, const void* a, const void* b, void* c, size_t M, size_t N, size_t K, const md_lin& lin) {
+    if (!md_gemm_tc_supported(a, b, c, M, N, K, 1) || lin.out_f32)
+        return md_fail(ctx, MD_ERR_UNSUPPORTED, "tcgen05 GEMM needs K %% 8 == 0, N %% 8 == 0, 16-byte aligned operands and a 16-bit output");
+    int bn = 64, mt = 1;
+    if (lin.tile_expert) {
+        // the number of row blocks is only known on the device: enough of them to fill the machine with wide tiles, or narrow ones
+        const size_t blocks = (M + BLOCK_M - 1) / BLOCK_M;
+        bn = blocks * ((N + 255) / 256) >= 2 * (size_t)ctx->sm_count ? 256 : blocks * ((N + 127) / 128) >= (size_t)ctx->sm_count ? 128 : 64;
+    } else {
+        // the same cost as for f16 operands (see md_launch_gemm_tc_ex)
+        const int cand_n[4] = {256, 256, 128, 64}, cand_mt[4] = {2, 1, 1, 1};
+        double best = -1.0;
+        for (int i = 0; i < 4; ++i) {
+            const size_t rows = (size_t)cand_mt[i] * BLOCK_M;
+            const size_t t = ((M + rows - 1) / rows) * ((N + cand_n[i] - 1) / cand_n[i]);
+            const size_t waves = (t + ctx->sm_count - 1) / ctx->sm_count;
+            const double kblocks = (double)((K + BLOCK_K - 1) / BLOCK_K);
+            const double cost = (double)waves * ((double)(rows + cand_n[i]) * kblocks * (cand_mt[i] == 2 ? 1.3 : 1.0) +
+                                                 (cand_mt[i] == 2 ? 7000.0 : 0.0));
+            if (best < 0.0 || cost < best) { best = cost; bn = cand_n[i]; mt = cand_mt[i]; }
+        }
+        if (bn == 256 && mt == 1 && M > 256 && ctx->tc_pair != 0) return md_launch_gemm_pair_lin(ctx, a, b, c, M, N, K, lin);
+    }
+    if (mt == 2) return launch_lin<256, 2>(ctx, a, b, c, M, N, K, lin);
+    if (bn == 256) return launch_lin<256, 1>(ctx, a, b, c, M, N, K, lin);
+    if (bn == 128) return launch_lin<128, 1>(ctx, a, b, c, M, N, K, lin);
+    return launch_lin<64, 1>(ctx, a, b, c, M, N, K, lin);
 }
 
 int md_launch_gemm_tc_ex(md_ctx* ctx, const __half* a, const __half* b, __half* c, size_t M, size_t N, size_t K,
@@ -638,6 +721,10 @@ int md_launch_gemm_tc_ex(md_ctx* ctx, const __half* a, const __half* b, __half* 
 int md_make_map_2d(md_ctx* ctx, CUtensorMap* map, const void* ptr, uint64_t inner, uint64_t outer, uint32_t box_inner,
                    uint32_t box_outer, uint64_t ld) {
     return make_map_2d(ctx, map, ptr, inner, outer, box_inner, box_outer, ld);
+}
+int md_make_map_2d_bf16(md_ctx* ctx, CUtensorMap* map, const void* ptr, uint64_t inner, uint64_t outer, uint32_t box_inner,
+                        uint32_t box_outer, bool swizzle_64) {
+    return make_map_2d(ctx, map, ptr, inner, outer, box_inner, box_outer, 0, true, swizzle_64);
 }
 
 // 4-D f16 tensor map (dim 0 contiguous), 128- or 32-byte swizzle, zero fill outside the extents; the box is

@@ -25,7 +25,10 @@
 // K / S of its 16 rows, leaves its 16 x 8 partial sums in shared memory, and after one
 // cluster barrier the first CTA of the cluster adds the S partials through distributed
 // shared memory (fixed order), applies the glue and stores.  No global scratch.
-#include "md_internal.cuh"
+//
+// gemv_lin_kernel is the same mapping for bfloat16 weights with the glue of md_lin: f32 bias, column activations, f32 or
+// bfloat16 results, or a gated product, where a CTA's 16 rows are 8 gate rows and the 8 up rows beside them.
+#include "stack.cuh"
 
 namespace {
 
@@ -190,6 +193,123 @@ gemv_nt_mma_kernel(const __half* A, const __half* __restrict__ Bt, __half* C, in
     asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
 }
 
+__device__ __forceinline__ void mma_16816_bf16(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3,
+                                               uint32_t b0, uint32_t b1) {
+    asm volatile(
+        "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+        : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+        : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+
+template <int WARPS, int UNROLL>
+__global__ void __launch_bounds__(WARPS * 32)
+gemv_lin_kernel(const __half* A, const __half* __restrict__ Bt, __nv_bfloat16* C, int M, int N, int K, md_lin ep) {
+    __shared__ float partial[WARPS][ROWS_PER_CTA][8];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int g = lane >> 2, t = lane & 3;
+    int r_lo, r_hi;
+    if (ep.glu) {   // output j: gate row (j / 32) * 64 + j % 32, up row 32 further
+        const int j = blockIdx.x * 8 + g;
+        r_lo = (j / MD_GLU_BLOCK) * (2 * MD_GLU_BLOCK) + j % MD_GLU_BLOCK;
+        r_hi = r_lo + MD_GLU_BLOCK;
+    } else {
+        r_lo = min((int)blockIdx.x * ROWS_PER_CTA + g, N - 1);
+        r_hi = min((int)blockIdx.x * ROWS_PER_CTA + g + 8, N - 1);
+    }
+    const __half* w_lo = Bt + (size_t)r_lo * K + t * 8;
+    const __half* w_hi = Bt + (size_t)r_hi * K + t * 8;
+    const bool has_x = g < M;
+    const __half* x = A + (size_t)(has_x ? g : 0) * K + t * 8;
+    const int chunks = K / 32;
+    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+    md_pdl_launch_dependents();
+    bool waited = false;
+    int ch = warp;
+    for (; ch + (UNROLL - 1) * WARPS < chunks; ch += UNROLL * WARPS) {
+        uint4 lo[UNROLL], hi[UNROLL], xv[UNROLL];
+#pragma unroll
+        for (int u = 0; u < UNROLL; ++u) {
+            const int k = (ch + u * WARPS) * 32;
+            lo[u] = ldg_stream(w_lo + k);
+            hi[u] = ldg_stream(w_hi + k);
+        }
+        if (!waited) {
+            md_pdl_wait();
+            waited = true;
+        }
+#pragma unroll
+        for (int u = 0; u < UNROLL; ++u) xv[u] = has_x ? ld_act(x + (ch + u * WARPS) * 32) : make_uint4(0, 0, 0, 0);
+#pragma unroll
+        for (int u = 0; u < UNROLL; ++u) {
+            mma_16816_bf16(acc, lo[u].x, hi[u].x, lo[u].y, hi[u].y, xv[u].x, xv[u].y);
+            mma_16816_bf16(acc, lo[u].z, hi[u].z, lo[u].w, hi[u].w, xv[u].z, xv[u].w);
+        }
+    }
+    // what is left of K: up to UNROLL - 1 chunks per warp, requested together
+    {
+        uint4 lo[UNROLL], hi[UNROLL], xv[UNROLL];
+#pragma unroll
+        for (int u = 0; u < UNROLL - 1; ++u) {
+            const int c = ch + u * WARPS;
+            const bool live = c < chunks;
+            lo[u] = live ? ldg_stream(w_lo + c * 32) : make_uint4(0, 0, 0, 0);
+            hi[u] = live ? ldg_stream(w_hi + c * 32) : make_uint4(0, 0, 0, 0);
+        }
+        if (!waited) md_pdl_wait();
+#pragma unroll
+        for (int u = 0; u < UNROLL - 1; ++u) {
+            const int c = ch + u * WARPS;
+            xv[u] = has_x && c < chunks ? ld_act(x + c * 32) : make_uint4(0, 0, 0, 0);
+        }
+#pragma unroll
+        for (int u = 0; u < UNROLL - 1; ++u) {
+            mma_16816_bf16(acc, lo[u].x, hi[u].x, lo[u].y, hi[u].y, xv[u].x, xv[u].y);
+            mma_16816_bf16(acc, lo[u].z, hi[u].z, lo[u].w, hi[u].w, xv[u].z, xv[u].w);
+        }
+    }
+    if (warp == 0 && chunks * 32 < K) {   // K % 32 != 0, still a multiple of 8
+        const int k = chunks * 32 + t * 8;
+        uint4 lo = make_uint4(0, 0, 0, 0), hi = lo, xv = lo;
+        if (k < K) {
+            lo = ldg_stream(Bt + (size_t)r_lo * K + k);
+            hi = ldg_stream(Bt + (size_t)r_hi * K + k);
+            if (has_x) xv = ld_act(A + (size_t)g * K + k);
+        }
+        mma_16816_bf16(acc, lo.x, hi.x, lo.y, hi.y, xv.x, xv.y);
+        mma_16816_bf16(acc, lo.z, hi.z, lo.w, hi.w, xv.z, xv.w);
+    }
+    partial[warp][g][2 * t] = acc[0];
+    partial[warp][g][2 * t + 1] = acc[1];
+    partial[warp][g + 8][2 * t] = acc[2];
+    partial[warp][g + 8][2 * t + 1] = acc[3];
+    __syncthreads();
+    if (ep.glu) {
+        for (int o = threadIdx.x; o < 64; o += WARPS * 32) {
+            const int m = o >> 3, r = o & 7;
+            if (m >= M) continue;
+            float a = 0.f, b = 0.f;
+#pragma unroll
+            for (int w = 0; w < WARPS; ++w) {
+                a += partial[w][r][m];
+                b += partial[w][r + 8][m];
+            }
+            C[(size_t)m * (N / 2) + blockIdx.x * 8 + r] = __float2bfloat16_rn(md_act(ep.glu, a) * b);
+        }
+        return;
+    }
+    for (int o = threadIdx.x; o < ROWS_PER_CTA * 8; o += WARPS * 32) {
+        const int m = o >> 4, r = o & 15, n = blockIdx.x * ROWS_PER_CTA + r;
+        if (m >= M || n >= N) continue;
+        float s = 0.f;
+#pragma unroll
+        for (int w = 0; w < WARPS; ++w) s += partial[w][r][m];
+        if (ep.bias) s += ep.bias[n];
+        s = md_lin_col(s, n, ep.silu_cols, ep.sigmoid_from);
+        if (ep.out_f32) ep.out_f32[(size_t)m * N + n] = s;
+        else C[(size_t)m * N + n] = __float2bfloat16_rn(s);
+    }
+}
+
 }  // namespace
 
 int md_launch_gemv_nt(md_ctx* ctx, const __half* a, const __half* bt, __half* c, size_t M, size_t N, size_t K,
@@ -260,4 +380,18 @@ int md_launch_gemv_nt(md_ctx* ctx, const __half* a, const __half* bt, __half* c,
     if (le != cudaSuccess) return md_fail(ctx, MD_ERR_CUDA, "launch of gemv_nt_mma_kernel failed: %s", cudaGetErrorString(le));
     MD_LAUNCH_CHECK(ctx, "gemv_nt_mma_kernel");
     return MD_OK;
+}
+
+int md_launch_gemv_lin(md_ctx* ctx, const void* a, const void* b, void* c, size_t M, size_t N, size_t K, const md_lin& lin) {
+    if (M == 0 || M > 8 || (K % 8) != 0 || K == 0 || N == 0 || lin.tile_expert ||
+        ((reinterpret_cast<uintptr_t>(a) | reinterpret_cast<uintptr_t>(b)) & 15))
+        return md_fail(ctx, MD_ERR_UNSUPPORTED, "gemv_lin needs 1 <= M <= 8, K %% 8 == 0 and 16-byte aligned operands (M=%zu K=%zu)", M, K);
+    const unsigned grid = (unsigned)((N + ROWS_PER_CTA - 1) / ROWS_PER_CTA);
+    const __half *A = reinterpret_cast<const __half*>(a), *B = reinterpret_cast<const __half*>(b);
+    __nv_bfloat16* C = reinterpret_cast<__nv_bfloat16*>(c);
+    // as for f16: many rows want small CTAs; few rows or long ones want the whole matrix in flight at once
+    if (N >= 16384) return md_launch_ex(ctx, gemv_lin_kernel<4, 4>, dim3(grid), dim3(128), 0, "gemv_lin_kernel", A, B, C, (int)M, (int)N, (int)K, lin);
+    if (K >= 4096 || N <= 2048)
+        return md_launch_ex(ctx, gemv_lin_kernel<16, 4>, dim3(grid), dim3(512), 0, "gemv_lin_kernel", A, B, C, (int)M, (int)N, (int)K, lin);
+    return md_launch_ex(ctx, gemv_lin_kernel<8, 8>, dim3(grid), dim3(256), 0, "gemv_lin_kernel", A, B, C, (int)M, (int)N, (int)K, lin);
 }

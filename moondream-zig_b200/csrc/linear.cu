@@ -1,4 +1,5 @@
-// Linear layers of the layer-stack decoders: md_linear picks the kernel, and gemm_plain_kernel is the one that takes any
+// Linear layers of the layer-stack decoders: md_linear picks the kernel (the bfloat16 forms of the GEMV, the skinny GEMM
+// and the tcgen05 GEMMs, by the rules of the f16 dispatch), and gemm_plain_kernel is the one that takes any
 // shape and either element type (the true 32-bit products, and bfloat16 shapes whose rows TMA or 16-byte loads cannot
 // address): 64 x 64 tiles, f32 FMA.
 #include "stack.cuh"
@@ -77,5 +78,22 @@ int md_linear(md_ctx* ctx, int dtype, const void* a, const void* w, void* c, siz
     if (M == 0 || N == 0) return MD_OK;
     if (ep.glu && (N % (2 * MD_GLU_BLOCK)) != 0) return md_fail(ctx, MD_ERR_INVALID_ARG, "md_linear: gate / up rows must come in blocks");
     if (dtype == MD_DTYPE_F32) return launch_plain<float>(ctx, a, w, c, M, N, K, ep);
+    const uintptr_t align = reinterpret_cast<uintptr_t>(a) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(c);
+    if (ctx->gemm_mode != 1 && (K % 8) == 0 && (align & 15) == 0) {
+        if (!ep.tile_expert && (M <= 8 || ep.out_f32)) {
+            // f32 results of many rows (the head over the wanted rows of a prompt): eight rows at a time
+            for (size_t m = 0; m < M; m += 8) {
+                md_lin part = ep;
+                if (ep.out_f32) part.out_f32 = ep.out_f32 + m * N;
+                MD_TRY(md_launch_gemv_lin(ctx, reinterpret_cast<const __nv_bfloat16*>(a) + m * K, w, c, M - m < 8 ? M - m : 8, N, K, part));
+            }
+            return MD_OK;
+        }
+        if ((N % 8) == 0 && !ep.out_f32) {
+            if (!ep.tile_expert && ctx->skinny && md_gemm_skinny_supported(a, w, c, M, N, K))
+                return md_launch_gemm_skinny_lin(ctx, a, w, c, M, N, K, ep);
+            return md_launch_gemm_tc_lin(ctx, a, w, c, M, N, K, ep);
+        }
+    }
     return launch_plain<__nv_bfloat16>(ctx, a, w, c, M, N, K, ep);
 }

@@ -71,6 +71,7 @@ struct md_ctx {
     unsigned int* counters = nullptr;
     // cuTensorMapEncodeTiled resolved through the runtime (no link against libcuda)
     void* encode_tiled = nullptr;
+    uint32_t lin_configured = 0;   // bfloat16 GEMM kernels whose dynamic shared memory limit has been raised
     uint32_t pair_configured = 0;  // the same for the instantiations of gemm_pair_kernel
     uint32_t tc_configured = 0;  // tcgen05 kernels whose dynamic shared memory limit has been raised
     int skinny = 1;          // md_set_option("skinny"): 8 < M <= 64 takes the swapped-operand split-K kernel

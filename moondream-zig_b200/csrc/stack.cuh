@@ -29,6 +29,13 @@ struct md_lin {
     int n_experts = 0;
 };
 constexpr int MD_GLU_BLOCK = 32;
+// bfloat16 kernels behind md_linear (weights [N, K])
+int md_launch_gemm_tc_lin(md_ctx* ctx, const void* a, const void* b, void* c, size_t M, size_t N, size_t K, const md_lin& lin);
+int md_launch_gemm_pair_lin(md_ctx* ctx, const void* a, const void* b, void* c, size_t M, size_t N, size_t K, const md_lin& lin);
+int md_launch_gemm_skinny_lin(md_ctx* ctx, const void* a, const void* b, void* c, size_t M, size_t N, size_t K, const md_lin& lin);
+int md_launch_gemv_lin(md_ctx* ctx, const void* a, const void* b, void* c, size_t M, size_t N, size_t K, const md_lin& lin);
+int md_make_map_2d_bf16(md_ctx* ctx, CUtensorMap* map, const void* ptr, uint64_t inner, uint64_t outer, uint32_t box_inner,
+                        uint32_t box_outer, bool swizzle_64);
 int md_linear(md_ctx* ctx, int dtype, const void* a, const void* w, void* c, size_t M, size_t N, size_t K, const md_lin& ep);
 
 // ---- residual + norms + causal convolution ---------------------------------------------------------------

@@ -2,7 +2,7 @@
 // TMA tile loads / stores, tcgen05 MMA / commit / TMEM loads, shared-memory matrix descriptors.
 #pragma once
 
-#include "md_internal.cuh"
+#include "stack.cuh"
 
 namespace tc {
 
@@ -226,6 +226,51 @@ __device__ __forceinline__ void epilogue_glue8(const uint32_t* acc_bits, const m
     }
 #pragma unroll
     for (int j = 0; j < 4; ++j) pk[j] = *reinterpret_cast<uint32_t*>(&h[j]);
+}
+
+// Instruction-descriptor bits that name the operands' format (kind::f16): both f16, or both bf16.
+template <bool BF16> __host__ __device__ constexpr uint32_t idesc_format() { return BF16 ? (1u << 7) | (1u << 10) : 0u; }
+
+// exp-based forms of the activations with the hardware exp2 and a fast divide (relative error about 1e-6, far below the
+// bfloat16 rounding that follows)
+__device__ __forceinline__ float fast_logistic(float z) { return __fdividef(1.f, 1.f + __expf(-z)); }
+__device__ __forceinline__ float fast_silu(float z) { return z * fast_logistic(z); }
+__device__ __forceinline__ float fast_gelu_tanh(float z) {   // 0.5 z (1 + tanh u) = z * logistic(2 u)
+    return z * fast_logistic(1.5957691216057308f * (z + 0.044715f * z * z * z));
+}
+__device__ __forceinline__ float fast_act(int act, float z) { return act == MD_ACT_SILU ? fast_silu(z) : fast_gelu_tanh(z); }
+
+// md_lin on 8 consecutive output columns of one row: f32 accumulators in, four packed bfloat16 pairs out.  N % 8 == 0.
+__device__ __forceinline__ void lin_glue8(const uint32_t* acc_bits, const md_lin& ep, int cq, int N, uint32_t (&pk)[4]) {
+    float v[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[j] = __uint_as_float(acc_bits[j]);
+    if (cq < N) {
+        if (ep.bias) {
+            const float4 a = *reinterpret_cast<const float4*>(ep.bias + cq), b = *reinterpret_cast<const float4*>(ep.bias + cq + 4);
+            v[0] += a.x; v[1] += a.y; v[2] += a.z; v[3] += a.w;
+            v[4] += b.x; v[5] += b.y; v[6] += b.z; v[7] += b.w;
+        }
+        if (cq < ep.silu_cols || cq + 8 > ep.sigmoid_from) {
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+                const bool si = cq + j < ep.silu_cols, sg = cq + j >= ep.sigmoid_from;
+                if (si || sg) {
+                    const float g = fast_logistic(v[j]);
+                    v[j] = si ? v[j] * g : g;
+                }
+            }
+        }
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j) pk[j] = md_pack_bf16(v[2 * j], v[2 * j + 1]);
+}
+// 8 columns of a gated product: gate and up accumulators in
+__device__ __forceinline__ void glu_glue8(const uint32_t* gate, const uint32_t* up, int act, uint32_t (&pk)[4]) {
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+        pk[j] = md_pack_bf16(fast_act(act, __uint_as_float(gate[2 * j])) * __uint_as_float(up[2 * j]),
+                             fast_act(act, __uint_as_float(gate[2 * j + 1])) * __uint_as_float(up[2 * j + 1]));
 }
 
 // Shared-memory matrix descriptor (version 1, sm_100) as built by desc_lo / desc_hi:

@@ -155,12 +155,12 @@ class ColSplitGemm:
 # ----------------------------------------------------------------------------- independent requests
 
 class Request:
-    """One request of the box-scale workload: the crops of an image and the prompt's token ids."""
+    """One request: the crops of an image (None for a text-only prompt) and the prompt's token ids."""
 
-    def __init__(self, crops_u8: np.ndarray, prompt_ids):
-        self.crops = np.ascontiguousarray(crops_u8, np.uint8)
+    def __init__(self, crops_u8: np.ndarray | None, prompt_ids):
+        self.crops = None if crops_u8 is None else np.ascontiguousarray(crops_u8, np.uint8)
         self.ids = np.ascontiguousarray(prompt_ids, np.uint32)
-        assert self.crops.ndim == 4 and self.ids.size >= 1
+        assert (self.crops is None or self.crops.ndim == 4) and self.ids.size >= 1
 
 
 def serve_requests(ctx, vision, text, requests: list, world: int, rank: int, n_steps: int, max_streams: int = 8,
@@ -171,6 +171,7 @@ def serve_requests(ctx, vision, text, requests: list, world: int, rank: int, n_s
     the device: vision encode -> [embed(tok0), 729 image rows, embed(tok1..)] (moondream.zig:286-303) -> prefill ->
     first token -> n_steps greedy decode steps.  Up to `max_streams` (<= 8) requests decode together as M <= 8 GEMVs
     (md_text_generate_batch).  tokens = [first token, then the n_steps generated tokens].
+    With vision None every request is a token prompt: one md_text_step, then the same batched decoding.
     forced: {index: uint32 [n_steps]} feeds those tokens instead of the model's own (teacher forcing, for parity
     checks).  state: a dict reused across calls to keep the KV caches and buffers (8 x 384 MiB at full size)."""
     assert 1 <= max_streams <= 8
@@ -179,12 +180,19 @@ def serve_requests(ctx, vision, text, requests: list, world: int, rank: int, n_s
     reqs = state.setdefault("reqs", [])
     while len(reqs) < min(max_streams, len(mine)):
         reqs.append(text.request())
-    dim, tokens = text.dim, vision.tokens
-    assert vision.proj_out == dim
+    dim, tokens = text.dim, vision.tokens if vision is not None else 0
+    assert vision is None or vision.proj_out == dim
     embeds = state.setdefault("embeds", {})          # slot -> (DevBuf [rows, dim], rows)
     out: dict = {}
     for g0 in range(0, len(mine), max_streams):
         group = mine[g0:g0 + max_streams]
+        if vision is None:
+            firsts = []
+            for slot, idx in enumerate(group):
+                reqs[slot].reset()
+                firsts.append(text.step(reqs[slot], requests[idx].ids, want_token=True)[1])
+            _decode_group(text, reqs, group, firsts, n_steps, forced, out)
+            continue
         bases = []
         for slot, idx in enumerate(group):
             rows = requests[idx].ids.size + tokens
@@ -210,13 +218,18 @@ def serve_requests(ctx, vision, text, requests: list, world: int, rank: int, n_s
             reqs[slot].reset()
             _, _, tok = text.forward(reqs[slot], base, want_hidden=False, want_logits=False, rows=rows)
             firsts.append(tok)
-        f = None
-        if forced is not None:
-            f = np.stack([np.ascontiguousarray(forced[idx], np.uint32) for idx in group])
-        toks = text.generate_batch(reqs[:len(group)], firsts, n_steps, forced=f)
-        for slot, idx in enumerate(group):
-            out[idx] = np.concatenate([np.array([firsts[slot]], np.uint32), toks[slot]])
+        _decode_group(text, reqs, group, firsts, n_steps, forced, out)
     return out
+
+
+def _decode_group(text, reqs: list, group: list, firsts: list, n_steps: int, forced: dict | None, out: dict) -> None:
+    """The batched decode of the requests whose prompts are in reqs[:len(group)]."""
+    f = None
+    if forced is not None:
+        f = np.stack([np.ascontiguousarray(forced[idx], np.uint32) for idx in group])
+    toks = text.generate_batch(reqs[:len(group)], firsts, n_steps, forced=f)
+    for slot, idx in enumerate(group):
+        out[idx] = np.concatenate([np.array([firsts[slot]], np.uint32), toks[slot]])
 
 
 def gather_tokens(local: dict, n_requests: int, group=None) -> list:

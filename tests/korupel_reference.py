@@ -149,7 +149,9 @@ def to_bf16(a):
 
 def random_weights(cfg, seed):
     """Random weights for a configuration (bfloat16 values held as float32), sized so that the activations stay of
-    order one and every mechanism has a visible share of the output."""
+    order one and every mechanism has a visible share of the output.  Which experts a token takes must not hang on
+    rounding: the first channels (one per expert) carry a pattern of the token's own that no sublayer writes to, and the
+    routers read mostly those."""
     rng = np.random.default_rng(seed)
     W, V, taps = cfg["width"], cfg["vocab"], cfg["canon"]["taps"]
     w = {}
@@ -161,12 +163,22 @@ def random_weights(cfg, seed):
         w[name] = rng.uniform(lo, hi, n)
 
     w["embed"] = rng.standard_normal((V, W))
+    routers = [l["mlp"]["router"] for l in cfg["layers"] if l["mlp"] and l["mlp"]["kind"] == "moe"]
+    R = max((r["experts"] for r in routers), default=0)
+    if R:   # ranks of the experts per token, in clear steps
+        order = np.argsort(rng.standard_normal((V, R)), axis=1)
+        w["embed"][:, :R] = 1.5 - 3.0 * order / max(R - 1, 1)
     for i, layer in enumerate(cfg["layers"]):
         p, m = f"l{i}.", layer["mixer"]
         for n in ("norm1", "norm1b") + (("norm2", "norm2b") if layer["mlp"] is not None else ()):
             vec(p + n, W, 0.6, 1.4)
         for n in ("canon1",) + (("canon2",) if layer["mlp"] is not None else ()):
             w[p + n] = rng.standard_normal((W, taps)) * 0.4
+            w[p + n][:R] = 0
+        for n in ("norm1b",) + (("norm2b",) if layer["mlp"] is not None else ()):
+            w[p + n][:R] = 0
+        if layer["mlp"] is not None:
+            w[p + "norm2"][:R] = 1
         H, d = m["heads"], m["dim"]
         if layer["type"] == "attention":
             G = m["kv_heads"]
@@ -193,7 +205,8 @@ def random_weights(cfg, seed):
             lin(q + "gate", F, W); lin(q + "up", F, W); lin(q + "down", W, F)
         else:
             F, E = layer["mlp"]["expert"]["ff"], layer["mlp"]["router"]["experts"]
-            lin(q + "router", E, W)
+            lin(q + "router", E, W, 0.015)
+            w[q + "router"][:, :R] = 2.0 * np.eye(E, R)
             for e in range(E):
                 lin(f"{q}e{e}.gate", F, W); lin(f"{q}e{e}.up", F, W); lin(f"{q}e{e}.down", W, F)
     vec("final.norm", W, 0.6, 1.4)
