@@ -40,7 +40,7 @@ struct md_graph {
     cudaGraphExec_t exec = nullptr;
 };
 
-constexpr size_t MD_COUNTER_WORDS = 256;
+constexpr size_t MD_COUNTER_WORDS = 2048;
 constexpr size_t MD_SPLITK_TICKETS = 1024;   // tiles of a split-K GEMM (one arrival ticket each)
 
 struct md_ctx {
