@@ -593,6 +593,10 @@ ONLY_CASES = {
     "prefill": "text prefill of 761 rows through all 24 layers, three passes",
     "decode": "text decode, one request, 761-row prefill then 40 steps",
     "decode8": "text decode, eight requests batched, 761-row prefill each then 40 steps",
+    "korupel": "layer-stack decoder (Korupel design) beside the Phi-style decoder at equal size: prefill and decode",
+    "korupel_prefill": "layer-stack decoder, width 2048, six layers, 761-token prompt, three passes",
+    "korupel_decode": "layer-stack decoder, width 2048, six layers, 761-token prompt then 24 steps",
+    "korupel_decode8": "layer-stack decoder, width 2048, six layers, eight requests batched, 761-token prompts then 24 steps",
     "vision1": "vision encode + projection, one crop, three passes",
     "vision13": "vision encode + projection, thirteen crops, three passes",
 }
@@ -663,6 +667,28 @@ def run_only(ctx, torch, stream, case):
             r.close()
         tm.close()
         return out
+    if case == "korupel":
+        return korupel_case(ctx, torch)
+    if case.startswith("korupel_"):
+        m = build_stack_model(ctx, torch, g, STACK_SIZES["2048"], 6)
+        batch = 8 if case.endswith("8") else 1
+        reqs = [m.request() for _ in range(batch)]
+        ids = np.random.default_rng(4100).integers(0, m.vocab, 761)
+        for _ in range(3 if case == "korupel_prefill" else 1):
+            for r in reqs:
+                r.reset()
+                t0 = time.perf_counter()
+                m.step(r, ids, want_token=True)
+                ms = (time.perf_counter() - t0) * 1e3
+        out = {"prefill_ms": round(ms, 3)}
+        if case != "korupel_prefill":
+            t0 = time.perf_counter()
+            m.generate_batch(reqs, [1] * batch, 24)
+            out["us_per_step"] = round((time.perf_counter() - t0) / 24 * 1e6, 1)
+        for r in reqs:
+            r.close()
+        m.close()
+        return out
     crops = 13 if case == "vision13" else 1
     vw, make_vm = build_vision_model(ctx, torch, g, n)
     vm = make_vm(crops)
@@ -673,6 +699,138 @@ def run_only(ctx, torch, stream, case):
         ms = (time.perf_counter() - t0) * 1e3
     vm.close()
     return {"crops": crops, "encode_ms": round(ms, 3)}
+
+
+# The layer-stack decoder at sizes of a real model's layers.  A layer's active weights equal those of a Phi layer of the
+# same width (12 width^2): 5 width^2 in the mixer, 7 width^2 in the feed-forward (of one token, for experts).
+STACK_SIZES = {
+    "2048": dict(width=2048, heads=32, kv_heads=8, dim=64, vdim=64, window=1024, keep=4, experts=16, top=2),
+    "4096": dict(width=4096, heads=32, kv_heads=8, dim=128, vdim=128, window=1024, keep=4, experts=8, top=2),
+}
+
+
+def build_stack_model(ctx, torch, g, z, layers, ff=("dense", "moe"), max_seq=2560, vocab=51200):
+    """Random-init Korupel-design decoder generated on the device: two lightning layers, then one attention layer, in turn;
+    feed-forwards alternate between dense and mixture of experts."""
+    import importlib
+    import __graft_entry__ as entry
+    models = importlib.import_module(entry.PKG_NAME + ".models")
+    W, H, G, d, e, taps = z["width"], z["heads"], z["kv_heads"], z["dim"], z["vdim"], 4
+
+    def n(*shape, std=0.02):
+        return (torch.randn(*shape, device="cuda", generator=g) * std).bfloat16()
+
+    def vec(*shape, mean=1.0, std=0.1):
+        return torch.randn(*shape, device="cuda", generator=g) * std + mean
+    out = []
+    for i in range(layers):
+        s = {"norm1": vec(W), "norm1b": vec(W), "norm2": vec(W), "norm2b": vec(W), "conv1": vec(W, taps, mean=0.0),
+             "conv2": vec(W, taps, mean=0.0), "heads": H, "dim": d, "vdim": e}
+        if i % 3 == 2:
+            rows = (H + G) * d + H
+            s.update(mixer=models.MIXER_WINDOW_ATTENTION, kv_heads=G, scale=d ** -0.5, window=z["window"], keep_first=z["keep"],
+                     r1=vec(H, mean=0.4), r2=vec(H, mean=0.4), b_in=vec(rows, mean=0.0), vdim=d)
+        else:
+            rows = 2 * H * (d + e)
+            s.update(mixer=models.MIXER_LIGHTNING, decay=torch.linspace(0.6, 0.999, H, device="cuda"), mix_norm=vec(H * e))
+        s.update(w_in=n((rows + 7) // 8 * 8, W), w_out=n(W, H * s["vdim"]))
+        if ff[i % len(ff)] == "dense":
+            F = 7 * W // 3 // 32 * 32
+            s.update(ff=models.FF_DENSE, act=models.ACT_GELU_TANH, ff_dim=F, w_gate_up=n(2 * F, W), w_down=n(W, F))
+        else:
+            E, F = z["experts"], 7 * W // 3 // z["top"] // 32 * 32
+            s.update(ff=models.FF_MOE, act=models.ACT_SILU, ff_dim=F, experts=E, top=z["top"], router=n(E, W),
+                     w_gate_up=n(E, 2 * F, W), w_down=n(E, W, F))
+        out.append(s)
+    return models.StackModel(ctx, out, embed=n(vocab, W, std=1.0), head=n(vocab, W), final_norm=vec(W), eps=1e-5, residual_mult=0.5,
+                             taps=taps, max_seq=max_seq)
+
+
+def korupel_case(ctx, torch):
+    """Prefill and decode throughput of the layer-stack decoder and of the Phi-style decoder with as many layers of the same
+    width, vocabulary and active weights.  Host wall clock around the library's calls (ids or embeddings copied up, tokens
+    read back), best of the repetitions that replay recorded graphs."""
+    import importlib
+    import __graft_entry__ as entry
+    models = importlib.import_module(entry.PKG_NAME + ".models")
+    out = {"note": "tokens/s; weights random, vocabulary 51200, prompts of 761 and 2048 tokens, 200 greedy steps after 761 tokens"}
+
+    def best(fn, reps=5):
+        times = []
+        for _ in range(reps):
+            t0 = time.perf_counter()
+            fn()
+            times.append(time.perf_counter() - t0)
+        return min(times[2:])
+
+    for name, layers in (("2048", 12), ("4096", 6)):
+        z = STACK_SIZES[name]
+        W = z["width"]
+        rows = {}
+        for ff in (("dense",), ("moe",)):
+            g = torch.Generator(device="cuda").manual_seed(4200)
+            m = build_stack_model(ctx, torch, g, z, layers, ff=ff)
+            reqs = [m.request() for _ in range(8)]
+            r, res = reqs[0], {}
+            for n in (761, 2048):
+                ids = np.random.default_rng(n).integers(0, m.vocab, n)
+
+                def prefill():
+                    r.reset()
+                    m.step(r, ids, want_token=True)
+                res[f"prefill_{n}"] = round(n / best(prefill), 0)
+
+            def decode(batch):
+                def fn():
+                    m.generate_batch(reqs[:batch], [1] * batch, 200)
+                for q in reqs[:batch]:
+                    q.reset()
+                    m.step(q, np.arange(761))
+                return round(batch * 200 / best(fn, 4), 1)
+            res["decode_1"], res["decode_8"] = decode(1), decode(8)
+            rows["korupel_" + ff[0]] = res
+            for q in reqs:
+                q.close()
+            m.close()
+            del m, reqs, r
+            torch.cuda.empty_cache()
+        g = torch.Generator(device="cuda").manual_seed(4300)
+
+        def n(*shape, std=0.02):
+            return (torch.randn(*shape, device="cuda", generator=g) * std).half()
+        D, F, V = W, 4 * W, 51200
+        ones, zeros = torch.ones(D, device="cuda").half(), torch.zeros(D, device="cuda").half()
+        w = {"ln_w": [ones] * layers, "ln_b": [zeros] * layers, "wqkv": [n(3 * D, D) for _ in range(layers)],
+             "bqkv": [n(3 * D) for _ in range(layers)], "wout": [n(D, D) for _ in range(layers)], "bout": [n(D) for _ in range(layers)],
+             "wfc1": [n(F, D) for _ in range(layers)], "bfc1": [n(F) for _ in range(layers)],
+             "wfc2": [n(D, F) for _ in range(layers)], "bfc2": [n(D) for _ in range(layers)], "ln_out_w": ones, "ln_out_b": zeros,
+             "lm_w": n(V, D), "lm_b": n(V), "wte": n(V, D)}
+        tm = models.TextModel(ctx, w, n_heads=D // 64, max_seq=2560)
+        reqs, res = [tm.request() for _ in range(8)], {}
+        for k in (761, 2048):
+            ids = np.random.default_rng(k).integers(0, V, k)
+
+            def prefill():
+                reqs[0].reset()
+                tm.step(reqs[0], ids, want_token=True)
+            res[f"prefill_{k}"] = round(k / best(prefill), 0)
+
+        def decode(batch):
+            def fn():
+                tm.generate_batch(reqs[:batch], [1] * batch, 200)
+            for q in reqs[:batch]:
+                q.reset()
+                tm.step(q, np.arange(761))
+            return round(batch * 200 / best(fn, 4), 1)
+        res["decode_1"], res["decode_8"] = decode(1), decode(8)
+        rows["phi"] = res
+        for q in reqs:
+            q.close()
+        tm.close()
+        del w, tm
+        torch.cuda.empty_cache()
+        out[f"width_{name}_layers_{layers}"] = rows
+    return out
 
 
 def build_text_model(ctx, torch, g):

@@ -1,13 +1,45 @@
 // Mixture of experts with independent logistic scores (md_moe in stack.cuh).
-//   moe_router_kernel   scores and top choice per token (f32), and each (token, expert) pair's rank within its expert
+//
+// Prompts (and every shape the kernels below cannot take):
+//   moe_router_kernel, moe_router_mma_kernel
+//                       scores and top choice per token (f32 sums of exact bfloat16 products, or f32 throughout), and each
+//                       (token, expert) pair's rank within its expert
 //   moe_permute_kernel  rows sorted by expert, every expert's rows starting at a multiple of 128
 // then the two expert products run as grouped products over the sorted rows, and the weighted sum of a token's experts
 // is taken where the residual is updated (md_glue::slot).
-#include "stack.cuh"
+//
+// Up to eight bfloat16 tokens (a decode step), weights streamed as in gemv.cu:
+//   moe_route_kernel    scores of all tokens; the last block to arrive chooses and lists the experts in use ("slots") with
+//                       every token's weight in each (zero where the token does not use it)
+//   moe_up_kernel       the slots' gated products, times the token's weight
+//   moe_down_kernel     one long product over all slots' columns, so the weighted sum needs no second pass
+#include "mma_bf16.cuh"
 
 namespace {
 
 constexpr int MAX_EXPERTS = 512, MAX_TOP = 32;
+
+// The `top` largest of s[0 .. E) (shared memory, lowest index first among equals), by one warp: fn(k, expert, score).
+template <class F>
+__device__ __forceinline__ void warp_top(float* s, int E, int top, int lane, F&& fn) {
+    for (int k = 0; k < top; ++k) {
+        float best = -1.f;
+        int bi = 0;
+        for (int e = lane; e < E; e += 32)
+            if (s[e] > best) { best = s[e]; bi = e; }
+#pragma unroll
+        for (int o = 16; o; o >>= 1) {
+            const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+            const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+            if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; }
+        }
+        if (lane == 0) {
+            fn(k, bi, best);
+            s[bi] = -2.f;
+        }
+        __syncwarp();
+    }
+}
 
 // one warp per token
 template <class T>
@@ -30,25 +62,11 @@ moe_router_kernel(const T* __restrict__ h, const T* __restrict__ router, int row
         if (lane == 0) s[e] = md_logistic(z);
     }
     __syncwarp();
-    for (int k = 0; k < top; ++k) {
-        float best = -1.f;
-        int bi = 0;
-        for (int e = lane; e < E; e += 32)
-            if (s[e] > best) { best = s[e]; bi = e; }
-#pragma unroll
-        for (int o = 16; o; o >>= 1) {
-            const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-            const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-            if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; }
-        }
-        if (lane == 0) {
-            score[(size_t)t * top + k] = best;
-            sel[(size_t)t * top + k] = bi;
-            rank[(size_t)t * top + k] = atomicAdd(count + bi, 1);
-            s[bi] = -2.f;
-        }
-        __syncwarp();
-    }
+    warp_top(s, E, top, lane, [&](int k, int e, float v) {
+        score[(size_t)t * top + k] = v;
+        sel[(size_t)t * top + k] = e;
+        rank[(size_t)t * top + k] = atomicAdd(count + e, 1);
+    });
 }
 
 template <class T>
@@ -86,7 +104,10 @@ moe_permute_kernel(const T* __restrict__ h, int W, int E, int top, const int* __
         const int e = sel[(size_t)t * top + k], row = first[e] * MD_GROUP_ROWS + rank[(size_t)t * top + k];
         if (threadIdx.x == 0) slot[(size_t)t * top + k] = row;
         T* dst = xs + (size_t)row * W;
-        if ((W % 4) == 0) {
+        if ((W * sizeof(T)) % 16 == 0) {
+            for (int c = threadIdx.x; c < (int)(W * sizeof(T) / 16); c += blockDim.x)
+                reinterpret_cast<uint4*>(dst)[c] = reinterpret_cast<const uint4*>(src)[c];
+        } else if ((W % 4) == 0) {
             for (int c = threadIdx.x * 4; c < W; c += blockDim.x * 4) {
                 float f[4];
                 md_load4<T>(src + c, f);
@@ -98,12 +119,308 @@ moe_permute_kernel(const T* __restrict__ h, int W, int E, int top, const int* __
     }
 }
 
+__device__ __forceinline__ uint4 ldg_stream(const void* p) {
+    uint4 v;
+    asm volatile("ld.global.nc.L1::no_allocate.v4.u32 {%0,%1,%2,%3}, [%4];"
+                 : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w)
+                 : "l"(p));
+    return v;
+}
+__device__ __forceinline__ uint4 ld_act(const void* p) {
+    uint4 v;
+    asm volatile("ld.global.cg.v4.u32 {%0,%1,%2,%3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p) : "memory");
+    return v;
+}
+// 32 k values of 16 rows (lo: rows g, hi: rows g + 8) against 8 columns: the order of k inside a sum is free, so a lane's
+// 8 consecutive values feed two MMAs
+__device__ __forceinline__ void mma_piece(float (&c)[4], const uint4& lo, const uint4& hi, const uint4& x) {
+    mb::mma(c, lo.x, hi.x, lo.y, hi.y, x.x, x.y);
+    mb::mma(c, lo.z, hi.z, lo.w, hi.w, x.z, x.w);
+}
+
+constexpr int RT = 16, RE = 64;   // tokens per block, experts per pass
+
+__global__ void __launch_bounds__(256)
+moe_router_mma_kernel(const __nv_bfloat16* h, const __nv_bfloat16* __restrict__ router, int rows, int W, int E, int top, float* score,
+                      int* sel, int* rank, int* count) {
+    extern __shared__ float smf[];
+    float (*part)[RT][RE] = reinterpret_cast<float (*)[RT][RE]>(smf);   // [8 warps]
+    float* sc = smf + 8 * RT * RE;                                      // [RT][E]
+    int* cnt = reinterpret_cast<int*>(sc + RT * E);                     // [E]: this block's tokens per expert, then its base
+    md_pdl_launch_dependents();
+    md_pdl_wait();
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+    const int t0 = blockIdx.x * RT, n = min(RT, rows - t0);
+    for (int e = tid; e < E; e += 256) cnt[e] = 0;
+    const __nv_bfloat16* lo = h + (size_t)(t0 + min(g, n - 1)) * W + t * 8;
+    const __nv_bfloat16* hi = h + (size_t)(t0 + min(g + 8, n - 1)) * W + t * 8;
+    for (int e0 = 0; e0 < E; e0 += RE) {
+        float acc[RE / 8][4];
+#pragma unroll
+        for (int i = 0; i < RE / 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+        for (int k = warp * 32; k < W; k += 256) {
+            const bool live = k + t * 8 < W;      // W % 8 == 0
+            const uint4 z = make_uint4(0, 0, 0, 0), a = live ? ld_act(lo + k) : z, b = live ? ld_act(hi + k) : z;
+#pragma unroll
+            for (int i = 0; i < RE / 8; ++i) {
+                const int e = e0 + i * 8 + g;
+                const uint4 x = live && e < E ? *reinterpret_cast<const uint4*>(router + (size_t)e * W + t * 8 + k) : z;
+                mma_piece(acc[i], a, b, x);
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < RE / 8; ++i) {
+            part[warp][g][i * 8 + 2 * t] = acc[i][0];
+            part[warp][g][i * 8 + 2 * t + 1] = acc[i][1];
+            part[warp][g + 8][i * 8 + 2 * t] = acc[i][2];
+            part[warp][g + 8][i * 8 + 2 * t + 1] = acc[i][3];
+        }
+        __syncthreads();
+        for (int i = tid; i < RT * RE; i += 256) {
+            const int r = i / RE, e = i % RE;
+            float v = 0.f;
+#pragma unroll
+            for (int w = 0; w < 8; ++w) v += part[w][r][e];
+            if (e0 + e < E) sc[r * E + e0 + e] = md_logistic(v);
+        }
+        __syncthreads();
+    }
+    for (int r = warp; r < n; r += 8)
+        warp_top(sc + r * E, E, top, lane, [&](int k, int e, float v) {
+            const size_t at = (size_t)(t0 + r) * top + k;
+            score[at] = v;
+            sel[at] = e;
+            rank[at] = atomicAdd(cnt + e, 1);
+        });
+    __syncthreads();
+    for (int e = tid; e < E; e += 256)
+        if (cnt[e]) cnt[e] = atomicAdd(count + e, cnt[e]);
+    __syncthreads();
+    for (int i = tid; i < n * top; i += 256) {   // this block wrote sel and rank of its tokens
+        const size_t at = (size_t)t0 * top + i;
+        rank[at] += cnt[sel[at]];
+    }
+}
+
+// ---- up to eight tokens
+struct Route {
+    float* score;        // [8][E]
+    float* weight;       // [slots][8]
+    int *expert, *n_slots;
+    unsigned* ticket;    // zero between launches
+};
+
+__global__ void __launch_bounds__(512)
+moe_route_kernel(const __nv_bfloat16* h, const __nv_bfloat16* __restrict__ router, int T, int W, int E, int top, Route r) {
+    extern __shared__ float sc[];            // last block: [8][E] scores, then [8][E] chosen scores
+    __shared__ float partial[16][16][8];
+    __shared__ int last_s;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+    const int row0 = blockIdx.x * 16;
+    const __nv_bfloat16* w_lo = router + (size_t)min(row0 + g, E - 1) * W + t * 8;
+    const __nv_bfloat16* w_hi = router + (size_t)min(row0 + g + 8, E - 1) * W + t * 8;
+    const __nv_bfloat16* x = h + (size_t)min(g, T - 1) * W + t * 8;
+    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+    const uint4 zero = make_uint4(0, 0, 0, 0);
+    md_pdl_launch_dependents();
+    bool waited = false;
+    for (int k0 = warp * 32; k0 < W; k0 += 4 * 512) {
+        uint4 lo[4], hi[4], xv[4];
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+            const int k = k0 + u * 512;
+            const bool live = k + t * 8 < W;
+            lo[u] = live ? ldg_stream(w_lo + k) : zero;
+            hi[u] = live ? ldg_stream(w_hi + k) : zero;
+        }
+        if (!waited) md_pdl_wait();
+        waited = true;
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+            const int k = k0 + u * 512;
+            xv[u] = g < T && k + t * 8 < W ? ld_act(x + k) : zero;
+        }
+#pragma unroll
+        for (int u = 0; u < 4; ++u) mma_piece(acc, lo[u], hi[u], xv[u]);
+    }
+    if (!waited) md_pdl_wait();
+    partial[warp][g][2 * t] = acc[0];
+    partial[warp][g][2 * t + 1] = acc[1];
+    partial[warp][g + 8][2 * t] = acc[2];
+    partial[warp][g + 8][2 * t + 1] = acc[3];
+    __syncthreads();
+    if (tid < 128) {
+        const int m = tid >> 4, e = tid & 15;
+        float v = 0.f;
+#pragma unroll
+        for (int w = 0; w < 16; ++w) v += partial[w][e][m];
+        if (m < T && row0 + e < E) r.score[m * E + row0 + e] = md_logistic(v);
+    }
+    __threadfence();
+    __syncthreads();
+    if (tid == 0) last_s = atomicAdd(r.ticket, 1u) == gridDim.x - 1;
+    __syncthreads();
+    if (!last_s) return;
+    __threadfence();
+    if (tid == 0) *r.ticket = 0u;
+    float* chosen = sc + 8 * E;
+    for (int i = tid; i < T * E; i += 512) {
+        sc[i] = __ldcg(r.score + i);
+        chosen[i] = 0.f;
+    }
+    __syncthreads();
+    if (warp < T) warp_top(sc + warp * E, E, top, lane, [&](int, int e, float v) { chosen[warp * E + e] = v; });
+    __syncthreads();
+    if (warp == 0) {
+        int slots = 0;
+        for (int e0 = 0; e0 < E; e0 += 32) {
+            const int e = e0 + lane;
+            bool used = false;
+            for (int m = 0; m < T; ++m) used |= e < E && chosen[m * E + e] != 0.f;
+            const unsigned b = __ballot_sync(0xffffffffu, used);
+            if (used) {
+                const int s = slots + __popc(b & ((1u << lane) - 1u));
+                r.expert[s] = e;
+                for (int m = 0; m < 8; ++m) r.weight[s * 8 + m] = m < T ? chosen[m * E + e] : 0.f;
+            }
+            slots += __popc(b);
+        }
+        if (lane == 0) *r.n_slots = slots;
+    }
+}
+
+// act[token][slot * ff_pad + j] = weight * act(gate_j) * up_j
+__global__ void __launch_bounds__(256)
+moe_up_kernel(const __nv_bfloat16* h, const __nv_bfloat16* __restrict__ w_gu, __nv_bfloat16* out, int T, int W, int ff_pad, int act,
+              int out_stride, Route r) {
+    __shared__ float partial[8][16][8];
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+    const int slot = blockIdx.y, j = blockIdx.x * 8 + g;
+    md_pdl_launch_dependents();
+    md_pdl_wait();
+    if (slot >= __ldcg(r.n_slots)) return;
+    const __nv_bfloat16* w = w_gu + (size_t)__ldcg(r.expert + slot) * 2 * ff_pad * W;
+    const __nv_bfloat16* w_lo = w + (size_t)((j / MD_GLU_BLOCK) * (2 * MD_GLU_BLOCK) + j % MD_GLU_BLOCK) * W + t * 8;
+    const __nv_bfloat16* w_hi = w_lo + (size_t)MD_GLU_BLOCK * W;
+    const bool has_x = g < T && __ldcg(r.weight + slot * 8 + g) != 0.f;
+    const __nv_bfloat16* x = h + (size_t)(has_x ? g : 0) * W + t * 8;
+    const uint4 zero = make_uint4(0, 0, 0, 0);
+    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+    for (int k0 = warp * 32; k0 < W; k0 += 8 * 256) {
+        uint4 lo[8], hi[8], xv[8];
+#pragma unroll
+        for (int u = 0; u < 8; ++u) {
+            const int k = k0 + u * 256;
+            const bool live = k + t * 8 < W;
+            lo[u] = live ? ldg_stream(w_lo + k) : zero;
+            hi[u] = live ? ldg_stream(w_hi + k) : zero;
+            xv[u] = live && has_x ? ld_act(x + k) : zero;
+        }
+#pragma unroll
+        for (int u = 0; u < 8; ++u) mma_piece(acc, lo[u], hi[u], xv[u]);
+    }
+    partial[warp][g][2 * t] = acc[0];
+    partial[warp][g][2 * t + 1] = acc[1];
+    partial[warp][g + 8][2 * t] = acc[2];
+    partial[warp][g + 8][2 * t + 1] = acc[3];
+    __syncthreads();
+    if (tid < 64) {
+        const int m = tid >> 3, e = tid & 7;
+        if (m < T) {
+            float a = 0.f, b = 0.f;
+#pragma unroll
+            for (int q = 0; q < 8; ++q) {
+                a += partial[q][e][m];
+                b += partial[q][e + 8][m];
+            }
+            const float wt = __ldcg(r.weight + slot * 8 + m);
+            out[(size_t)m * out_stride + slot * ff_pad + blockIdx.x * 8 + e] = __float2bfloat16_rn(wt * md_act(act, a) * b);
+        }
+    }
+}
+
+// y[token][n] = sum over the slots' columns
+__global__ void __launch_bounds__(512)
+moe_down_kernel(const __nv_bfloat16* act, const __nv_bfloat16* __restrict__ w_down, float* y, int T, int W, int ff_pad, int act_stride,
+                Route r) {
+    __shared__ float partial[16][16][8];
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+    const int row0 = blockIdx.x * 16;
+    md_pdl_launch_dependents();
+    md_pdl_wait();
+    const int per = ff_pad / 32, chunks = __ldcg(r.n_slots) * per;
+    const size_t r_lo = min(row0 + g, W - 1), r_hi = min(row0 + g + 8, W - 1);
+    const __nv_bfloat16* x = act + (size_t)(g < T ? g : 0) * act_stride + t * 8;
+    const uint4 zero = make_uint4(0, 0, 0, 0);
+    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+    constexpr int U = 4;
+    for (int c0 = warp; c0 < chunks; c0 += U * 16) {
+        uint4 lo[U], hi[U], xv[U];
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+            const int c = c0 + u * 16;
+            lo[u] = hi[u] = xv[u] = zero;
+            if (c < chunks) {
+                const int slot = c / per, k = (c - slot * per) * 32 + t * 8;
+                const __nv_bfloat16* w = w_down + (size_t)__ldcg(r.expert + slot) * W * ff_pad + k;
+                lo[u] = ldg_stream(w + r_lo * ff_pad);
+                hi[u] = ldg_stream(w + r_hi * ff_pad);
+                if (g < T) xv[u] = ld_act(x + c * 32);
+            }
+        }
+#pragma unroll
+        for (int u = 0; u < U; ++u) mma_piece(acc, lo[u], hi[u], xv[u]);
+    }
+    partial[warp][g][2 * t] = acc[0];
+    partial[warp][g][2 * t + 1] = acc[1];
+    partial[warp][g + 8][2 * t] = acc[2];
+    partial[warp][g + 8][2 * t + 1] = acc[3];
+    __syncthreads();
+    if (tid < 128) {
+        const int m = tid >> 4, e = tid & 15;
+        if (m < T && row0 + e < W) {
+            float v = 0.f;
+#pragma unroll
+            for (int w = 0; w < 16; ++w) v += partial[w][e][m];
+            y[(size_t)m * W + row0 + e] = v;
+        }
+    }
+}
+
+int launch_few(md_ctx* ctx, const md_moe& m, const void* h, size_t rows, const md_moe_buffers& b) {
+    const int T = (int)rows, E = m.experts, slots = T * m.top < E ? T * m.top : E;
+    Route r;
+    // the ticket first: layers of different sizes share the buffer, and it must stay what the last launch left, zero
+    r.ticket = reinterpret_cast<unsigned*>(b.route);
+    r.n_slots = reinterpret_cast<int*>(b.route) + 1;
+    r.score = b.route + 8;
+    r.weight = r.score + 8 * (size_t)E;
+    r.expert = reinterpret_cast<int*>(r.weight + 8 * (size_t)E);
+    const __nv_bfloat16* x = reinterpret_cast<const __nv_bfloat16*>(h);
+    __nv_bfloat16* act = reinterpret_cast<__nv_bfloat16*>(b.act);
+    MD_TRY(md_launch_ex(ctx, moe_route_kernel, dim3((unsigned)((E + 15) / 16)), dim3(512), 16 * (size_t)E * sizeof(float), "moe_route_kernel",
+                        x, reinterpret_cast<const __nv_bfloat16*>(m.router), T, m.width, E, m.top, r));
+    MD_TRY(md_launch_ex(ctx, moe_up_kernel, dim3((unsigned)(m.ff_pad / 8), (unsigned)slots), dim3(256), 0, "moe_up_kernel", x,
+                        reinterpret_cast<const __nv_bfloat16*>(m.w_gu), act, T, m.width, m.ff_pad, m.act, slots * m.ff_pad, r));
+    return md_launch_ex(ctx, moe_down_kernel, dim3((unsigned)((m.width + 15) / 16)), dim3(512), 0, "moe_down_kernel", act,
+                        reinterpret_cast<const __nv_bfloat16*>(m.w_down), b.y_f32, T, m.width, m.ff_pad, slots * m.ff_pad, r);
+}
+
 template <class T>
 int launch_sorted(md_ctx* ctx, int dtype, const md_moe& m, const void* h, size_t rows, const md_moe_buffers& b) {
     MD_CUDA(ctx, cudaMemsetAsync(b.count, 0, m.experts * sizeof(int), ctx->stream));
-    MD_TRY(md_launch_ex(ctx, moe_router_kernel<T>, dim3((unsigned)((rows + 3) / 4)), dim3(128), 0, "moe_router_kernel",
-                        reinterpret_cast<const T*>(h), reinterpret_cast<const T*>(m.router), (int)rows, m.width, m.experts,
-                        m.top, b.score, b.sel, b.rank, b.count));
+    if (dtype == MD_DTYPE_BF16 && (m.width % 8) == 0) {
+        const size_t smem = (8 * RT * RE + RT * (size_t)m.experts + m.experts) * sizeof(float);
+        if (smem > 48 * 1024)
+            MD_CUDA(ctx, cudaFuncSetAttribute(moe_router_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        MD_TRY(md_launch_ex(ctx, moe_router_mma_kernel, dim3((unsigned)((rows + RT - 1) / RT)), dim3(256), smem, "moe_router_mma_kernel",
+                            reinterpret_cast<const __nv_bfloat16*>(h), reinterpret_cast<const __nv_bfloat16*>(m.router), (int)rows,
+                            m.width, m.experts, m.top, b.score, b.sel, b.rank, b.count));
+    } else {
+        MD_TRY(md_launch_ex(ctx, moe_router_kernel<T>, dim3((unsigned)((rows + 3) / 4)), dim3(128), 0, "moe_router_kernel",
+                            reinterpret_cast<const T*>(h), reinterpret_cast<const T*>(m.router), (int)rows, m.width, m.experts,
+                            m.top, b.score, b.sel, b.rank, b.count));
+    }
     MD_TRY(md_launch_ex(ctx, moe_permute_kernel<T>, dim3((unsigned)rows), dim3(256), 0, "moe_permute_kernel",
                         reinterpret_cast<const T*>(h), m.width, m.experts, m.top, b.sel, b.rank, b.count, b.slot,
                         b.tile_expert, b.n_blocks, reinterpret_cast<T*>(b.xs)));
@@ -121,9 +438,8 @@ int launch_sorted(md_ctx* ctx, int dtype, const md_moe& m, const void* h, size_t
 
 }  // namespace
 
-bool md_moe_sorted(int dtype, size_t rows) {
-    (void)dtype, (void)rows;
-    return true;
+bool md_moe_sorted(int dtype, size_t width, size_t rows) {
+    return dtype != MD_DTYPE_BF16 || (width % 8) != 0 || rows > 8;
 }
 
 size_t md_moe_sorted_rows(size_t rows, int experts, int top) {
@@ -135,6 +451,7 @@ size_t md_moe_sorted_rows(size_t rows, int experts, int top) {
 int md_launch_moe(md_ctx* ctx, int dtype, const md_moe& m, const void* h, size_t rows, const md_moe_buffers& b) {
     if (m.experts > MAX_EXPERTS || m.top > MAX_TOP || m.top > m.experts)
         return md_fail(ctx, MD_ERR_UNSUPPORTED, "mixture of experts: %d experts, %d per token", m.experts, m.top);
+    if (!md_moe_sorted(dtype, m.width, rows)) return launch_few(ctx, m, h, rows, b);
     return dtype == MD_DTYPE_F32 ? launch_sorted<float>(ctx, dtype, m, h, rows, b)
                                  : launch_sorted<__nv_bfloat16>(ctx, dtype, m, h, rows, b);
 }

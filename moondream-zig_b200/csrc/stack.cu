@@ -20,7 +20,7 @@ struct md_stack_request {
     DevPtr keys;      // all key caches
     DevPtr state;     // all f32 states, zeroed by a reset
     DevPtr x[2], h, in, o, y, ff, ssq;
-    DevPtr score, sel, rank, slot, count, tile_expert, n_blocks, xs, act, ys;
+    DevPtr route, score, sel, rank, slot, count, tile_expert, n_blocks, xs, act, ys;
     DevPtr trace;     // [layers][rows][width] when stack_trace is set
     size_t cap_rows = 0, trace_rows = 0;
 };
@@ -50,7 +50,7 @@ md_glue update_after(const md_stack& s, md_stack_request* b, size_t i, bool ff, 
     const md_stack_layer& l = s.layers[i];
     md_glue g = base_glue(s, rows, seqs);
     g.w_post = ff ? l.norm2b : l.norm1b;
-    if (ff && l.ff == MD_FF_MOE && md_moe_sorted(s.w.dtype, rows * seqs)) {
+    if (ff && l.ff == MD_FF_MOE && md_moe_sorted(s.w.dtype, s.w.width, rows * seqs)) {
         g.slot = b->slot.as<int>(), g.score = b->score.as<float>(), g.top = (int)l.top;
         g.y = b->ys.p;
         return g;
@@ -147,6 +147,11 @@ int md_stack_request_create(md_text_request* req) {
     md_stack_request* r = req->stack = new md_stack_request();
     MD_TRY(r->keys.ensure(ctx, std::max<size_t>(s.kv_bytes, 256)));
     MD_TRY(r->state.ensure(ctx, std::max<size_t>(s.state_floats, 64) * sizeof(float)));
+    if (s.max_experts) {
+        const size_t bytes = md_moe_route_floats(s.max_experts) * sizeof(float);
+        MD_TRY(r->route.ensure(ctx, bytes));
+        MD_CUDA(ctx, cudaMemsetAsync(r->route.p, 0, bytes, ctx->stream));
+    }
     MD_TRY(md_stack_reserve(req, MD_STACK_MAX_SEQS));
     return md_stack_request_reset(req);
 }
@@ -284,7 +289,7 @@ int md_stack_layers(md_text_model* m, md_text_request* const* reqs, size_t seqs,
             md_moe_buffers mb;
             mb.score = b->score.as<float>(), mb.sel = b->sel.as<int>(), mb.rank = b->rank.as<int>(), mb.slot = b->slot.as<int>();
             mb.count = b->count.as<int>(), mb.tile_expert = b->tile_expert.as<int>(), mb.n_blocks = b->n_blocks.as<int>();
-            mb.xs = b->xs.p, mb.act = b->act.p, mb.ys = b->ys.p, mb.y_f32 = b->y.as<float>();
+            mb.xs = b->xs.p, mb.act = b->act.p, mb.ys = b->ys.p, mb.y_f32 = b->y.as<float>(), mb.route = b->route.as<float>();
             MD_TRY(md_launch_moe(ctx, dt, e, b->h.p, T, mb));
         }
         next = update_after(s, b, i, true, rows, seqs);

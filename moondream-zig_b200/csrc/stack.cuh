@@ -118,11 +118,13 @@ struct md_moe_buffers {
     int *count = nullptr;         // [experts]
     int *tile_expert = nullptr, *n_blocks = nullptr;
     void *xs = nullptr, *act = nullptr, *ys = nullptr;        // sorted rows
-    float* y_f32 = nullptr;       // [rows, width] (decode)
+    float* y_f32 = nullptr;       // [rows, width], rows <= 8
+    float* route = nullptr;       // md_moe_route_floats(experts), zeroed once
 };
+inline size_t md_moe_route_floats(size_t experts) { return 17 * experts + 8; }
 size_t md_moe_sorted_rows(size_t rows, int experts, int top);   // capacity of the sorted buffers
 // true: md_launch_moe leaves a token's outputs in the sorted rows (slot, score, ys); false: their sum in y_f32
-bool md_moe_sorted(int dtype, size_t rows);
+bool md_moe_sorted(int dtype, size_t width, size_t rows);
 int md_launch_moe(md_ctx* ctx, int dtype, const md_moe& m, const void* h, size_t rows, const md_moe_buffers& b);
 
 int md_launch_argmax_f32(md_ctx* ctx, const float* x, size_t n, size_t stride, size_t rows, unsigned long long* idx_dev);

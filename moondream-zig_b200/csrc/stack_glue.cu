@@ -208,7 +208,7 @@ int launch_glue(md_ctx* ctx, const md_glue& g) {
     const bool wide = g.rows == 1 || (g.gather && g.rows <= 8);
     const size_t row_bytes = (size_t)g.width * sizeof(float);
     int R = wide ? 1 : 8 - halo;
-    if (R < halo) R = halo;
+    if (!wide && R < halo) R = halo;
     if (R < 1) R = 1;
     while (!wide && R > halo && R > 1 && (R + halo) * row_bytes > 100 * 1024) --R;   // two blocks per SM where possible
     const size_t smem = (R + halo) * row_bytes;
@@ -217,7 +217,7 @@ int launch_glue(md_ctx* ctx, const md_glue& g) {
     const bool v4 = (g.width % 4) == 0;
     auto kern = wide ? (v4 ? stack_glue_kernel<T, 4, true> : stack_glue_kernel<T, 1, true>)
                      : (v4 ? stack_glue_kernel<T, 4, false> : stack_glue_kernel<T, 1, false>);
-    if (smem > 48 * 1024) MD_CUDA(ctx, cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
+    if (smem > 47 * 1024) MD_CUDA(ctx, cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
     return md_launch_ex(ctx, kern, dim3((unsigned)((g.rows + R - 1) / R), (unsigned)g.seqs), dim3(wide ? 512 : 256), smem,
                         "stack_glue_kernel", g, R);
 }

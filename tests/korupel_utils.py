@@ -38,7 +38,7 @@ CONFIGS = {
                               attention(4, 1, 18, 5, 9, moe(4, 4, 11))], eps=3e-4, mult=1.3),
     # values that are 1 or equal: one tap, one expert per token, a window of one key, one head, width = head size
     "ones": config(32, 40, 1, [attention(1, 1, 32, 1, 1, moe(3, 1, 32)), lightning(1, 32, 32, dense(32), decay=[1.0]),
-                               attention(2, 2, 16, 3, 0, dense(64)), lightning(2, 1, 1, None, decay=[0.0, 0.5])], mult=1.0),
+                               attention(2, 2, 16, 3, 0, dense(64)), lightning(2, 1, 1, None, decay=[0.0, 0.5])], eps=0.05, mult=1.0),
     # multiples of 8 and 16: the tensor-core and vector paths
     "even": config(192, 136, 3, [lightning(3, 64, 48, dense(320)), attention(8, 2, 64, 100, 5, moe(16, 3, 64)),
                                  lightning(4, 32, 64, moe(9, 4, 96)), attention(6, 1, 80, 33, 1, dense(128))]),
@@ -66,12 +66,10 @@ def rel_err(got, want):
 
 
 LIMITS = {"float32": 5e-5, "bfloat16": 0.1}
-# the RMS norm over two single-value heads blows rounding up where both are small
-SLACK = {"ones": 3.0}
 
 
 def assert_logits(got, want, dtype, what=""):
-    e = rel_err(got, want) / SLACK.get(what[:4], 1.0)
+    e = rel_err(got, want)
     assert np.isfinite(np.asarray(got)).all(), what
     over = int((e > LIMITS[dtype]).sum())
     assert over == 0, f"{what}: {over} of {e.size} rows over {LIMITS[dtype]}, worst {e.max():.3e}, first {np.nonzero(e > LIMITS[dtype])[0][:8]}"
