@@ -307,6 +307,18 @@ gemv_lin_kernel(const __half* A, const __half* __restrict__ Bt, __nv_bfloat16* C
         s = md_lin_col(s, n, ep.silu_cols, ep.sigmoid_from);
         if (ep.out_f32) ep.out_f32[(size_t)m * N + n] = s;
         else C[(size_t)m * N + n] = __float2bfloat16_rn(s);
+        if (ep.amax) partial[0][r][m] = s;     // the sums of this output are read: its place is free
+    }
+    if (ep.amax) {      // greedy sampling: one atomic per block and row
+        __syncthreads();
+        if ((int)threadIdx.x < M) {
+            unsigned long long best = 0ull;
+            for (int r = 0; r < ROWS_PER_CTA && (int)blockIdx.x * ROWS_PER_CTA + r < N; ++r) {
+                const unsigned long long key = md_argmax_key(partial[0][r][threadIdx.x], blockIdx.x * ROWS_PER_CTA + r);
+                best = key > best ? key : best;
+            }
+            atomicMax(ep.amax + threadIdx.x, best);
+        }
     }
 }
 

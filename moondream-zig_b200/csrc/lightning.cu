@@ -374,10 +374,15 @@ lightning_carry_kernel(const __grid_constant__ md_lightning p, float* seg_state,
     if (i >= n) return;
     const float f = powf(p.decay[i / per], (float)seg_tokens);
     float S = p.state[0][i];
-    for (int s = 0; s < n_seg; ++s) {
-        const float u = s < n_seg - 1 ? seg_state[s * n + i] : 0.f;
-        seg_state[s * n + i] = S;
-        S = fmaf(f, S, u);
+    for (int s0 = 0; s0 < n_seg; s0 += 8) {     // eight contributions requested at a time
+        float u[8];
+#pragma unroll
+        for (int k = 0; k < 8; ++k) u[k] = s0 + k < n_seg - 1 ? seg_state[(s0 + k) * n + i] : 0.f;
+#pragma unroll
+        for (int k = 0; k < 8; ++k) {
+            if (s0 + k < n_seg) seg_state[(s0 + k) * n + i] = S;
+            S = fmaf(f, S, u[k]);
+        }
     }
 }
 
@@ -390,11 +395,11 @@ int launch_chunks_as(md_ctx* ctx, const md_lightning& l) {
         MD_CUDA(ctx, cudaFuncSetAttribute(out, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Sh::SMEM));
         MD_CUDA(ctx, cudaFuncSetAttribute(acc, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Sh::SMEM));
     }
-    // segments: about two blocks per SM, at least two chunks each (the state is computed twice per segment)
+    // segments: about three blocks per SM; two chunks are not worth the two further kernels
     const int chunks = (l.rows + C - 1) / C;
-    int n_seg = (2 * ctx->sm_count + l.heads - 1) / l.heads;
-    if (n_seg > chunks / 2) n_seg = chunks / 2;
-    if (n_seg < 1) n_seg = 1;
+    int n_seg = (3 * ctx->sm_count + l.heads - 1) / l.heads;
+    if (n_seg > chunks) n_seg = chunks;
+    if (chunks <= 2) n_seg = 1;
     const int per = (chunks + n_seg - 1) / n_seg;
     n_seg = (chunks + per - 1) / per;
     const size_t n = (size_t)l.heads * l.dim * l.vdim;

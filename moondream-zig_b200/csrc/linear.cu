@@ -79,7 +79,7 @@ int md_linear(md_ctx* ctx, int dtype, const void* a, const void* w, void* c, siz
     if (ep.glu && (N % (2 * MD_GLU_BLOCK)) != 0) return md_fail(ctx, MD_ERR_INVALID_ARG, "md_linear: gate / up rows must come in blocks");
     if (dtype == MD_DTYPE_F32) return launch_plain<float>(ctx, a, w, c, M, N, K, ep);
     const uintptr_t align = reinterpret_cast<uintptr_t>(a) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(c);
-    if (ctx->gemm_mode != 1 && (K % 8) == 0 && (align & 15) == 0) {
+    if ((ctx->gemm_mode != 1 || ep.amax) && (K % 8) == 0 && (align & 15) == 0) {
         if (!ep.tile_expert && (M <= 8 || ep.out_f32)) {
             // f32 results of many rows (the head over the wanted rows of a prompt): eight rows at a time
             for (size_t m = 0; m < M; m += 8) {

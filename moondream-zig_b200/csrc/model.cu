@@ -602,7 +602,7 @@ int md_text_step(md_text_model* model, md_text_request* req, const uint32_t* tok
         if (model->stack) {
             int* rows_dev = reinterpret_cast<int*>(req->cur_token.as<char>() + ids_bytes);
             MD_CUDA(ctx, cudaMemcpyAsync(rows_dev, rows.data(), n_rows * sizeof(int), cudaMemcpyHostToDevice, ctx->stream));
-            MD_TRY(md_stack_head(model, req, n, rows_dev, n_rows, logits));
+            MD_TRY(md_stack_head(model, req, n, rows_dev, n_rows, logits, nullptr, nullptr));
         } else {
             for (size_t i = 0; i < n_rows; ++i) {
                 MD_TRY(text_lm_head(model, req->hidden.as<__half>() + (size_t)rows[i] * w.dim, 1, req->ln_last.as<__half>(),
@@ -636,13 +636,13 @@ static int enqueue_decode_step(md_text_model* model, md_text_request* const* req
     if (model->stack) {
         float* logits = r0->logits.as<float>();
         MD_TRY(md_stack_layers(model, reqs, batch, 1, r0->cur_token.as<unsigned long long>(), true, 0));
-        MD_TRY(md_stack_head(model, r0, batch, nullptr, batch, logits));
-        MD_TRY(md_launch_argmax_f32(ctx, logits, w.vocab, w.vocab, batch, r0->sampled.as<unsigned long long>()));
+        bool keys = false;
+        MD_TRY(md_stack_head(model, r0, batch, nullptr, batch, logits, r0->sampled.as<unsigned long long>(), &keys));
         if (keep_logits) {
             copy_logits_kernel<float><<<32, 256, 0, ctx->stream>>>(logits, r0->logits_all.as<float>(), (int)w.vocab, r0->step.as<int>());
             MD_LAUNCH_CHECK(ctx, "copy_logits_kernel");
         }
-        advance_kernel<<<1, 256, 0, ctx->stream>>>(r0->cur_token.as<unsigned long long>(), r0->sampled.as<unsigned long long>(), 0,
+        advance_kernel<<<1, 256, 0, ctx->stream>>>(r0->cur_token.as<unsigned long long>(), r0->sampled.as<unsigned long long>(), keys,
                                                    (int)batch, r0->tokens_out.as<unsigned int>(), (int)n_steps,
                                                    forced ? r0->forced.as<unsigned int>() : nullptr, r0->step.as<int>(),
                                                    r0->pos_ptrs.as<int*>(), nullptr, nullptr, (int)w.dim, (int)w.vocab);

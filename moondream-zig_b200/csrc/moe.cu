@@ -140,30 +140,34 @@ __device__ __forceinline__ void mma_piece(float (&c)[4], const uint4& lo, const 
 
 constexpr int RT = 16, RE = 64;   // tokens per block, experts per pass
 
-__global__ void __launch_bounds__(256)
+constexpr int RW = 16;   // warps that split the width
+
+__global__ void __launch_bounds__(RW * 32)
 moe_router_mma_kernel(const __nv_bfloat16* h, const __nv_bfloat16* __restrict__ router, int rows, int W, int E, int top, float* score,
                       int* sel, int* rank, int* count) {
     extern __shared__ float smf[];
-    float (*part)[RT][RE] = reinterpret_cast<float (*)[RT][RE]>(smf);   // [8 warps]
-    float* sc = smf + 8 * RT * RE;                                      // [RT][E]
+    float (*part)[RT][RE] = reinterpret_cast<float (*)[RT][RE]>(smf);   // [RW]
+    float* sc = smf + RW * RT * RE;                                      // [RT][E]
     int* cnt = reinterpret_cast<int*>(sc + RT * E);                     // [E]: this block's tokens per expert, then its base
     md_pdl_launch_dependents();
     md_pdl_wait();
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
     const int t0 = blockIdx.x * RT, n = min(RT, rows - t0);
-    for (int e = tid; e < E; e += 256) cnt[e] = 0;
+    for (int e = tid; e < E; e += RW * 32) cnt[e] = 0;
     const __nv_bfloat16* lo = h + (size_t)(t0 + min(g, n - 1)) * W + t * 8;
     const __nv_bfloat16* hi = h + (size_t)(t0 + min(g + 8, n - 1)) * W + t * 8;
     for (int e0 = 0; e0 < E; e0 += RE) {
         float acc[RE / 8][4];
 #pragma unroll
         for (int i = 0; i < RE / 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
-        for (int k = warp * 32; k < W; k += 256) {
+#pragma unroll 2
+        for (int k = warp * 32; k < W; k += RW * 32) {
             const bool live = k + t * 8 < W;      // W % 8 == 0
             const uint4 z = make_uint4(0, 0, 0, 0), a = live ? ld_act(lo + k) : z, b = live ? ld_act(hi + k) : z;
 #pragma unroll
             for (int i = 0; i < RE / 8; ++i) {
                 const int e = e0 + i * 8 + g;
+                if (e0 + i * 8 >= E) break;
                 const uint4 x = live && e < E ? *reinterpret_cast<const uint4*>(router + (size_t)e * W + t * 8 + k) : z;
                 mma_piece(acc[i], a, b, x);
             }
@@ -176,16 +180,16 @@ moe_router_mma_kernel(const __nv_bfloat16* h, const __nv_bfloat16* __restrict__ 
             part[warp][g + 8][i * 8 + 2 * t + 1] = acc[i][3];
         }
         __syncthreads();
-        for (int i = tid; i < RT * RE; i += 256) {
+        for (int i = tid; i < RT * RE; i += RW * 32) {
             const int r = i / RE, e = i % RE;
             float v = 0.f;
 #pragma unroll
-            for (int w = 0; w < 8; ++w) v += part[w][r][e];
+            for (int w = 0; w < RW; ++w) v += part[w][r][e];
             if (e0 + e < E) sc[r * E + e0 + e] = md_logistic(v);
         }
         __syncthreads();
     }
-    for (int r = warp; r < n; r += 8)
+    for (int r = warp; r < n; r += RW)
         warp_top(sc + r * E, E, top, lane, [&](int k, int e, float v) {
             const size_t at = (size_t)(t0 + r) * top + k;
             score[at] = v;
@@ -193,10 +197,10 @@ moe_router_mma_kernel(const __nv_bfloat16* h, const __nv_bfloat16* __restrict__ 
             rank[at] = atomicAdd(cnt + e, 1);
         });
     __syncthreads();
-    for (int e = tid; e < E; e += 256)
+    for (int e = tid; e < E; e += RW * 32)
         if (cnt[e]) cnt[e] = atomicAdd(count + e, cnt[e]);
     __syncthreads();
-    for (int i = tid; i < n * top; i += 256) {   // this block wrote sel and rank of its tokens
+    for (int i = tid; i < n * top; i += RW * 32) {   // this block wrote sel and rank of its tokens
         const size_t at = (size_t)t0 * top + i;
         rank[at] += cnt[sel[at]];
     }
@@ -254,19 +258,19 @@ moe_route_kernel(const __nv_bfloat16* h, const __nv_bfloat16* __restrict__ route
         float v = 0.f;
 #pragma unroll
         for (int w = 0; w < 16; ++w) v += partial[w][e][m];
-        if (m < T && row0 + e < E) r.score[m * E + row0 + e] = md_logistic(v);
+        if (m < T && row0 + e < E) (gridDim.x == 1 ? sc : r.score)[m * E + row0 + e] = md_logistic(v);
     }
-    __threadfence();
-    __syncthreads();
-    if (tid == 0) last_s = atomicAdd(r.ticket, 1u) == gridDim.x - 1;
-    __syncthreads();
-    if (!last_s) return;
-    __threadfence();
-    if (tid == 0) *r.ticket = 0u;
     float* chosen = sc + 8 * E;
-    for (int i = tid; i < T * E; i += 512) {
-        sc[i] = __ldcg(r.score + i);
-        chosen[i] = 0.f;
+    for (int i = tid; i < T * E; i += 512) chosen[i] = 0.f;
+    if (gridDim.x > 1) {
+        __threadfence();
+        __syncthreads();
+        if (tid == 0) last_s = atomicAdd(r.ticket, 1u) == gridDim.x - 1;
+        __syncthreads();
+        if (!last_s) return;
+        __threadfence();
+        if (tid == 0) *r.ticket = 0u;
+        for (int i = tid; i < T * E; i += 512) sc[i] = __ldcg(r.score + i);
     }
     __syncthreads();
     if (warp < T) warp_top(sc + warp * E, E, top, lane, [&](int, int e, float v) { chosen[warp * E + e] = v; });
@@ -353,7 +357,7 @@ moe_down_kernel(const __nv_bfloat16* act, const __nv_bfloat16* __restrict__ w_do
     const __nv_bfloat16* x = act + (size_t)(g < T ? g : 0) * act_stride + t * 8;
     const uint4 zero = make_uint4(0, 0, 0, 0);
     float acc[4] = {0.f, 0.f, 0.f, 0.f};
-    constexpr int U = 4;
+    constexpr int U = 6;
     for (int c0 = warp; c0 < chunks; c0 += U * 16) {
         uint4 lo[U], hi[U], xv[U];
 #pragma unroll
@@ -410,10 +414,10 @@ template <class T>
 int launch_sorted(md_ctx* ctx, int dtype, const md_moe& m, const void* h, size_t rows, const md_moe_buffers& b) {
     MD_CUDA(ctx, cudaMemsetAsync(b.count, 0, m.experts * sizeof(int), ctx->stream));
     if (dtype == MD_DTYPE_BF16 && (m.width % 8) == 0) {
-        const size_t smem = (8 * RT * RE + RT * (size_t)m.experts + m.experts) * sizeof(float);
+        const size_t smem = (RW * RT * RE + RT * (size_t)m.experts + m.experts) * sizeof(float);
         if (smem > 48 * 1024)
             MD_CUDA(ctx, cudaFuncSetAttribute(moe_router_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-        MD_TRY(md_launch_ex(ctx, moe_router_mma_kernel, dim3((unsigned)((rows + RT - 1) / RT)), dim3(256), smem, "moe_router_mma_kernel",
+        MD_TRY(md_launch_ex(ctx, moe_router_mma_kernel, dim3((unsigned)((rows + RT - 1) / RT)), dim3(RW * 32), smem, "moe_router_mma_kernel",
                             reinterpret_cast<const __nv_bfloat16*>(h), reinterpret_cast<const __nv_bfloat16*>(m.router), (int)rows,
                             m.width, m.experts, m.top, b.score, b.sel, b.rank, b.count));
     } else {

@@ -307,7 +307,8 @@ int md_stack_layers(md_text_model* m, md_text_request* const* reqs, size_t seqs,
     return MD_OK;
 }
 
-int md_stack_head(md_text_model* m, md_text_request* r0, size_t step_rows, const int* rows_dev, size_t n, float* logits) {
+int md_stack_head(md_text_model* m, md_text_request* r0, size_t step_rows, const int* rows_dev, size_t n, float* logits,
+                  unsigned long long* sampled, bool* keys) {
     md_ctx* ctx = m->ctx;
     const md_stack& s = *m->stack;
     md_stack_request* b = r0->stack;
@@ -329,7 +330,12 @@ int md_stack_head(md_text_model* m, md_text_request* r0, size_t step_rows, const
     MD_TRY(md_launch_glue(ctx, s.w.dtype, g));
     md_lin head;
     head.out_f32 = logits;
-    return md_linear(ctx, s.w.dtype, b->h.p, s.w.head, nullptr, n, s.w.vocab, s.w.width, head);
+    const bool fused = sampled && s.w.dtype == MD_DTYPE_BF16 && n <= 8 && md_gemv_lin_supported(b->h.p, s.w.head, s.w.width);
+    if (fused) head.amax = sampled;
+    MD_TRY(md_linear(ctx, s.w.dtype, b->h.p, s.w.head, nullptr, n, s.w.vocab, s.w.width, head));
+    if (sampled && !fused) MD_TRY(md_launch_argmax_f32(ctx, logits, s.w.vocab, s.w.vocab, n, sampled));
+    if (keys) *keys = fused;
+    return MD_OK;
 }
 
 int md_stack_copy_stream(md_text_request* req, size_t layer, float* out, size_t rows) {

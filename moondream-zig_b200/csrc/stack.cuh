@@ -22,6 +22,7 @@ struct md_lin {
     // glu != 0: W's rows are gate and up rows in alternating blocks of 32 (MD_GLU_BLOCK) and C[M, N/2] = act(gate) * up
     int glu = 0;                     // MD_ACT_*
     float* out_f32 = nullptr;        // write f32 sums here instead of T to C
+    unsigned long long* amax = nullptr;   // [M] running maximum of md_argmax_key over each row (bfloat16, M <= 8; zero before)
     // rows sorted by expert: row block b (128 rows) belongs to expert tile_expert[b], whose matrix is W + e * N * K;
     // only the first *n_blocks blocks are computed
     const int* tile_expert = nullptr;
@@ -34,6 +35,9 @@ int md_launch_gemm_tc_lin(md_ctx* ctx, const void* a, const void* b, void* c, si
 int md_launch_gemm_pair_lin(md_ctx* ctx, const void* a, const void* b, void* c, size_t M, size_t N, size_t K, const md_lin& lin);
 int md_launch_gemm_skinny_lin(md_ctx* ctx, const void* a, const void* b, void* c, size_t M, size_t N, size_t K, const md_lin& lin);
 int md_launch_gemv_lin(md_ctx* ctx, const void* a, const void* b, void* c, size_t M, size_t N, size_t K, const md_lin& lin);
+inline bool md_gemv_lin_supported(const void* a, const void* w, size_t K) {
+    return (K % 8) == 0 && ((reinterpret_cast<uintptr_t>(a) | reinterpret_cast<uintptr_t>(w)) & 15) == 0;
+}
 int md_make_map_2d_bf16(md_ctx* ctx, CUtensorMap* map, const void* ptr, uint64_t inner, uint64_t outer, uint32_t box_inner,
                         uint32_t box_outer, bool swizzle_64);
 int md_linear(md_ctx* ctx, int dtype, const void* a, const void* w, void* c, size_t M, size_t N, size_t K, const md_lin& ep);
@@ -130,6 +134,11 @@ int md_launch_moe(md_ctx* ctx, int dtype, const md_moe& m, const void* h, size_t
 int md_launch_argmax_f32(md_ctx* ctx, const float* x, size_t n, size_t stride, size_t rows, unsigned long long* idx_dev);
 
 #ifdef __CUDACC__
+// An order-preserving image of the value above the complement of the index: the largest key is the first largest value.
+__device__ __forceinline__ unsigned long long md_argmax_key(float v, uint32_t i) {
+    const uint32_t b = __float_as_uint(v);
+    return ((unsigned long long)((b & 0x80000000u) ? ~b : (b | 0x80000000u)) << 32) | (0xFFFFFFFFu - i);
+}
 template <class T> struct md_elem;
 template <> struct md_elem<__nv_bfloat16> {
     static __device__ __forceinline__ float get(__nv_bfloat16 v) { return __bfloat162float(v); }

@@ -1,6 +1,11 @@
 // What sits between the matrix products of a layer-stack decoder: residual update, RMS norms and the causal
 // convolution in one kernel (md_glue in stack.cuh states the arithmetic), the append of new keys to a cache, and the
 // greedy sample of f32 logits.  Everything is f32; only the row handed to the next product is rounded to T.
+//   stack_glue_step_kernel   one row per sequence (a decode step, or the final norm of a few rows): a thread keeps its
+//                            columns' inputs, weights and convolution state in registers, and all weights and the state are
+//                            requested before the dependency wait
+//   stack_glue_rows_kernel   rows of a prompt: a row per warp group, its inputs read once into registers
+//   stack_glue_any_kernel    widths that are not a multiple of 4 or too wide for the others
 #include "stack.cuh"
 
 namespace {
@@ -40,7 +45,7 @@ template <class T, int V> __device__ __forceinline__ void stv(T* p, const Vec<V>
 // it reads the old one before it recomputes the sequence's last taps - 1 rows and stores them.
 template <class T, int V, bool WIDE>
 __global__ void __launch_bounds__(WIDE ? 512 : 256)
-stack_glue_kernel(const __grid_constant__ md_glue p, int R) {
+stack_glue_any_kernel(const __grid_constant__ md_glue p, int R) {
     extern __shared__ __align__(16) float xs[];   // [R + halo][width]
     __shared__ float red[16];
     const int W = p.width, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -175,6 +180,305 @@ stack_glue_kernel(const __grid_constant__ md_glue p, int R) {
     for (int i = tid; i < halo * W; i += blockDim.x) state[i] = xs[(size_t)base * W + i];
 }
 
+constexpr int STEP_THREADS = 512;
+
+// sum over the threads of a block of `WARPS` warps; red holds 2 * WARPS floats, `turn` alternates between its halves
+template <int WARPS>
+__device__ __forceinline__ float block_sum(float v, float* red, int turn) {
+    v = warp_sum(v);
+    float* r = red + turn * WARPS;
+    if ((threadIdx.x & 31) == 0) r[threadIdx.x >> 5] = v;
+    __syncthreads();
+    v = 0.f;
+#pragma unroll
+    for (int i = 0; i < WARPS; ++i) v += r[i];
+    return v;
+}
+
+// block x = row; width % 4 == 0, width <= 2048 * NV, taps <= TAPS
+template <class T, int NV, int TAPS>
+__global__ void __launch_bounds__(STEP_THREADS)
+stack_glue_step_kernel(const __grid_constant__ md_glue p) {
+    __shared__ float red[2 * STEP_THREADS / 32];
+    const int W = p.width, tid = threadIdx.x, lane = tid & 31, row = blockIdx.x;
+    md_pdl_launch_dependents();
+    Vec<4> w_pre[NV], w_post[NV], conv[NV][TAPS], st[NV][TAPS - 1];
+    const int halo = p.conv ? p.taps - 1 : 0;
+    float* state = halo ? p.state[row] : nullptr;
+#pragma unroll
+    for (int n = 0; n < NV; ++n) {
+        const int c = (tid + n * STEP_THREADS) * 4;
+        if (c >= W) continue;
+        w_pre[n] = ldv<float, 4>(p.w_pre + c);
+        if (p.w_post) w_post[n] = ldv<float, 4>(p.w_post + c);
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j)
+            if (p.conv && j < p.taps) conv[n][j] = ldv<float, 4>(p.conv + (size_t)j * W + c);
+#pragma unroll
+        for (int j = 0; j < TAPS - 1; ++j)
+            if (j < halo) st[n][j] = ldv<float, 4>(state + (size_t)j * W + c);
+    }
+    md_pdl_wait();
+    const size_t src = p.gather ? (size_t)p.gather[row] : row;
+    Vec<4> x[NV], y[NV];
+    const T* xe = p.tokens ? reinterpret_cast<const T*>(p.embed) +
+                                 (size_t)(p.tokens[src] < (unsigned long long)p.vocab ? p.tokens[src] : 0ull) * W : nullptr;
+#pragma unroll
+    for (int n = 0; n < NV; ++n) {
+        const int c = (tid + n * STEP_THREADS) * 4;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) x[n].f[i] = y[n].f[i] = 0.f;
+        if (c >= W) continue;
+        x[n] = xe ? ldv<T, 4>(xe + c) : ldv<float, 4>(p.x + src * W + c);
+        if (p.w_post && !p.slot) y[n] = p.y_f32 ? ldv<float, 4>(p.y_f32 + src * W + c) : ldv<T, 4>(reinterpret_cast<const T*>(p.y) + src * W + c);
+    }
+    if (p.w_post) {
+        float scale = 1.f;
+        if (p.ssq) {
+            float s = 0.f;
+            for (int i = lane; i < p.ssq_parts; i += 32) s += __ldcg(p.ssq + src * p.ssq_parts + i);
+            scale = 1.f / sqrtf(warp_sum(s) / (float)p.ssq_n + p.eps);
+        }
+        if (p.slot)
+            for (int k = 0; k < p.top; ++k) {
+                const float s = p.score[src * p.top + k];
+                const T* e = reinterpret_cast<const T*>(p.y) + (size_t)p.slot[src * p.top + k] * W;
+#pragma unroll
+                for (int n = 0; n < NV; ++n) {
+                    const int c = (tid + n * STEP_THREADS) * 4;
+                    if (c >= W) continue;
+                    const Vec<4> v = ldv<T, 4>(e + c);
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) y[n].f[i] = fmaf(s, v.f[i], y[n].f[i]);
+                }
+            }
+        float ss = 0.f;
+#pragma unroll
+        for (int n = 0; n < NV; ++n) {
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                y[n].f[i] *= scale;
+                ss = fmaf(y[n].f[i], y[n].f[i], ss);
+            }
+        }
+        const float inv = p.mult / sqrtf(block_sum<STEP_THREADS / 32>(ss, red, 0) / (float)W + p.eps);
+#pragma unroll
+        for (int n = 0; n < NV; ++n) {
+            if ((tid + n * STEP_THREADS) * 4 >= W) continue;
+#pragma unroll
+            for (int i = 0; i < 4; ++i) x[n].f[i] = fmaf(y[n].f[i] * inv, w_post[n].f[i], x[n].f[i]);
+        }
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int n = 0; n < NV; ++n) {
+        const int c = (tid + n * STEP_THREADS) * 4;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) ss = fmaf(x[n].f[i], x[n].f[i], ss);
+        if (c < W && p.x_out) stv<float, 4>(p.x_out + (size_t)row * W + c, x[n]);
+    }
+    const float inv2 = 1.f / sqrtf(block_sum<STEP_THREADS / 32>(ss, red, 1) / (float)W + p.eps);
+#pragma unroll
+    for (int n = 0; n < NV; ++n) {
+        const int c = (tid + n * STEP_THREADS) * 4;
+        if (c >= W) continue;
+        Vec<4> v, o;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) o.f[i] = v.f[i] = x[n].f[i] * (inv2 * w_pre[n].f[i]);
+        if (p.conv) {
+            Vec<4> s;
+#pragma unroll
+            for (int i = 0; i < 4; ++i) s.f[i] = 0.f;
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) {
+                if (j >= p.taps) break;
+                const Vec<4>& in = j < halo ? st[n][j < TAPS - 1 ? j : 0] : v;
+#pragma unroll
+                for (int i = 0; i < 4; ++i) s.f[i] = fmaf(conv[n][j].f[i], in.f[i], s.f[i]);
+            }
+#pragma unroll
+            for (int i = 0; i < 4; ++i) o.f[i] += s.f[i];
+#pragma unroll
+            for (int j = 0; j < TAPS - 1; ++j) {
+                if (j >= halo) break;
+                stv<float, 4>(state + (size_t)j * W + c, j + 1 < halo ? st[n][j + 1 < TAPS - 1 ? j + 1 : 0] : v);
+            }
+        }
+        stv<T, 4>(reinterpret_cast<T*>(p.out) + (size_t)row * W + c, o);
+    }
+}
+
+// GW warps per row, NV vectors of 4 columns per lane: width <= 128 * GW * NV.  Eight warps; blocks, halo rows and state as
+// in stack_glue_any_kernel.
+template <class T, int GW, int NV>
+__global__ void __launch_bounds__(256, NV <= 8 ? 2 : 1)
+stack_glue_rows_kernel(const __grid_constant__ md_glue p, int R) {
+    extern __shared__ __align__(16) float xs[];   // [R + halo][width]
+    __shared__ float red[2][8];
+    constexpr int GROUPS = 8 / GW;
+    const int W = p.width, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int grp = warp / GW, gl = (warp % GW) * 32 + lane;    // this thread's place within its row
+    const int t0 = blockIdx.x * R, own = min(R, p.rows - t0), halo = p.conv ? p.taps - 1 : 0;
+    const bool first = blockIdx.x == 0;
+    md_pdl_launch_dependents();
+    md_pdl_wait();
+    auto total = [&](float v, int turn) {
+        v = warp_sum(v);
+        if (GW > 1) {
+            if (lane == 0) red[turn][warp] = v;
+            __syncthreads();
+            v = 0.f;
+#pragma unroll
+            for (int i = 0; i < GW; ++i) v += red[turn][grp * GW + i];
+        }
+        return v;
+    };
+    float* state = halo ? p.state[0] : nullptr;
+    if (first && halo)
+        for (int i = tid; i < halo * W; i += 256) xs[i] = state[i];
+    // pass 0: this block's rows (with those ahead of them); pass 1, first block of a longer sequence: its last rows again
+    for (int pass = 0; pass < 2; ++pass) {
+        int lo = first ? halo : 0, hi = halo + own, shift = t0 - halo;    // xs[l] = n[shift + l]
+        if (pass == 1) {
+            if (!first || !halo || p.rows <= own) break;
+            __syncthreads();
+            lo = 0, hi = halo, shift = p.rows - halo;
+        }
+        for (int l0 = lo; l0 < hi; l0 += GROUPS) {
+            const int l = l0 + grp, t = shift + l;
+            const bool live = l < hi;
+            Vec<4> x[NV], y[NV];
+#pragma unroll
+            for (int n = 0; n < NV; ++n) {
+#pragma unroll
+                for (int i = 0; i < 4; ++i) x[n].f[i] = y[n].f[i] = 0.f;
+            }
+            const size_t src = live ? (p.gather ? (size_t)p.gather[t] : t) : 0;
+            float scale = 1.f;
+            if (live) {
+                if (p.w_post && !p.slot) {
+                    const T* yr = reinterpret_cast<const T*>(p.y) + src * W;
+#pragma unroll
+                    for (int n = 0; n < NV; ++n) {
+                        const int c = (gl + n * 32 * GW) * 4;
+                        if (c < W) y[n] = p.y_f32 ? ldv<float, 4>(p.y_f32 + src * W + c) : ldv<T, 4>(yr + c);
+                    }
+                }
+                const T* xe = p.tokens ? reinterpret_cast<const T*>(p.embed) +
+                                             (size_t)(p.tokens[src] < (unsigned long long)p.vocab ? p.tokens[src] : 0ull) * W : nullptr;
+#pragma unroll
+                for (int n = 0; n < NV; ++n) {
+                    const int c = (gl + n * 32 * GW) * 4;
+                    if (c < W) x[n] = xe ? ldv<T, 4>(xe + c) : ldv<float, 4>(p.x + src * W + c);
+                }
+                if (p.w_post && p.ssq) {
+                    float s = 0.f;
+                    for (int i = lane; i < p.ssq_parts; i += 32) s += p.ssq[src * p.ssq_parts + i];
+                    scale = 1.f / sqrtf(warp_sum(s) / (float)p.ssq_n + p.eps);
+                }
+                if (p.w_post && p.slot)
+                    for (int k = 0; k < p.top; ++k) {
+                        const float s = p.score[src * p.top + k];
+                        const T* e = reinterpret_cast<const T*>(p.y) + (size_t)p.slot[src * p.top + k] * W;
+#pragma unroll
+                        for (int n = 0; n < NV; ++n) {
+                            const int c = (gl + n * 32 * GW) * 4;
+                            if (c >= W) continue;
+                            const Vec<4> v = ldv<T, 4>(e + c);
+#pragma unroll
+                            for (int i = 0; i < 4; ++i) y[n].f[i] = fmaf(s, v.f[i], y[n].f[i]);
+                        }
+                    }
+            }
+            if (p.w_post) {
+                float ss = 0.f;
+#pragma unroll
+                for (int n = 0; n < NV; ++n) {
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) {
+                        y[n].f[i] *= scale;
+                        ss = fmaf(y[n].f[i], y[n].f[i], ss);
+                    }
+                }
+                const float inv = p.mult / sqrtf(total(ss, 0) / (float)W + p.eps);
+#pragma unroll
+                for (int n = 0; n < NV; ++n) {
+                    const int c = (gl + n * 32 * GW) * 4;
+                    if (c >= W) continue;
+                    const Vec<4> w = ldv<float, 4>(p.w_post + c);
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) x[n].f[i] = fmaf(y[n].f[i] * inv, w.f[i], x[n].f[i]);
+                }
+            }
+            float ss = 0.f;
+            const bool store = live && pass == 0 && l >= halo && p.x_out;
+#pragma unroll
+            for (int n = 0; n < NV; ++n) {
+                const int c = (gl + n * 32 * GW) * 4;
+#pragma unroll
+                for (int i = 0; i < 4; ++i) ss = fmaf(x[n].f[i], x[n].f[i], ss);
+                if (store && c < W) stv<float, 4>(p.x_out + (size_t)t * W + c, x[n]);
+            }
+            const float inv2 = 1.f / sqrtf(total(ss, 1) / (float)W + p.eps);
+#pragma unroll
+            for (int n = 0; n < NV; ++n) {
+                const int c = (gl + n * 32 * GW) * 4;
+                if (!live || c >= W) continue;
+                const Vec<4> w = ldv<float, 4>(p.w_pre + c);
+                Vec<4> v;
+#pragma unroll
+                for (int i = 0; i < 4; ++i) v.f[i] = x[n].f[i] * (inv2 * w.f[i]);
+                stv<float, 4>(xs + (size_t)l * W + c, v);
+            }
+            if (GW > 1) __syncthreads();    // `red` is free for the next rows
+        }
+        __syncthreads();
+        if (pass == 0) {
+            T* out = reinterpret_cast<T*>(p.out) + (size_t)t0 * W;
+            const int per = W / 4;
+            for (int i = tid; i < per; i += 256) {       // a thread walks down the rows of its columns
+                const int c = i * 4;
+                Vec<4> w[4];
+                const bool short_conv = p.conv && p.taps <= 4;
+                if (short_conv) {
+#pragma unroll
+                    for (int j = 0; j < 4; ++j)
+                        if (j < p.taps) w[j] = ldv<float, 4>(p.conv + (size_t)j * W + c);
+                }
+                for (int r = 0; r < own; ++r) {
+                    Vec<4> v = lds<4>(xs + (size_t)(r + halo) * W + c);
+                    if (p.conv) {
+                        Vec<4> s;
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) s.f[e] = 0.f;
+                        if (short_conv) {
+#pragma unroll
+                            for (int j = 0; j < 4; ++j) {
+                                if (j >= p.taps) break;
+                                const Vec<4> n = lds<4>(xs + (size_t)(r + j) * W + c);
+#pragma unroll
+                                for (int e = 0; e < 4; ++e) s.f[e] = fmaf(w[j].f[e], n.f[e], s.f[e]);
+                            }
+                        } else {
+                            for (int j = 0; j < p.taps; ++j) {
+                                const Vec<4> n = lds<4>(xs + (size_t)(r + j) * W + c), cw = ldv<float, 4>(p.conv + (size_t)j * W + c);
+#pragma unroll
+                                for (int e = 0; e < 4; ++e) s.f[e] = fmaf(cw.f[e], n.f[e], s.f[e]);
+                            }
+                        }
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) v.f[e] += s.f[e];
+                    }
+                    stv<T, 4>(out + (size_t)r * W + c, v);
+                }
+            }
+        }
+    }
+    if (!first || !halo) return;
+    const int base = p.rows > own ? 0 : p.rows;    // see stack_glue_any_kernel
+    for (int i = tid; i < halo * W; i += 256) state[i] = xs[(size_t)base * W + i];
+}
+
 // rows of f32 logits -> index of the largest (the lowest index of equal ones)
 __global__ void __launch_bounds__(1024)
 argmax_f32_kernel(const float* __restrict__ x, size_t n, size_t stride, unsigned long long* __restrict__ out) {
@@ -182,12 +486,27 @@ argmax_f32_kernel(const float* __restrict__ x, size_t n, size_t stride, unsigned
     md_pdl_launch_dependents();
     md_pdl_wait();
     const float* xr = x + (size_t)blockIdx.x * stride;
-    unsigned long long best = 0ull;   // (order-preserving image of the value) << 32 | ~index
-    for (size_t i = threadIdx.x; i < n; i += blockDim.x) {
-        const uint32_t b = __float_as_uint(xr[i]);
-        const uint32_t o = (b & 0x80000000u) ? ~b : (b | 0x80000000u);
-        const unsigned long long key = ((unsigned long long)o << 32) | (0xFFFFFFFFull - i);
+    unsigned long long best = 0ull;
+    auto take = [&](float v, size_t i) {
+        const unsigned long long key = md_argmax_key(v, (uint32_t)i);
         best = key > best ? key : best;
+    };
+    if ((n % 4) == 0 && ((reinterpret_cast<uintptr_t>(xr)) & 15) == 0) {
+        const size_t nv = n / 4;
+        for (size_t i0 = threadIdx.x; i0 < nv; i0 += 8 * 1024) {
+            float4 v[8];
+#pragma unroll
+            for (int u = 0; u < 8; ++u)
+                if (i0 + u * 1024 < nv) v[u] = __ldcg(reinterpret_cast<const float4*>(xr) + i0 + u * 1024);
+#pragma unroll
+            for (int u = 0; u < 8; ++u) {
+                const size_t i = (i0 + u * 1024) * 4;
+                if (i >= n) continue;
+                take(v[u].x, i), take(v[u].y, i + 1), take(v[u].z, i + 2), take(v[u].w, i + 3);
+            }
+        }
+    } else {
+        for (size_t i = threadIdx.x; i < n; i += blockDim.x) take(xr[i], i);
     }
 #pragma unroll
     for (int o = 16; o; o >>= 1) {
@@ -205,8 +524,16 @@ argmax_f32_kernel(const float* __restrict__ x, size_t n, size_t stride, unsigned
 template <class T>
 int launch_glue(md_ctx* ctx, const md_glue& g) {
     const int halo = g.conv ? g.taps - 1 : 0;
-    const bool wide = g.rows == 1 || (g.gather && g.rows <= 8);
+    const bool v4 = (g.width % 4) == 0;
     const size_t row_bytes = (size_t)g.width * sizeof(float);
+    if (g.rows > 1 && g.seqs > 1) return md_fail(ctx, MD_ERR_UNSUPPORTED, "md_glue: several rows of several sequences");
+    if (v4 && g.width <= 8192 && g.taps <= 4 && (g.rows == 1 || (g.gather && g.rows <= 8))) {
+        const dim3 grid((unsigned)(g.rows * g.seqs));
+        if (g.width <= 2048) return md_launch_ex(ctx, stack_glue_step_kernel<T, 1, 4>, grid, dim3(STEP_THREADS), 0, "stack_glue_step_kernel", g);
+        if (g.width <= 4096) return md_launch_ex(ctx, stack_glue_step_kernel<T, 2, 4>, grid, dim3(STEP_THREADS), 0, "stack_glue_step_kernel", g);
+        return md_launch_ex(ctx, stack_glue_step_kernel<T, 4, 4>, grid, dim3(STEP_THREADS), 0, "stack_glue_step_kernel", g);
+    }
+    const bool wide = g.rows == 1 || (g.gather && g.rows <= 8);
     int R = wide ? 1 : 8 - halo;
     if (!wide && R < halo) R = halo;
     if (R < 1) R = 1;
@@ -214,9 +541,14 @@ int launch_glue(md_ctx* ctx, const md_glue& g) {
     const size_t smem = (R + halo) * row_bytes;
     if (smem > 220 * 1024) return md_fail(ctx, MD_ERR_UNSUPPORTED, "a width of %d with %d taps exceeds shared memory", g.width, g.taps);
     if (g.x && g.x == g.x_out && g.rows > R) return md_fail(ctx, MD_ERR_INVALID_ARG, "md_glue: in-place residual over several blocks");
-    const bool v4 = (g.width % 4) == 0;
-    auto kern = wide ? (v4 ? stack_glue_kernel<T, 4, true> : stack_glue_kernel<T, 1, true>)
-                     : (v4 ? stack_glue_kernel<T, 4, false> : stack_glue_kernel<T, 1, false>);
+    void (*kern)(md_glue, int) = nullptr;
+    if (v4 && !wide && g.width <= 16384)
+        kern = g.width <= 512 ? stack_glue_rows_kernel<T, 1, 4> : g.width <= 1024 ? stack_glue_rows_kernel<T, 1, 8>
+             : g.width <= 2048 ? stack_glue_rows_kernel<T, 2, 8> : g.width <= 4096 ? stack_glue_rows_kernel<T, 4, 8>
+             : g.width <= 8192 ? stack_glue_rows_kernel<T, 8, 8> : stack_glue_rows_kernel<T, 8, 16>;
+    else
+        kern = wide ? (v4 ? stack_glue_any_kernel<T, 4, true> : stack_glue_any_kernel<T, 1, true>)
+                    : (v4 ? stack_glue_any_kernel<T, 4, false> : stack_glue_any_kernel<T, 1, false>);
     if (smem > 47 * 1024) MD_CUDA(ctx, cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
     return md_launch_ex(ctx, kern, dim3((unsigned)((g.rows + R - 1) / R), (unsigned)g.seqs), dim3(wide ? 512 : 256), smem,
                         "stack_glue_kernel", g, R);

@@ -81,6 +81,8 @@ int md_stack_reserve(md_text_request* req, size_t rows);
 int md_stack_layers(md_text_model* m, md_text_request* const* reqs, size_t seqs, size_t rows,
                     const unsigned long long* tokens_dev, bool decode, size_t pos0);
 // Final norm and head over `n` of the `step_rows` rows md_stack_layers has run: rows_dev (device indices), or the first n.
-// logits f32 [n, vocab].
-int md_stack_head(md_text_model* m, md_text_request* r0, size_t step_rows, const int* rows_dev, size_t n, float* logits);
+// logits f32 [n, vocab].  sampled != null (n <= 8, zero before the call): the rows' greedy samples, as keys for
+// advance_kernel if the call returns with *keys set, as indices otherwise.
+int md_stack_head(md_text_model* m, md_text_request* r0, size_t step_rows, const int* rows_dev, size_t n, float* logits,
+                  unsigned long long* sampled, bool* keys);
 int md_stack_copy_stream(md_text_request* req, size_t layer, float* out, size_t rows);
