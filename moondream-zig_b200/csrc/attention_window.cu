@@ -265,7 +265,7 @@ window_prefill_kernel(const __grid_constant__ md_win_attn p) {
     }
 }
 
-constexpr int DEC_KEYS = 64, DEC_THREADS = 128, DEC_MAX_DIM = 256;
+constexpr int DEC_KEYS = 64, DEC_THREADS = 128, DEC_MAX_DIM = 256, DEC_MAX_GROUP = DEC_THREADS;
 
 // visible keys of a token at `pos`, in order: the kept ones ahead of the window, then the window's; `index` counts them
 __device__ __forceinline__ int visible_key(int index, int kept, int first) { return index < kept ? index : first + (index - kept); }
@@ -280,6 +280,7 @@ window_decode_kernel(const __grid_constant__ md_win_attn p, float* partial, unsi
     float* Ps = reinterpret_cast<float*>(Qs + 8 * pitch);             // [8][64]
     float* ms = Ps + 8 * DEC_KEYS;                                    // [4][8] maxima, then [4][8] sums
     __shared__ int last_s;
+    __shared__ float gates[DEC_MAX_GROUP], rs1[DEC_MAX_GROUP], rs2[DEC_MAX_GROUP];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
     const int split = blockIdx.x, kvh = blockIdx.y, seq = blockIdx.z;
     const int pos = *p.pos_dev[seq];   // written by the kernel that ended the previous step
@@ -300,6 +301,10 @@ window_decode_kernel(const __grid_constant__ md_win_attn p, float* partial, unsi
             *reinterpret_cast<uint4*>(Ks + r * pitch + c * 8) = make_uint4(0, 0, 0, 0);
     }
     cp_async_commit();
+    if (tid < R) {
+        rs1[tid] = p.r1[kvh * R + tid];
+        rs2[tid] = p.r2[kvh * R + tid];
+    }
     md_pdl_wait();
     const __nv_bfloat16* row = reinterpret_cast<const __nv_bfloat16*>(p.qkg) + (size_t)seq * p.row_stride;
     if (newest && tid < real) {
@@ -307,6 +312,7 @@ window_decode_kernel(const __grid_constant__ md_win_attn p, float* partial, unsi
         *reinterpret_cast<uint4*>(Ks + (n - 1) * pitch + tid * 8) = k;
         *reinterpret_cast<uint4*>(cache + (size_t)pos * dim + tid * 8) = k;
     }
+    if (tid < R) gates[tid] = __bfloat162float(row[(p.heads + p.kv_heads) * dim + kvh * R + tid]);
     const size_t slot = (size_t)seq * p.kv_heads + kvh;
     float* mine = partial + (slot * max_splits + split) * R * (dim + 2);
     for (int h0 = 0; h0 < R; h0 += 8) {
@@ -333,8 +339,8 @@ window_decode_kernel(const __grid_constant__ md_win_attn p, float* partial, unsi
             const int r = warp * 16 + g + (e >> 1) * 8, hh = 2 * t + (e & 1);
             float v = -INFINITY;
             if (r < n && hh < heads) {
-                const int h = kvh * R + h0 + hh, d = pos - visible_key(split * DEC_KEYS + r, kept, first);
-                v = (s[e] * p.scale - p.r1[h] * log1pf(p.r2[h] * (float)d)) * LOG2E;
+                const int h = h0 + hh, d = pos - visible_key(split * DEC_KEYS + r, kept, first);
+                v = (s[e] * p.scale - rs1[h] * log1pf(rs2[h] * (float)d)) * LOG2E;
             }
             s[e] = v;
             mx[e & 1] = fmaxf(mx[e & 1], v);
@@ -432,8 +438,7 @@ window_decode_kernel(const __grid_constant__ md_win_attn p, float* partial, unsi
             }
             m = mn;
         }
-        const float gate = __bfloat162float(row[(p.heads + p.kv_heads) * dim + h]);
-        reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)seq * p.heads * dim + h * dim + d] = __float2bfloat16_rn(o / l * gate);
+        reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)seq * p.heads * dim + h * dim + d] = __float2bfloat16_rn(o / l * gates[hh]);
     }
 }
 
@@ -490,7 +495,7 @@ int launch(md_ctx* ctx, const md_win_attn& a) {
 
 int md_launch_window_attention(md_ctx* ctx, int dtype, const md_win_attn& a, bool decode) {
     if (dtype == MD_DTYPE_BF16 && vector_ok(a)) {
-        if (decode && a.rows == 1) return launch_decode(ctx, a);
+        if (decode && a.rows == 1 && a.heads / a.kv_heads <= DEC_MAX_GROUP) return launch_decode(ctx, a);
         if (!decode && a.seqs == 1) return launch_prefill(ctx, a);
     }
     if (a.dim > 32 * PER_LANE) return md_fail(ctx, MD_ERR_UNSUPPORTED, "window attention: head size %d > %d", a.dim, 32 * PER_LANE);

@@ -374,12 +374,12 @@ lightning_carry_kernel(const __grid_constant__ md_lightning p, float* seg_state,
     if (i >= n) return;
     const float f = powf(p.decay[i / per], (float)seg_tokens);
     float S = p.state[0][i];
-    for (int s0 = 0; s0 < n_seg; s0 += 8) {     // eight contributions requested at a time
-        float u[8];
+    for (int s0 = 0; s0 < n_seg; s0 += 16) {     // sixteen contributions requested at a time
+        float u[16];
 #pragma unroll
-        for (int k = 0; k < 8; ++k) u[k] = s0 + k < n_seg - 1 ? seg_state[(s0 + k) * n + i] : 0.f;
+        for (int k = 0; k < 16; ++k) u[k] = s0 + k < n_seg - 1 ? seg_state[(s0 + k) * n + i] : 0.f;
 #pragma unroll
-        for (int k = 0; k < 8; ++k) {
+        for (int k = 0; k < 16; ++k) {
             if (s0 + k < n_seg) seg_state[(s0 + k) * n + i] = S;
             S = fmaf(f, S, u[k]);
         }

@@ -78,7 +78,11 @@ __global__ void copy_logits_kernel(const T* __restrict__ logits, T* __restrict__
 }
 
 __global__ void set_int_kernel(int* p, int v) { *p = v; }
-__global__ void add_int_kernel(int* p, int v) { *p += v; }
+// the end of a step over n tokens: position, and (a prompt's portion) the other copy of the convolution states is current
+__global__ void end_step_kernel(int* pos, int n) {
+    pos[0] += n;
+    if (n > 1) pos[1] ^= 1;
+}
 __global__ void widen_kernel(const __half* __restrict__ x, float* __restrict__ y, int n) {
     for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < n; i += gridDim.x * blockDim.x) y[i] = __half2float(x[i]);
 }
@@ -435,11 +439,11 @@ int md_text_request_create(md_text_model* model, md_text_request** out) {
         r->kc.push_back((__half*)k);
         r->vc.push_back((__half*)v);
     }
-    if (cudaMalloc((void**)&r->pos_dev, sizeof(int)) != cudaSuccess) {
+    if (cudaMalloc((void**)&r->pos_dev, 2 * sizeof(int)) != cudaSuccess) {
         md_text_request_destroy(r);
         return md_fail(ctx, MD_ERR_OOM, "request state allocation failed");
     }
-    cudaMemsetAsync(r->pos_dev, 0, sizeof(int), ctx->stream);
+    cudaMemsetAsync(r->pos_dev, 0, 2 * sizeof(int), ctx->stream);
     int st = model->stack ? r->logits.ensure(ctx, 8 * w.vocab * sizeof(float)) : ensure_rows(r, 8);
     if (st == MD_OK) st = r->cur_token.ensure(ctx, 8 * sizeof(unsigned long long));
     if (st == MD_OK) st = r->sampled.ensure(ctx, 8 * sizeof(unsigned long long));
@@ -470,7 +474,7 @@ int md_text_request_reset(md_text_request* req) {
     if (!req) return MD_ERR_INVALID_ARG;
     md_ctx* ctx = req->model->ctx;
     req->pos = 0;
-    MD_CUDA(ctx, cudaMemsetAsync(req->pos_dev, 0, sizeof(int), ctx->stream));
+    MD_CUDA(ctx, cudaMemsetAsync(req->pos_dev, 0, 2 * sizeof(int), ctx->stream));
     return req->stack ? md_stack_request_reset(req) : MD_OK;
 }
 
@@ -587,8 +591,8 @@ int md_text_step(md_text_model* model, md_text_request* req, const uint32_t* tok
             const LayerIO io = io_of(req);
             for (size_t l = 0; l < w.n_layers; ++l) MD_TRY(text_layer(model, l, io, n, n == 1, &req, pos0));
         }
-        add_int_kernel<<<1, 1, 0, ctx->stream>>>(req->pos_dev, (int)n);
-        MD_LAUNCH_CHECK(ctx, "add_int_kernel");
+        end_step_kernel<<<1, 1, 0, ctx->stream>>>(req->pos_dev, (int)n);
+        MD_LAUNCH_CHECK(ctx, "end_step_kernel");
         return MD_OK;
     };
     // a decoded token finds its position in device memory, so one recording serves every position

@@ -302,11 +302,14 @@ moe_up_kernel(const __nv_bfloat16* h, const __nv_bfloat16* __restrict__ w_gu, __
     const int slot = blockIdx.y, j = blockIdx.x * 8 + g;
     md_pdl_launch_dependents();
     md_pdl_wait();
-    if (slot >= __ldcg(r.n_slots)) return;
-    const __nv_bfloat16* w = w_gu + (size_t)__ldcg(r.expert + slot) * 2 * ff_pad * W;
+    // (the three small loads together; entries past n_slots are dropped right after)
+    const int n_slots = __ldcg(r.n_slots), expert = __ldcg(r.expert + slot);
+    const float mine = __ldcg(r.weight + slot * 8 + g);
+    if (slot >= n_slots) return;
+    const __nv_bfloat16* w = w_gu + (size_t)expert * 2 * ff_pad * W;
     const __nv_bfloat16* w_lo = w + (size_t)((j / MD_GLU_BLOCK) * (2 * MD_GLU_BLOCK) + j % MD_GLU_BLOCK) * W + t * 8;
     const __nv_bfloat16* w_hi = w_lo + (size_t)MD_GLU_BLOCK * W;
-    const bool has_x = g < T && __ldcg(r.weight + slot * 8 + g) != 0.f;
+    const bool has_x = g < T && mine != 0.f;
     const __nv_bfloat16* x = h + (size_t)(has_x ? g : 0) * W + t * 8;
     const uint4 zero = make_uint4(0, 0, 0, 0);
     float acc[4] = {0.f, 0.f, 0.f, 0.f};
@@ -344,20 +347,23 @@ moe_up_kernel(const __nv_bfloat16* h, const __nv_bfloat16* __restrict__ w_gu, __
 }
 
 // y[token][n] = sum over the slots' columns
-__global__ void __launch_bounds__(512)
+__global__ void __launch_bounds__(512, 2)
 moe_down_kernel(const __nv_bfloat16* act, const __nv_bfloat16* __restrict__ w_down, float* y, int T, int W, int ff_pad, int act_stride,
                 Route r) {
     __shared__ float partial[16][16][8];
+    __shared__ int list[MAX_EXPERTS];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
-    const int row0 = blockIdx.x * 16;
+    const int row0 = blockIdx.x * 16, per = ff_pad / 32;
     md_pdl_launch_dependents();
     md_pdl_wait();
-    const int per = ff_pad / 32, chunks = __ldcg(r.n_slots) * per;
+    const int n_slots = __ldcg(r.n_slots), chunks = n_slots * per;
+    if (tid < act_stride / ff_pad) list[tid] = __ldcg(r.expert + tid);   // what is past n_slots is not used
+    __syncthreads();
     const size_t r_lo = min(row0 + g, W - 1), r_hi = min(row0 + g + 8, W - 1);
     const __nv_bfloat16* x = act + (size_t)(g < T ? g : 0) * act_stride + t * 8;
     const uint4 zero = make_uint4(0, 0, 0, 0);
     float acc[4] = {0.f, 0.f, 0.f, 0.f};
-    constexpr int U = 6;
+    constexpr int U = 4;
     for (int c0 = warp; c0 < chunks; c0 += U * 16) {
         uint4 lo[U], hi[U], xv[U];
 #pragma unroll
@@ -366,7 +372,7 @@ moe_down_kernel(const __nv_bfloat16* act, const __nv_bfloat16* __restrict__ w_do
             lo[u] = hi[u] = xv[u] = zero;
             if (c < chunks) {
                 const int slot = c / per, k = (c - slot * per) * 32 + t * 8;
-                const __nv_bfloat16* w = w_down + (size_t)__ldcg(r.expert + slot) * W * ff_pad + k;
+                const __nv_bfloat16* w = w_down + (size_t)list[slot] * W * ff_pad + k;
                 lo[u] = ldg_stream(w + r_lo * ff_pad);
                 hi[u] = ldg_stream(w + r_hi * ff_pad);
                 if (g < T) xv[u] = ld_act(x + c * 32);

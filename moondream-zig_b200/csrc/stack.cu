@@ -112,9 +112,9 @@ extern "C" int md_stack_model_create(md_ctx* ctx, const md_stack_weights* w, md_
         s.rec_off.push_back(s.state_floats);
         if (!attn) s.state_floats += align_up(l.heads * l.dim * l.vdim, 64);
         s.conv1_off.push_back(s.state_floats);
-        s.state_floats += align_up((w->taps - 1) * w->width, 64);
+        s.state_floats += align_up(2 * (w->taps - 1) * w->width, 64);
         s.conv2_off.push_back(s.state_floats);
-        if (l.ff != MD_FF_NONE) s.state_floats += align_up((w->taps - 1) * w->width, 64);
+        if (l.ff != MD_FF_NONE) s.state_floats += align_up(2 * (w->taps - 1) * w->width, 64);
         s.max_in = std::max(s.max_in, l.in_rows);
         s.max_o = std::max(s.max_o, l.heads * l.vdim);
         if (!attn) s.max_ssq = std::max(s.max_ssq, (size_t)md_lightning_ssq_parts((int)l.heads, (int)l.vdim));
@@ -226,7 +226,10 @@ int md_stack_layers(md_text_model* m, md_text_request* const* reqs, size_t seqs,
         cur ^= 1;
         g.w_pre = w_pre;
         g.conv = conv;
-        for (size_t i = 0; i < seqs; ++i) g.state[i] = reqs[i]->stack->state.as<float>() + off[layer];
+        for (size_t i = 0; i < seqs; ++i) {
+            g.state[i] = reqs[i]->stack->state.as<float>() + off[layer];
+            g.state_slot[i] = reqs[i]->pos_dev + 1;
+        }
         g.out = b->h.p;
         return md_launch_glue(ctx, dt, g);
     };

@@ -47,7 +47,10 @@ int md_linear(md_ctx* ctx, int dtype, const void* a, const void* w, void* c, siz
 //   x_out[t] = x[t] + mult * rms_norm(y[t]; w_post)             (y == null: x_out = x; tokens != null: x = embed[token])
 //   n[t]     = rms_norm(x_out[t]; w_pre)
 //   out[t]   = n[t] + sum_j conv[j] * n[t - taps + 1 + j]       (conv == null: out = n)
-// The convolution's last taps - 1 inputs live in `state` ([taps - 1][width] f32) between calls.
+// The convolution's last taps - 1 inputs live in `state` between calls: two copies of [taps - 1][width] f32, of which
+// *state_slot (device memory) names the current one.  A decode step (rows == 1) updates it in place; a prompt's portion
+// reads it and writes the other one, since different blocks read the start and write the end, and whoever ends the step
+// flips *state_slot.
 struct md_glue {
     int width = 0, rows = 0, taps = 0;      // rows per sequence
     float eps = 0.f, mult = 0.f;
@@ -64,7 +67,7 @@ struct md_glue {
     const float* ssq = nullptr;             // [rows, ssq_parts]
     int ssq_parts = 0, ssq_n = 0;
     // mixture of experts: y of row t = sum_k score[t][k] * y[slot[t][k]]
-    const int* slot = nullptr;              // [rows, top]
+    const int* slot = nullptr;              // [rows, top]: place in the sorted rows
     const float* score = nullptr;
     int top = 0;
     const float* w_pre = nullptr;
@@ -73,6 +76,7 @@ struct md_glue {
     const int* gather = nullptr;            // rows to take (final norm of the wanted rows): x row = gather[i], no x_out
     int seqs = 1;
     float* state[MD_STACK_MAX_SEQS] = {};
+    const int* state_slot[MD_STACK_MAX_SEQS] = {};
 };
 int md_launch_glue(md_ctx* ctx, int dtype, const md_glue& g);
 

@@ -16,6 +16,8 @@ __device__ __forceinline__ float warp_sum(float v) {
     return v;
 }
 
+__device__ __forceinline__ void prefetch_l2(const void* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
+
 template <int V> struct Vec { float f[V]; };
 template <class T, int V> __device__ __forceinline__ Vec<V> ldv(const T* p) {
     Vec<V> r;
@@ -41,8 +43,8 @@ template <class T, int V> __device__ __forceinline__ void stv(T* p, const Vec<V>
 
 // WIDE: all warps of the block work on one row at a time (a decode step has one row per sequence); otherwise one warp
 // per row and as many rows as warps at once.  A block owns `R` rows of a sequence and recomputes the taps - 1 rows ahead
-// of them; the first block of a sequence takes those from the state instead, and is the only one that touches the state:
-// it reads the old one before it recomputes the sequence's last taps - 1 rows and stores them.
+// of them; the first block of a sequence takes those from the state instead, and the last one, which then holds the
+// sequence's last taps - 1 values of n (with older ones from the state if the sequence is that short), stores them.
 template <class T, int V, bool WIDE>
 __global__ void __launch_bounds__(WIDE ? 512 : 256)
 stack_glue_any_kernel(const __grid_constant__ md_glue p, int R) {
@@ -134,9 +136,10 @@ stack_glue_any_kernel(const __grid_constant__ md_glue p, int R) {
         }
     };
 
+    const int slot = halo ? *p.state_slot[seq] : 0;
     float* state = halo ? p.state[seq] : nullptr;
     if (first && halo)
-        for (int i = tid; i < halo * W; i += blockDim.x) xs[i] = state[i];
+        for (int i = tid; i < halo * W; i += blockDim.x) xs[i] = state[slot * halo * W + i];
     const int lo = first ? halo : 0;
     if (WIDE) {
         for (int l = lo; l < halo + own; ++l) row(l, t0 - halo + l, l >= halo);
@@ -163,21 +166,9 @@ stack_glue_any_kernel(const __grid_constant__ md_glue p, int R) {
         }
         stv<T, V>(out + (size_t)r * W + c, v);
     }
-    if (!first || !halo) return;
-    // the sequence's last taps - 1 values of n: in xs if this block holds the whole sequence (older ones are the old
-    // state, which sits in xs[0 .. halo) ), otherwise recomputed
-    int base = p.rows;
-    if (p.rows > own) {
-        __syncthreads();
-        if (WIDE) {
-            for (int l = 0; l < halo; ++l) row(l, p.rows - halo + l, false);
-        } else {
-            for (int l = warp; l < halo; l += 8) row(l, p.rows - halo + l, false);
-        }
-        base = 0;
-        __syncthreads();
-    }
-    for (int i = tid; i < halo * W; i += blockDim.x) state[i] = xs[(size_t)base * W + i];
+    if (blockIdx.x + 1 < gridDim.x || !halo) return;
+    float* dst = state + (size_t)(p.rows == 1 ? slot : slot ^ 1) * halo * W;
+    for (int i = tid; i < halo * W; i += blockDim.x) dst[i] = xs[(size_t)own * W + i];
 }
 
 constexpr int STEP_THREADS = 512;
@@ -204,7 +195,7 @@ stack_glue_step_kernel(const __grid_constant__ md_glue p) {
     md_pdl_launch_dependents();
     Vec<4> w_pre[NV], w_post[NV], conv[NV][TAPS], st[NV][TAPS - 1];
     const int halo = p.conv ? p.taps - 1 : 0;
-    float* state = halo ? p.state[row] : nullptr;
+    float* state = halo ? p.state[row] + (size_t)*p.state_slot[row] * halo * W : nullptr;
 #pragma unroll
     for (int n = 0; n < NV; ++n) {
         const int c = (tid + n * STEP_THREADS) * 4;
@@ -308,19 +299,27 @@ stack_glue_step_kernel(const __grid_constant__ md_glue p) {
     }
 }
 
-// GW warps per row, NV vectors of 4 columns per lane: width <= 128 * GW * NV.  Eight warps; blocks, halo rows and state as
+constexpr int ROWS_THREADS = 512;
+
+// GW warps per row, NV vectors of 4 columns per lane: width <= 128 * GW * NV.  Sixteen warps; blocks, halo rows and state as
 // in stack_glue_any_kernel.
 template <class T, int GW, int NV>
-__global__ void __launch_bounds__(256, NV <= 8 ? 2 : 1)
+__global__ void __launch_bounds__(ROWS_THREADS, NV <= 4 ? 2 : 1)
 stack_glue_rows_kernel(const __grid_constant__ md_glue p, int R) {
     extern __shared__ __align__(16) float xs[];   // [R + halo][width]
-    __shared__ float red[2][8];
-    constexpr int GROUPS = 8 / GW;
+    __shared__ float red[2][ROWS_THREADS / 32];
+    constexpr int GROUPS = ROWS_THREADS / 32 / GW;
     const int W = p.width, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int grp = warp / GW, gl = (warp % GW) * 32 + lane;    // this thread's place within its row
     const int t0 = blockIdx.x * R, own = min(R, p.rows - t0), halo = p.conv ? p.taps - 1 : 0;
     const bool first = blockIdx.x == 0;
     md_pdl_launch_dependents();
+    // the weights come from HBM once per pass over the model: on their way to L2 before the wait
+    for (int i = tid * 32; i < W; i += ROWS_THREADS * 32) {
+        prefetch_l2(p.w_pre + i);
+        if (p.w_post) prefetch_l2(p.w_post + i);
+        for (int j = 0; p.conv && j < p.taps; ++j) prefetch_l2(p.conv + (size_t)j * W + i);
+    }
     md_pdl_wait();
     auto total = [&](float v, int turn) {
         v = warp_sum(v);
@@ -333,150 +332,123 @@ stack_glue_rows_kernel(const __grid_constant__ md_glue p, int R) {
         }
         return v;
     };
+    const int slot = halo ? *p.state_slot[0] : 0;
     float* state = halo ? p.state[0] : nullptr;
     if (first && halo)
-        for (int i = tid; i < halo * W; i += 256) xs[i] = state[i];
-    // pass 0: this block's rows (with those ahead of them); pass 1, first block of a longer sequence: its last rows again
-    for (int pass = 0; pass < 2; ++pass) {
-        int lo = first ? halo : 0, hi = halo + own, shift = t0 - halo;    // xs[l] = n[shift + l]
-        if (pass == 1) {
-            if (!first || !halo || p.rows <= own) break;
-            __syncthreads();
-            lo = 0, hi = halo, shift = p.rows - halo;
+        for (int i = tid; i < halo * W; i += ROWS_THREADS) xs[i] = state[slot * halo * W + i];
+    const int lo = first ? halo : 0, hi = halo + own;      // xs[l] = n[t0 - halo + l]
+    for (int l0 = lo; l0 < hi; l0 += GROUPS) {
+        const int l = l0 + grp, t = t0 - halo + l;
+        const bool live = l < hi;
+        Vec<4> x[NV], y[NV];
+#pragma unroll
+        for (int n = 0; n < NV; ++n) {
+#pragma unroll
+            for (int i = 0; i < 4; ++i) x[n].f[i] = y[n].f[i] = 0.f;
         }
-        for (int l0 = lo; l0 < hi; l0 += GROUPS) {
-            const int l = l0 + grp, t = shift + l;
-            const bool live = l < hi;
-            Vec<4> x[NV], y[NV];
+        const size_t src = live ? (p.gather ? (size_t)p.gather[t] : t) : 0;
+        float scale = 1.f;
+        if (live) {
+            if (p.w_post && !p.slot) {
+                const T* yr = reinterpret_cast<const T*>(p.y) + src * W;
+#pragma unroll
+                for (int n = 0; n < NV; ++n) {
+                    const int c = (gl + n * 32 * GW) * 4;
+                    if (c < W) y[n] = p.y_f32 ? ldv<float, 4>(p.y_f32 + src * W + c) : ldv<T, 4>(yr + c);
+                }
+            }
+            const T* xe = p.tokens ? reinterpret_cast<const T*>(p.embed) +
+                                         (size_t)(p.tokens[src] < (unsigned long long)p.vocab ? p.tokens[src] : 0ull) * W : nullptr;
 #pragma unroll
             for (int n = 0; n < NV; ++n) {
-#pragma unroll
-                for (int i = 0; i < 4; ++i) x[n].f[i] = y[n].f[i] = 0.f;
+                const int c = (gl + n * 32 * GW) * 4;
+                if (c < W) x[n] = xe ? ldv<T, 4>(xe + c) : ldv<float, 4>(p.x + src * W + c);
             }
-            const size_t src = live ? (p.gather ? (size_t)p.gather[t] : t) : 0;
-            float scale = 1.f;
-            if (live) {
-                if (p.w_post && !p.slot) {
-                    const T* yr = reinterpret_cast<const T*>(p.y) + src * W;
+            if (p.w_post && p.ssq) {
+                float s = 0.f;
+                for (int i = lane; i < p.ssq_parts; i += 32) s += p.ssq[src * p.ssq_parts + i];
+                scale = 1.f / sqrtf(warp_sum(s) / (float)p.ssq_n + p.eps);
+            }
+            if (p.w_post && p.slot)
+                for (int k = 0; k < p.top; ++k) {
+                    const float s = p.score[src * p.top + k];
+                    const T* e = reinterpret_cast<const T*>(p.y) + (size_t)p.slot[src * p.top + k] * W;
 #pragma unroll
                     for (int n = 0; n < NV; ++n) {
                         const int c = (gl + n * 32 * GW) * 4;
-                        if (c < W) y[n] = p.y_f32 ? ldv<float, 4>(p.y_f32 + src * W + c) : ldv<T, 4>(yr + c);
+                        if (c >= W) continue;
+                        const Vec<4> v = ldv<T, 4>(e + c);
+#pragma unroll
+                        for (int i = 0; i < 4; ++i) y[n].f[i] = fmaf(s, v.f[i], y[n].f[i]);
                     }
                 }
-                const T* xe = p.tokens ? reinterpret_cast<const T*>(p.embed) +
-                                             (size_t)(p.tokens[src] < (unsigned long long)p.vocab ? p.tokens[src] : 0ull) * W : nullptr;
-#pragma unroll
-                for (int n = 0; n < NV; ++n) {
-                    const int c = (gl + n * 32 * GW) * 4;
-                    if (c < W) x[n] = xe ? ldv<T, 4>(xe + c) : ldv<float, 4>(p.x + src * W + c);
-                }
-                if (p.w_post && p.ssq) {
-                    float s = 0.f;
-                    for (int i = lane; i < p.ssq_parts; i += 32) s += p.ssq[src * p.ssq_parts + i];
-                    scale = 1.f / sqrtf(warp_sum(s) / (float)p.ssq_n + p.eps);
-                }
-                if (p.w_post && p.slot)
-                    for (int k = 0; k < p.top; ++k) {
-                        const float s = p.score[src * p.top + k];
-                        const T* e = reinterpret_cast<const T*>(p.y) + (size_t)p.slot[src * p.top + k] * W;
-#pragma unroll
-                        for (int n = 0; n < NV; ++n) {
-                            const int c = (gl + n * 32 * GW) * 4;
-                            if (c >= W) continue;
-                            const Vec<4> v = ldv<T, 4>(e + c);
-#pragma unroll
-                            for (int i = 0; i < 4; ++i) y[n].f[i] = fmaf(s, v.f[i], y[n].f[i]);
-                        }
-                    }
-            }
-            if (p.w_post) {
-                float ss = 0.f;
-#pragma unroll
-                for (int n = 0; n < NV; ++n) {
-#pragma unroll
-                    for (int i = 0; i < 4; ++i) {
-                        y[n].f[i] *= scale;
-                        ss = fmaf(y[n].f[i], y[n].f[i], ss);
-                    }
-                }
-                const float inv = p.mult / sqrtf(total(ss, 0) / (float)W + p.eps);
-#pragma unroll
-                for (int n = 0; n < NV; ++n) {
-                    const int c = (gl + n * 32 * GW) * 4;
-                    if (c >= W) continue;
-                    const Vec<4> w = ldv<float, 4>(p.w_post + c);
-#pragma unroll
-                    for (int i = 0; i < 4; ++i) x[n].f[i] = fmaf(y[n].f[i] * inv, w.f[i], x[n].f[i]);
-                }
-            }
+        }
+        if (p.w_post) {
             float ss = 0.f;
-            const bool store = live && pass == 0 && l >= halo && p.x_out;
+#pragma unroll
+            for (int n = 0; n < NV; ++n) {
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    y[n].f[i] *= scale;
+                    ss = fmaf(y[n].f[i], y[n].f[i], ss);
+                }
+            }
+            const float inv = p.mult / sqrtf(total(ss, 0) / (float)W + p.eps);
 #pragma unroll
             for (int n = 0; n < NV; ++n) {
                 const int c = (gl + n * 32 * GW) * 4;
+                if (c >= W) continue;
+                const Vec<4> w = ldv<float, 4>(p.w_post + c);
 #pragma unroll
-                for (int i = 0; i < 4; ++i) ss = fmaf(x[n].f[i], x[n].f[i], ss);
-                if (store && c < W) stv<float, 4>(p.x_out + (size_t)t * W + c, x[n]);
-            }
-            const float inv2 = 1.f / sqrtf(total(ss, 1) / (float)W + p.eps);
-#pragma unroll
-            for (int n = 0; n < NV; ++n) {
-                const int c = (gl + n * 32 * GW) * 4;
-                if (!live || c >= W) continue;
-                const Vec<4> w = ldv<float, 4>(p.w_pre + c);
-                Vec<4> v;
-#pragma unroll
-                for (int i = 0; i < 4; ++i) v.f[i] = x[n].f[i] * (inv2 * w.f[i]);
-                stv<float, 4>(xs + (size_t)l * W + c, v);
-            }
-            if (GW > 1) __syncthreads();    // `red` is free for the next rows
-        }
-        __syncthreads();
-        if (pass == 0) {
-            T* out = reinterpret_cast<T*>(p.out) + (size_t)t0 * W;
-            const int per = W / 4;
-            for (int i = tid; i < per; i += 256) {       // a thread walks down the rows of its columns
-                const int c = i * 4;
-                Vec<4> w[4];
-                const bool short_conv = p.conv && p.taps <= 4;
-                if (short_conv) {
-#pragma unroll
-                    for (int j = 0; j < 4; ++j)
-                        if (j < p.taps) w[j] = ldv<float, 4>(p.conv + (size_t)j * W + c);
-                }
-                for (int r = 0; r < own; ++r) {
-                    Vec<4> v = lds<4>(xs + (size_t)(r + halo) * W + c);
-                    if (p.conv) {
-                        Vec<4> s;
-#pragma unroll
-                        for (int e = 0; e < 4; ++e) s.f[e] = 0.f;
-                        if (short_conv) {
-#pragma unroll
-                            for (int j = 0; j < 4; ++j) {
-                                if (j >= p.taps) break;
-                                const Vec<4> n = lds<4>(xs + (size_t)(r + j) * W + c);
-#pragma unroll
-                                for (int e = 0; e < 4; ++e) s.f[e] = fmaf(w[j].f[e], n.f[e], s.f[e]);
-                            }
-                        } else {
-                            for (int j = 0; j < p.taps; ++j) {
-                                const Vec<4> n = lds<4>(xs + (size_t)(r + j) * W + c), cw = ldv<float, 4>(p.conv + (size_t)j * W + c);
-#pragma unroll
-                                for (int e = 0; e < 4; ++e) s.f[e] = fmaf(cw.f[e], n.f[e], s.f[e]);
-                            }
-                        }
-#pragma unroll
-                        for (int e = 0; e < 4; ++e) v.f[e] += s.f[e];
-                    }
-                    stv<T, 4>(out + (size_t)r * W + c, v);
-                }
+                for (int i = 0; i < 4; ++i) x[n].f[i] = fmaf(y[n].f[i] * inv, w.f[i], x[n].f[i]);
             }
         }
+        float ss = 0.f;
+        const bool store = live && l >= halo && p.x_out;
+#pragma unroll
+        for (int n = 0; n < NV; ++n) {
+            const int c = (gl + n * 32 * GW) * 4;
+#pragma unroll
+            for (int i = 0; i < 4; ++i) ss = fmaf(x[n].f[i], x[n].f[i], ss);
+            if (store && c < W) stv<float, 4>(p.x_out + (size_t)t * W + c, x[n]);
+        }
+        const float inv2 = 1.f / sqrtf(total(ss, 1) / (float)W + p.eps);
+#pragma unroll
+        for (int n = 0; n < NV; ++n) {
+            const int c = (gl + n * 32 * GW) * 4;
+            if (!live || c >= W) continue;
+            const Vec<4> w = ldv<float, 4>(p.w_pre + c);
+            Vec<4> v;
+#pragma unroll
+            for (int i = 0; i < 4; ++i) v.f[i] = x[n].f[i] * (inv2 * w.f[i]);
+            stv<float, 4>(xs + (size_t)l * W + c, v);
+        }
+        if (GW > 1) __syncthreads();    // `red` is free for the next rows
     }
-    if (!first || !halo) return;
-    const int base = p.rows > own ? 0 : p.rows;    // see stack_glue_any_kernel
-    for (int i = tid; i < halo * W; i += 256) state[i] = xs[(size_t)base * W + i];
+    __syncthreads();
+    T* out = reinterpret_cast<T*>(p.out) + (size_t)t0 * W;
+    const int per = W / 4;
+    for (int i = tid; i < own * per; i += ROWS_THREADS) {
+        const int r = i / per, c = (i - r * per) * 4;
+        Vec<4> v = lds<4>(xs + (size_t)(r + halo) * W + c);
+        if (p.conv) {
+            Vec<4> s;
+#pragma unroll
+            for (int e = 0; e < 4; ++e) s.f[e] = 0.f;
+#pragma unroll 4
+            for (int j = 0; j < p.taps; ++j) {
+                const Vec<4> n = lds<4>(xs + (size_t)(r + j) * W + c), w = ldv<float, 4>(p.conv + (size_t)j * W + c);
+#pragma unroll
+                for (int e = 0; e < 4; ++e) s.f[e] = fmaf(w.f[e], n.f[e], s.f[e]);
+            }
+#pragma unroll
+            for (int e = 0; e < 4; ++e) v.f[e] += s.f[e];
+        }
+        stv<T, 4>(out + (size_t)r * W + c, v);
+    }
+    if (blockIdx.x + 1 < gridDim.x || !halo) return;
+    float* dst = state + (size_t)(p.rows == 1 ? slot : slot ^ 1) * halo * W;
+    for (int i = tid; i < halo * W; i += ROWS_THREADS) dst[i] = xs[(size_t)own * W + i];
 }
 
 // rows of f32 logits -> index of the largest (the lowest index of equal ones)
@@ -537,20 +509,22 @@ int launch_glue(md_ctx* ctx, const md_glue& g) {
     int R = wide ? 1 : 8 - halo;
     if (!wide && R < halo) R = halo;
     if (R < 1) R = 1;
-    while (!wide && R > halo && R > 1 && (R + halo) * row_bytes > 100 * 1024) --R;   // two blocks per SM where possible
+    while (!wide && R > halo && R > 1 && (R + halo) * row_bytes > 112 * 1024) --R;   // two blocks per SM where possible
     const size_t smem = (R + halo) * row_bytes;
     if (smem > 220 * 1024) return md_fail(ctx, MD_ERR_UNSUPPORTED, "a width of %d with %d taps exceeds shared memory", g.width, g.taps);
     if (g.x && g.x == g.x_out && g.rows > R) return md_fail(ctx, MD_ERR_INVALID_ARG, "md_glue: in-place residual over several blocks");
     void (*kern)(md_glue, int) = nullptr;
-    if (v4 && !wide && g.width <= 16384)
-        kern = g.width <= 512 ? stack_glue_rows_kernel<T, 1, 4> : g.width <= 1024 ? stack_glue_rows_kernel<T, 1, 8>
-             : g.width <= 2048 ? stack_glue_rows_kernel<T, 2, 8> : g.width <= 4096 ? stack_glue_rows_kernel<T, 4, 8>
-             : g.width <= 8192 ? stack_glue_rows_kernel<T, 8, 8> : stack_glue_rows_kernel<T, 8, 16>;
+    const bool rows_form = v4 && !wide && g.width <= 16384;
+    const unsigned threads = wide ? 512 : rows_form ? ROWS_THREADS : 256;
+    if (rows_form)
+        kern = g.width <= 512 ? stack_glue_rows_kernel<T, 1, 4> : g.width <= 1024 ? stack_glue_rows_kernel<T, 2, 4>
+             : g.width <= 2048 ? stack_glue_rows_kernel<T, 4, 4> : g.width <= 4096 ? stack_glue_rows_kernel<T, 8, 4>
+             : g.width <= 8192 ? stack_glue_rows_kernel<T, 16, 4> : stack_glue_rows_kernel<T, 16, 8>;
     else
         kern = wide ? (v4 ? stack_glue_any_kernel<T, 4, true> : stack_glue_any_kernel<T, 1, true>)
                     : (v4 ? stack_glue_any_kernel<T, 4, false> : stack_glue_any_kernel<T, 1, false>);
     if (smem > 47 * 1024) MD_CUDA(ctx, cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
-    return md_launch_ex(ctx, kern, dim3((unsigned)((g.rows + R - 1) / R), (unsigned)g.seqs), dim3(wide ? 512 : 256), smem,
+    return md_launch_ex(ctx, kern, dim3((unsigned)((g.rows + R - 1) / R), (unsigned)g.seqs), dim3(threads), smem,
                         "stack_glue_kernel", g, R);
 }
 

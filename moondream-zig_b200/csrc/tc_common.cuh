@@ -251,7 +251,13 @@ __device__ __forceinline__ void lin_glue8(const uint32_t* acc_bits, const md_lin
             v[0] += a.x; v[1] += a.y; v[2] += a.z; v[3] += a.w;
             v[4] += b.x; v[5] += b.y; v[6] += b.z; v[7] += b.w;
         }
-        if (cq < ep.silu_cols || cq + 8 > ep.sigmoid_from) {
+        if (cq + 8 <= ep.silu_cols) {
+#pragma unroll
+            for (int j = 0; j < 8; ++j) v[j] = fast_silu(v[j]);
+        } else if (cq >= ep.sigmoid_from) {
+#pragma unroll
+            for (int j = 0; j < 8; ++j) v[j] = fast_logistic(v[j]);
+        } else if (cq < ep.silu_cols || cq + 8 > ep.sigmoid_from) {   // a group that a boundary cuts
 #pragma unroll
             for (int j = 0; j < 8; ++j) {
                 const bool si = cq + j < ep.silu_cols, sg = cq + j >= ep.sigmoid_from;

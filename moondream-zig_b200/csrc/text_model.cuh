@@ -44,7 +44,7 @@ struct md_text_request {
     std::vector<__half*> kc, vc;  // per layer [n_heads][max_seq][head_dim]
     md_stack_request* stack = nullptr;
     size_t pos = 0;               // host mirror of *pos_dev
-    int* pos_dev = nullptr;
+    int* pos_dev = nullptr;       // [0] tokens held, [1] current copy of the convolution states (layer-stack models)
     // activations of one forward over `rows` rows
     DevPtr hidden, ln, qkv, attn, attn_out, fc1, logits, ln_last;
     DevPtr mlp_part;  // up to four f32 [8, dim] partial products of fc2 (the decode layer whose MLP runs as two half-width chains)
