@@ -91,6 +91,13 @@ window_attention_kernel(const __grid_constant__ md_win_attn p) {
 constexpr float LOG2E = 1.4426950408889634f;
 constexpr int BQ = 64, BK = 64;
 
+// 2^x by the hardware instruction (relative error about 2^-22), without exp2f's care for denormal results
+__device__ __forceinline__ float ex2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
 // keys (8 values per thread) into the cache
 __global__ void __launch_bounds__(256)
 append_keys_vec_kernel(const __grid_constant__ md_win_attn p) {
@@ -107,7 +114,7 @@ append_keys_vec_kernel(const __grid_constant__ md_win_attn p) {
 
 // DP: head size rounded up to a multiple of 16 (the pad is zero in shared memory)
 template <int DP>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(128, DP <= 64 ? 4 : DP <= 96 ? 3 : DP <= 128 ? 2 : 1)
 window_prefill_kernel(const __grid_constant__ md_win_attn p) {
     using namespace mb;
     constexpr int PITCH = DP + 8, CH = DP / 8;
@@ -160,13 +167,9 @@ window_prefill_kernel(const __grid_constant__ md_win_attn p) {
 
     for (int it = 0; it < n_tiles; ++it) {
         const int k0 = tile_key(it), buf = it & 1;
-        if (it + 1 < n_tiles) {
-            load_tile(it + 1);
-            cp_async_wait<1>();
-        } else {
-            cp_async_wait<0>();
-        }
-        __syncthreads();
+        cp_async_wait<0>();
+        __syncthreads();                              // tile `it` is there, and nobody reads the other buffer any more
+        if (it + 1 < n_tiles) load_tile(it + 1);      // in flight while this tile is worked on
         if (Q_REGS && it == 0) {
 #pragma unroll
             for (int ks = 0; ks < DP / 16; ++ks) ldsm_x4(smem_u32(Qs + q_row * PITCH + ks * 16 + q_col), qf[Q_REGS ? ks : 0]);
@@ -211,14 +214,14 @@ window_prefill_kernel(const __grid_constant__ md_win_attn p) {
             mx[rr] = fmaxf(mx[rr], __shfl_xor_sync(0xffffffffu, mx[rr], 2));
             const float mn = fmaxf(m_run[rr], mx[rr]);
             m_use[rr] = mn == -INFINITY ? 0.f : mn;
-            corr[rr] = m_run[rr] == -INFINITY ? 0.f : exp2f(m_run[rr] - m_use[rr]);
+            corr[rr] = m_run[rr] == -INFINITY ? 0.f : ex2(m_run[rr] - m_use[rr]);
             m_run[rr] = mn;
         }
 #pragma unroll
         for (int nt = 0; nt < BK / 8; ++nt) {
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
-                s[nt][e] = exp2f(s[nt][e] - m_use[e >> 1]);
+                s[nt][e] = ex2(s[nt][e] - m_use[e >> 1]);
                 rs[e >> 1] += s[nt][e];
             }
         }
@@ -228,10 +231,12 @@ window_prefill_kernel(const __grid_constant__ md_win_attn p) {
             rs[rr] += __shfl_xor_sync(0xffffffffu, rs[rr], 2);
             l_run[rr] = l_run[rr] * corr[rr] + rs[rr];
         }
+        if (__any_sync(0xffffffffu, corr[0] != 1.f || corr[1] != 1.f)) {   // a maximum of this warp's rows moved
 #pragma unroll
-        for (int i = 0; i < DP / 8; ++i) {
-            o[i][0] *= corr[0]; o[i][1] *= corr[0];
-            o[i][2] *= corr[1]; o[i][3] *= corr[1];
+            for (int i = 0; i < DP / 8; ++i) {
+                o[i][0] *= corr[0]; o[i][1] *= corr[0];
+                o[i][2] *= corr[1]; o[i][3] *= corr[1];
+            }
         }
 #pragma unroll
         for (int kk = 0; kk < BK / 16; ++kk) {
@@ -250,7 +255,6 @@ window_prefill_kernel(const __grid_constant__ md_win_attn p) {
                 mma(o[2 * dp + 1], lo[0], lo[1], lo[2], lo[3], b[2], b[3]);
             }
         }
-        __syncthreads();
     }
 #pragma unroll
     for (int rr = 0; rr < 2; ++rr) {
