@@ -98,6 +98,8 @@ int md_text_generate_batch_forced(md_text_model* model, md_text_request* const* 
  * One layer, x being the f32 residual stream and m = residual_mult:
  *   u = rms(x; norm1);  u += causal_conv(u; conv1);  x += m * rms(mixer(u); norm1b)
  *   u = rms(x; norm2);  u += causal_conv(u; conv2);  x += m * rms(ff(u);    norm2b)      (ff != MD_FF_NONE)
+ * or, with form MD_LAYER_PARALLEL (no convolution, no norm1b / norm2b; all layers of a model have the same form),
+ *   x += ls1 * mixer(rms(x; norm1)) + ls2 * ff(rms(x; norm2))                             (both of the same x)
  *
  * Mixers
  *   MD_MIXER_WINDOW_ATTENTION  grouped-query softmax attention whose values are its keys; score(i, j) =
@@ -105,17 +107,30 @@ int md_text_generate_batch_forced(md_text_model* model, md_text_request* const* 
  *       j < keep_first); head h's output is multiplied by logistic(g_h).  w_in rows: q | k | g.
  *   MD_MIXER_LIGHTNING         linear attention: S_t = decay[h] S_(t-1) + k_t v_t^T, o_t = S_t^T q_t with q, k, v = silu
  *       of their projections; rms over all heads with mix_norm, times logistic(g).  w_in rows: q | k | v | g.
+ *   MD_MIXER_LATENT_ATTENTION  multi-head softmax attention whose keys and values are linear maps of one normed latent per
+ *       token (kv_rank values), with a rotated key part (rot_dim values) that all heads share; only those are cached.
+ *       w_in rows: query latent (q_rank) | key / value latent | rotated key part.  With cq = rms(query latent; q_norm) and
+ *       c = rms(key / value latent; kv_norm), both with a plain weight: q = w_uq cq, per head dim values and rot_dim rotated
+ *       ones; k = w_uk c, v = w_uv c; score(i, j) = scale * (q.k + rotated q . rotated k), visible iff 0 <= i - j < window;
+ *       exp(sink[h]) joins the softmax's denominator.  The rotation turns the pair (2 i, 2 i + 1) of the rotated part by
+ *       position * rope_base^(-2 i / rot_dim).
  * Feed-forward
- *   MD_FF_DENSE  w_down (act(w_gate u) * (w_up u));  MD_FF_MOE  `top` of `experts` such layers chosen by the largest
- *       logistic(router u) and weighted with those scores.
+ *   MD_FF_DENSE  w_down gated(w_gate u, w_up u);  MD_FF_MOE  `top` of `experts` such layers, weighted.  The router (32-bit)
+ *       takes the largest logits z = router u and weights with
+ *         MD_ROUTER_LOGISTIC  logistic(z)            MD_ROUTER_SOFTMAX  the softmax over the chosen logits
+ *       shared_ff > 0: one more such layer (shared_*) runs for every token; its weight is logistic(row `experts` of router . u).
+ *   gated(g, u) = act(g) * u, or with MD_ACT_CLAMPED, g' = min(g, limit) and u' = min(max(u, -limit), limit):
+ *       g' * logistic(act_alpha * g') * (u' + 1)
  *
  * dtype MD_DTYPE_BF16: matrices and activations bfloat16, f32 accumulation.  MD_DTYPE_F32: everything f32, no
  * reduced-precision product.  Matrices marked T below have that type; vectors are always f32.  All pointers are device
  * pointers that stay valid as long as the model. */
 enum { MD_DTYPE_F16 = 0, MD_DTYPE_BF16 = 1, MD_DTYPE_F32 = 2 };
-enum { MD_MIXER_WINDOW_ATTENTION = 1, MD_MIXER_LIGHTNING = 2 };
+enum { MD_MIXER_WINDOW_ATTENTION = 1, MD_MIXER_LIGHTNING = 2, MD_MIXER_LATENT_ATTENTION = 3 };
+enum { MD_LAYER_SANDWICH = 0, MD_LAYER_PARALLEL = 1 };
 enum { MD_FF_NONE = 0, MD_FF_DENSE = 1, MD_FF_MOE = 2 };
-enum { MD_ACT_GELU_TANH = 1, MD_ACT_SILU = 2 };
+enum { MD_ACT_GELU_TANH = 1, MD_ACT_SILU = 2, MD_ACT_CLAMPED = 3 };
+enum { MD_ROUTER_LOGISTIC = 0, MD_ROUTER_SOFTMAX = 1 };
 
 typedef struct md_stack_layer {
     int mixer, ff;
@@ -135,8 +150,21 @@ typedef struct md_stack_layer {
     size_t ff_dim, ff_pad;                 /* ff_pad: ff_dim rounded up to a multiple of 32 */
     const void* w_gate_up;                 /* T [(experts,) 2 * ff_pad, width]: blocks of 32 gate rows and 32 up rows in turn */
     const void* w_down;                    /* T [(experts,) width, ff_pad] */
-    const void* router;                    /* T [experts, width] */
+    const void* router;                    /* T [experts (+ 1 with a shared expert), width] */
     size_t experts, top;
+    int form, router_kind;                 /* MD_LAYER_*, MD_ROUTER_* */
+    const float* ls1; const float* ls2;    /* parallel form, [width] or NULL (ones) */
+    float act_limit, act_alpha;            /* MD_ACT_CLAMPED; shared expert: shared_limit and the same act and act_alpha */
+    size_t shared_ff, shared_pad;          /* shared expert; shared_pad: shared_ff rounded up to a multiple of 32 */
+    float shared_limit;
+    const void* shared_gate_up;            /* T [2 * shared_pad, width], as w_gate_up */
+    const void* shared_down;               /* T [width, shared_pad] */
+    size_t q_rank, kv_rank, rot_dim;       /* latent attention; rot_dim even */
+    float rope_base;
+    const float* q_norm; const float* kv_norm; const float* sink;   /* [q_rank], [kv_rank], [heads] */
+    const void* w_uq;                      /* T [heads * (dim + rot_dim), q_rank]: head by head, dim rows then rot_dim rows */
+    const void* w_ukv;                     /* T [heads * dim + heads * vdim, kv_rank]: w_uk, then w_uv, head by head */
+    const void* w_ukt;                     /* T [heads, kv_rank, dim]: w_uk transposed per head, or NULL (slower decoding) */
 } md_stack_layer;
 
 typedef struct md_stack_weights {

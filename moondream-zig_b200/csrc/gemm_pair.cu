@@ -260,7 +260,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant
 #pragma unroll
                     for (int q = 0; q < 4; ++q) {
                         uint32_t pk[4];
-                        glu_glue8(g + 8 * q, u + 8 * q, lin.glu, pk);
+                        glu_glue8(g + 8 * q, u + 8 * q, lin, pk);
                         const int chunk = q ^ ((lane >> 1) & 3);   // 64-byte swizzle
                         *reinterpret_cast<uint4*>(my_epi_ptr + lane * 64 + chunk * 16) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
                     }

@@ -201,7 +201,7 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_consta
                     for (int j = 0; j < 4; ++j) u[j] = __shfl_down_sync(0xffffffffu, f[j], 8);
                     if ((et & 8) || n >= N || m >= M) return;
 #pragma unroll
-                    for (int j = 0; j < 4; ++j) f[j] = fast_act(lin.glu, f[j]) * u[j];
+                    for (int j = 0; j < 4; ++j) f[j] = fast_gated(lin, f[j], u[j]);
                     md_store4<__nv_bfloat16>(Cb + (size_t)m * (N / 2) + (n & ~63) / 2 + (n & 31), f);
                     return;
                 }

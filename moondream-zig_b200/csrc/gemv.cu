@@ -293,7 +293,7 @@ gemv_lin_kernel(const __half* A, const __half* __restrict__ Bt, __nv_bfloat16* C
                 a += partial[w][r][m];
                 b += partial[w][r + 8][m];
             }
-            C[(size_t)m * (N / 2) + blockIdx.x * 8 + r] = __float2bfloat16_rn(md_act(ep.glu, a) * b);
+            C[(size_t)m * (N / 2) + blockIdx.x * 8 + r] = __float2bfloat16_rn(md_gated(ep.glu, ep.glu_limit, ep.glu_alpha, a, b));
         }
         return;
     }

@@ -53,7 +53,8 @@ gemm_plain_kernel(const T* __restrict__ A, const T* __restrict__ Wt, T* __restri
             const int n = n0 + tx * 2 + (j & 1) + (j >> 1) * 32;
             if (n >= N) continue;
             if (ep.glu) {
-                if (j < 2) C[(size_t)m * (N / 2) + n0 / 2 + tx * 2 + j] = md_elem<T>::put(md_act(ep.glu, acc[i][j]) * acc[i][j + 2]);
+                if (j < 2) C[(size_t)m * (N / 2) + n0 / 2 + tx * 2 + j] = 
+                    md_elem<T>::put(md_gated(ep.glu, ep.glu_limit, ep.glu_alpha, acc[i][j], acc[i][j + 2]));
                 continue;
             }
             float v = acc[i][j];

@@ -98,6 +98,14 @@ int copy_out(md_ctx* ctx, void* user, const void* dev, size_t bytes) {
 
 }  // namespace
 
+int md_side_stream(md_ctx* ctx) {
+    if (ctx->side_stream) return MD_OK;
+    MD_CUDA(ctx, cudaStreamCreateWithFlags(&ctx->side_stream, cudaStreamNonBlocking));
+    MD_CUDA(ctx, cudaEventCreateWithFlags(&ctx->ev_fork, cudaEventDisableTiming));
+    MD_CUDA(ctx, cudaEventCreateWithFlags(&ctx->ev_side, cudaEventDisableTiming));
+    return MD_OK;
+}
+
 // ------------------------------------------------------------------------------------ text
 
 namespace {
@@ -185,11 +193,7 @@ int text_layer(md_text_model* m, size_t layer, const LayerIO& io, size_t rows, b
             //   side: [LayerNorm + fc1 + GELU] -> [fc2 + bias -> mlp_out] --^
             // Same rounding points as the reference: attn_out = f16(f16(acc) + b), mlp_out likewise,
             // attn_out += mlp_out, hidden += attn_out (text_model.zig:162-171).
-            if (!ctx->side_stream) {
-                MD_CUDA(ctx, cudaStreamCreateWithFlags(&ctx->side_stream, cudaStreamNonBlocking));
-                MD_CUDA(ctx, cudaEventCreateWithFlags(&ctx->ev_fork, cudaEventDisableTiming));
-                MD_CUDA(ctx, cudaEventCreateWithFlags(&ctx->ev_side, cudaEventDisableTiming));
-            }
+            MD_TRY(md_side_stream(ctx));
             cudaStream_t main_stream = ctx->stream;
             MD_CUDA(ctx, cudaEventRecord(ctx->ev_fork, main_stream));            // hidden of the previous layer is final
             const int parts = ctx->decode_mlp_split;
@@ -279,11 +283,7 @@ int text_layer(md_text_model* m, size_t layer, const LayerIO& io, size_t rows, b
     // out-projection's epilogue (same roundings as the sequential form, text_model.zig:162-171).
     const bool fork_prefill = ctx->prefill_fork && (decode ? ctx->decode_fork != 0 : rows > 8);
     if (fork_prefill) {
-        if (!ctx->side_stream) {
-            MD_CUDA(ctx, cudaStreamCreateWithFlags(&ctx->side_stream, cudaStreamNonBlocking));
-            MD_CUDA(ctx, cudaEventCreateWithFlags(&ctx->ev_fork, cudaEventDisableTiming));
-            MD_CUDA(ctx, cudaEventCreateWithFlags(&ctx->ev_side, cudaEventDisableTiming));
-        }
+        MD_TRY(md_side_stream(ctx));
         cudaStream_t main_stream = ctx->stream;
         MD_CUDA(ctx, cudaEventRecord(ctx->ev_fork, main_stream));  // LayerNorm output ready
         MD_CUDA(ctx, cudaStreamWaitEvent(ctx->side_stream, ctx->ev_fork, 0));

@@ -1,4 +1,5 @@
-// Mixture of experts with independent logistic scores (md_moe in stack.cuh).
+// Mixture of experts (md_moe in stack.cuh): independent logistic scores, or a softmax over the chosen experts' logits, and
+// an optional shared expert that every token takes, weighted with the logistic of the router's last row.
 //
 // Prompts (and every shape the kernels below cannot take):
 //   moe_router_kernel, moe_router_mma_kernel
@@ -6,12 +7,13 @@
 //                       (token, expert) pair's rank within its expert
 //   moe_permute_kernel  rows sorted by expert, every expert's rows starting at a multiple of 128
 // then the two expert products run as grouped products over the sorted rows, and the weighted sum of a token's experts
-// is taken where the residual is updated (md_glue::slot).
+// is taken where the residual is updated (md_glue::slot).  The shared expert's two products run over the tokens as they
+// are, its rows land behind the sorted ones, and a token's last entry of slot and score points there.
 //
 // Up to eight bfloat16 tokens (a decode step), weights streamed as in gemv.cu:
 //   moe_route_kernel    scores of all tokens; the last block to arrive chooses and lists the experts in use ("slots") with
 //                       every token's weight in each (zero where the token does not use it)
-//   moe_up_kernel       the slots' gated products, times the token's weight
+//   moe_up_kernel       the slots' gated products, times the token's weight; the shared expert is one more slot
 //   moe_down_kernel     one long product over all slots' columns, so the weighted sum needs no second pass
 #include "mma_bf16.cuh"
 
@@ -19,11 +21,14 @@ namespace {
 
 constexpr int MAX_EXPERTS = 512, MAX_TOP = 32;
 
-// The `top` largest of s[0 .. E) (shared memory, lowest index first among equals), by one warp: fn(k, expert, score).
+// The `top` largest of the logits s[0 .. E) (shared memory, lowest index first among equals), by one warp:
+// fn(k, expert, weight) in lane k.
 template <class F>
-__device__ __forceinline__ void warp_top(float* s, int E, int top, int lane, F&& fn) {
+__device__ __forceinline__ void warp_top(float* s, int E, int top, int kind, int lane, F&& fn) {
+    float mine = -INFINITY, first = -INFINITY;
+    int expert = 0;
     for (int k = 0; k < top; ++k) {
-        float best = -1.f;
+        float best = -INFINITY;
         int bi = 0;
         for (int e = lane; e < E; e += 32)
             if (s[e] > best) { best = s[e]; bi = e; }
@@ -33,37 +38,51 @@ __device__ __forceinline__ void warp_top(float* s, int E, int top, int lane, F&&
             const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
             if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; }
         }
-        if (lane == 0) {
-            fn(k, bi, best);
-            s[bi] = -2.f;
+        if (k == 0) first = best;
+        if (lane == k) {
+            mine = best;
+            expert = bi;
         }
+        if (lane == 0) s[bi] = -INFINITY;
         __syncwarp();
     }
+    if (kind == MD_ROUTER_SOFTMAX) {
+        mine = lane < top ? expf(mine - first) : 0.f;
+        float sum = mine;
+#pragma unroll
+        for (int o = 16; o; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+        mine /= sum;
+    } else {
+        mine = md_logistic(mine);
+    }
+    if (lane < top) fn(lane, expert, mine);
+    __syncwarp();
 }
 
 // one warp per token
 template <class T>
 __global__ void __launch_bounds__(128)
-moe_router_kernel(const T* __restrict__ h, const T* __restrict__ router, int rows, int W, int E, int top, float* score,
-                  int* sel, int* rank, int* count) {
-    __shared__ float s_all[4][MAX_EXPERTS];
+moe_router_kernel(const T* __restrict__ h, const T* __restrict__ router, int rows, int W, int E, int shared, int top, int kind,
+                  float* score, int* sel, int* rank, int* count) {
+    __shared__ float s_all[4][MAX_EXPERTS + 1];
     md_pdl_launch_dependents();
     md_pdl_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x * 4 + warp;
     if (t >= rows) return;
     float* s = s_all[warp];
     const T* hr = h + (size_t)t * W;
-    for (int e = 0; e < E; ++e) {
+    for (int e = 0; e < E + shared; ++e) {
         const T* wr = router + (size_t)e * W;
         float z = 0.f;
         for (int c = lane; c < W; c += 32) z = fmaf(md_elem<T>::get(hr[c]), md_elem<T>::get(wr[c]), z);
 #pragma unroll
         for (int o = 16; o; o >>= 1) z += __shfl_xor_sync(0xffffffffu, z, o);
-        if (lane == 0) s[e] = md_logistic(z);
+        if (lane == 0) s[e] = z;
     }
     __syncwarp();
-    warp_top(s, E, top, lane, [&](int k, int e, float v) {
-        score[(size_t)t * top + k] = v;
+    if (shared && lane == 0) score[(size_t)t * (top + 1) + top] = md_logistic(s[E]);
+    warp_top(s, E, top, kind, lane, [&](int k, int e, float v) {
+        score[(size_t)t * (top + shared) + k] = v;
         sel[(size_t)t * top + k] = e;
         rank[(size_t)t * top + k] = atomicAdd(count + e, 1);
     });
@@ -71,8 +90,9 @@ moe_router_kernel(const T* __restrict__ h, const T* __restrict__ router, int row
 
 template <class T>
 __global__ void __launch_bounds__(256)
-moe_permute_kernel(const T* __restrict__ h, int W, int E, int top, const int* __restrict__ sel, const int* __restrict__ rank,
-                   const int* __restrict__ count, int* slot, int* tile_expert, int* n_blocks, T* __restrict__ xs) {
+moe_permute_kernel(const T* __restrict__ h, int W, int E, int shared_row, int top, const int* __restrict__ sel,
+                   const int* __restrict__ rank, const int* __restrict__ count, int* slot, int* tile_expert, int* n_blocks,
+                   T* __restrict__ xs) {
     __shared__ int first[MAX_EXPERTS + 1];   // first row block of every expert
     md_pdl_launch_dependents();
     md_pdl_wait();
@@ -100,9 +120,11 @@ moe_permute_kernel(const T* __restrict__ h, int W, int E, int top, const int* __
         if (threadIdx.x == 0) *n_blocks = first[E];
     }
     const T* src = h + (size_t)t * W;
+    const int choices = top + (shared_row >= 0 ? 1 : 0);
+    if (shared_row >= 0 && threadIdx.x == 0) slot[(size_t)t * choices + top] = shared_row + t;
     for (int k = 0; k < top; ++k) {
         const int e = sel[(size_t)t * top + k], row = first[e] * MD_GROUP_ROWS + rank[(size_t)t * top + k];
-        if (threadIdx.x == 0) slot[(size_t)t * top + k] = row;
+        if (threadIdx.x == 0) slot[(size_t)t * choices + k] = row;
         T* dst = xs + (size_t)row * W;
         if ((W * sizeof(T)) % 16 == 0) {
             for (int c = threadIdx.x; c < (int)(W * sizeof(T) / 16); c += blockDim.x)
@@ -143,12 +165,13 @@ constexpr int RT = 16, RE = 64;   // tokens per block, experts per pass
 constexpr int RW = 16;   // warps that split the width
 
 __global__ void __launch_bounds__(RW * 32)
-moe_router_mma_kernel(const __nv_bfloat16* h, const __nv_bfloat16* __restrict__ router, int rows, int W, int E, int top, float* score,
-                      int* sel, int* rank, int* count) {
+moe_router_mma_kernel(const __nv_bfloat16* h, const __nv_bfloat16* __restrict__ router, int rows, int W, int E, int shared, int top,
+                      int kind, float* score, int* sel, int* rank, int* count) {
+    const int EA = E + shared;   // rows of the router
     extern __shared__ float smf[];
     float (*part)[RT][RE] = reinterpret_cast<float (*)[RT][RE]>(smf);   // [RW]
-    float* sc = smf + RW * RT * RE;                                      // [RT][E]
-    int* cnt = reinterpret_cast<int*>(sc + RT * E);                     // [E]: this block's tokens per expert, then its base
+    float* sc = smf + RW * RT * RE;                                      // [RT][EA]
+    int* cnt = reinterpret_cast<int*>(sc + RT * EA);                    // [E]: this block's tokens per expert, then its base
     md_pdl_launch_dependents();
     md_pdl_wait();
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
@@ -156,7 +179,7 @@ moe_router_mma_kernel(const __nv_bfloat16* h, const __nv_bfloat16* __restrict__ 
     for (int e = tid; e < E; e += RW * 32) cnt[e] = 0;
     const __nv_bfloat16* lo = h + (size_t)(t0 + min(g, n - 1)) * W + t * 8;
     const __nv_bfloat16* hi = h + (size_t)(t0 + min(g + 8, n - 1)) * W + t * 8;
-    for (int e0 = 0; e0 < E; e0 += RE) {
+    for (int e0 = 0; e0 < EA; e0 += RE) {
         float acc[RE / 8][4];
 #pragma unroll
         for (int i = 0; i < RE / 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
@@ -167,8 +190,8 @@ moe_router_mma_kernel(const __nv_bfloat16* h, const __nv_bfloat16* __restrict__ 
 #pragma unroll
             for (int i = 0; i < RE / 8; ++i) {
                 const int e = e0 + i * 8 + g;
-                if (e0 + i * 8 >= E) break;
-                const uint4 x = live && e < E ? *reinterpret_cast<const uint4*>(router + (size_t)e * W + t * 8 + k) : z;
+                if (e0 + i * 8 >= EA) break;
+                const uint4 x = live && e < EA ? *reinterpret_cast<const uint4*>(router + (size_t)e * W + t * 8 + k) : z;
                 mma_piece(acc[i], a, b, x);
             }
         }
@@ -185,16 +208,17 @@ moe_router_mma_kernel(const __nv_bfloat16* h, const __nv_bfloat16* __restrict__ 
             float v = 0.f;
 #pragma unroll
             for (int w = 0; w < RW; ++w) v += part[w][r][e];
-            if (e0 + e < E) sc[r * E + e0 + e] = md_logistic(v);
+            if (e0 + e < EA) sc[r * EA + e0 + e] = v;
         }
         __syncthreads();
     }
     for (int r = warp; r < n; r += RW)
-        warp_top(sc + r * E, E, top, lane, [&](int k, int e, float v) {
+        warp_top(sc + r * EA, E, top, kind, lane, [&](int k, int e, float v) {
             const size_t at = (size_t)(t0 + r) * top + k;
-            score[at] = v;
+            score[(size_t)(t0 + r) * (top + shared) + k] = v;
             sel[at] = e;
             rank[at] = atomicAdd(cnt + e, 1);
+            if (k == 0 && shared) score[(size_t)(t0 + r) * (top + 1) + top] = md_logistic(sc[r * EA + E]);
         });
     __syncthreads();
     for (int e = tid; e < E; e += RW * 32)
@@ -208,21 +232,24 @@ moe_router_mma_kernel(const __nv_bfloat16* h, const __nv_bfloat16* __restrict__ 
 
 // ---- up to eight tokens
 struct Route {
-    float* score;        // [8][E]
+    float* score;        // [8][rows of the router]
     float* weight;       // [slots][8]
+    float* shared;       // [8] the shared expert's weight
     int *expert, *n_slots;
     unsigned* ticket;    // zero between launches
 };
 
 __global__ void __launch_bounds__(512)
-moe_route_kernel(const __nv_bfloat16* h, const __nv_bfloat16* __restrict__ router, int T, int W, int E, int top, Route r) {
-    extern __shared__ float sc[];            // last block: [8][E] scores, then [8][E] chosen scores
+moe_route_kernel(const __nv_bfloat16* h, const __nv_bfloat16* __restrict__ router, int T, int W, int E, int shared, int top, int kind,
+                 Route r) {
+    const int EA = E + shared;               // rows of the router
+    extern __shared__ float sc[];            // last block: [8][EA] logits, then [8][EA] chosen weights
     __shared__ float partial[16][16][8];
     __shared__ int last_s;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
     const int row0 = blockIdx.x * 16;
-    const __nv_bfloat16* w_lo = router + (size_t)min(row0 + g, E - 1) * W + t * 8;
-    const __nv_bfloat16* w_hi = router + (size_t)min(row0 + g + 8, E - 1) * W + t * 8;
+    const __nv_bfloat16* w_lo = router + (size_t)min(row0 + g, EA - 1) * W + t * 8;
+    const __nv_bfloat16* w_hi = router + (size_t)min(row0 + g + 8, EA - 1) * W + t * 8;
     const __nv_bfloat16* x = h + (size_t)min(g, T - 1) * W + t * 8;
     float acc[4] = {0.f, 0.f, 0.f, 0.f};
     const uint4 zero = make_uint4(0, 0, 0, 0);
@@ -258,10 +285,10 @@ moe_route_kernel(const __nv_bfloat16* h, const __nv_bfloat16* __restrict__ route
         float v = 0.f;
 #pragma unroll
         for (int w = 0; w < 16; ++w) v += partial[w][e][m];
-        if (m < T && row0 + e < E) (gridDim.x == 1 ? sc : r.score)[m * E + row0 + e] = md_logistic(v);
+        if (m < T && row0 + e < EA) (gridDim.x == 1 ? sc : r.score)[m * EA + row0 + e] = v;
     }
-    float* chosen = sc + 8 * E;
-    for (int i = tid; i < T * E; i += 512) chosen[i] = 0.f;
+    float* chosen = sc + 8 * EA;
+    for (int i = tid; i < T * EA; i += 512) chosen[i] = 0.f;
     if (gridDim.x > 1) {
         __threadfence();
         __syncthreads();
@@ -270,22 +297,23 @@ moe_route_kernel(const __nv_bfloat16* h, const __nv_bfloat16* __restrict__ route
         if (!last_s) return;
         __threadfence();
         if (tid == 0) *r.ticket = 0u;
-        for (int i = tid; i < T * E; i += 512) sc[i] = __ldcg(r.score + i);
+        for (int i = tid; i < T * EA; i += 512) sc[i] = __ldcg(r.score + i);
     }
     __syncthreads();
-    if (warp < T) warp_top(sc + warp * E, E, top, lane, [&](int, int e, float v) { chosen[warp * E + e] = v; });
+    if (shared && tid < 8) r.shared[tid] = tid < T ? md_logistic(sc[tid * EA + E]) : 0.f;
+    if (warp < T) warp_top(sc + warp * EA, E, top, kind, lane, [&](int, int e, float v) { chosen[warp * EA + e] = v; });
     __syncthreads();
     if (warp == 0) {
         int slots = 0;
         for (int e0 = 0; e0 < E; e0 += 32) {
             const int e = e0 + lane;
             bool used = false;
-            for (int m = 0; m < T; ++m) used |= e < E && chosen[m * E + e] != 0.f;
+            for (int m = 0; m < T; ++m) used |= e < E && chosen[m * EA + e] != 0.f;
             const unsigned b = __ballot_sync(0xffffffffu, used);
             if (used) {
                 const int s = slots + __popc(b & ((1u << lane) - 1u));
                 r.expert[s] = e;
-                for (int m = 0; m < 8; ++m) r.weight[s * 8 + m] = m < T ? chosen[m * E + e] : 0.f;
+                for (int m = 0; m < 8; ++m) r.weight[s * 8 + m] = m < T ? chosen[m * EA + e] : 0.f;
             }
             slots += __popc(b);
         }
@@ -293,20 +321,29 @@ moe_route_kernel(const __nv_bfloat16* h, const __nv_bfloat16* __restrict__ route
     }
 }
 
-// act[token][slot * ff_pad + j] = weight * act(gate_j) * up_j
+struct FewShared {       // the shared expert's products; pad 0: none
+    const __nv_bfloat16 *gu, *down;
+    int pad;
+    float limit;
+};
+
+// act[token][slot * ff_pad + j] = weight * gated(gate_j, up_j); the shared expert's columns follow those of all `slots`
 __global__ void __launch_bounds__(256)
 moe_up_kernel(const __nv_bfloat16* h, const __nv_bfloat16* __restrict__ w_gu, __nv_bfloat16* out, int T, int W, int ff_pad, int act,
-              int out_stride, Route r) {
+              float limit, float alpha, int slots, FewShared sh, Route r) {
     __shared__ float partial[8][16][8];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
     const int slot = blockIdx.y, j = blockIdx.x * 8 + g;
     md_pdl_launch_dependents();
     md_pdl_wait();
     // (the three small loads together; entries past n_slots are dropped right after)
-    const int n_slots = __ldcg(r.n_slots), expert = __ldcg(r.expert + slot);
-    const float mine = __ldcg(r.weight + slot * 8 + g);
-    if (slot >= n_slots) return;
-    const __nv_bfloat16* w = w_gu + (size_t)expert * 2 * ff_pad * W;
+    const bool is_shared = slot == slots;
+    const float* weight = is_shared ? r.shared : r.weight + slot * 8;
+    const int n_slots = __ldcg(r.n_slots), expert = is_shared ? 0 : __ldcg(r.expert + slot);
+    const float mine = __ldcg(weight + g);
+    if (is_shared ? (int)blockIdx.x * 8 >= sh.pad : slot >= n_slots || (int)blockIdx.x * 8 >= ff_pad) return;
+    if (is_shared) limit = sh.limit;
+    const __nv_bfloat16* w = is_shared ? sh.gu : w_gu + (size_t)expert * 2 * ff_pad * W;
     const __nv_bfloat16* w_lo = w + (size_t)((j / MD_GLU_BLOCK) * (2 * MD_GLU_BLOCK) + j % MD_GLU_BLOCK) * W + t * 8;
     const __nv_bfloat16* w_hi = w_lo + (size_t)MD_GLU_BLOCK * W;
     const bool has_x = g < T && mine != 0.f;
@@ -340,24 +377,24 @@ moe_up_kernel(const __nv_bfloat16* h, const __nv_bfloat16* __restrict__ w_gu, __
                 a += partial[q][e][m];
                 b += partial[q][e + 8][m];
             }
-            const float wt = __ldcg(r.weight + slot * 8 + m);
-            out[(size_t)m * out_stride + slot * ff_pad + blockIdx.x * 8 + e] = __float2bfloat16_rn(wt * md_act(act, a) * b);
+            out[(size_t)m * (slots * ff_pad + sh.pad) + slot * ff_pad + blockIdx.x * 8 + e] =
+                __float2bfloat16_rn(__ldcg(weight + m) * md_gated(act, limit, alpha, a, b));
         }
     }
 }
 
 // y[token][n] = sum over the slots' columns
 __global__ void __launch_bounds__(512, 2)
-moe_down_kernel(const __nv_bfloat16* act, const __nv_bfloat16* __restrict__ w_down, float* y, int T, int W, int ff_pad, int act_stride,
-                Route r) {
+moe_down_kernel(const __nv_bfloat16* act, const __nv_bfloat16* __restrict__ w_down, float* y, int T, int W, int ff_pad, int slots,
+                FewShared sh, Route r) {
     __shared__ float partial[16][16][8];
     __shared__ int list[MAX_EXPERTS];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
-    const int row0 = blockIdx.x * 16, per = ff_pad / 32;
+    const int row0 = blockIdx.x * 16, per = ff_pad / 32, act_stride = slots * ff_pad + sh.pad;
     md_pdl_launch_dependents();
     md_pdl_wait();
-    const int n_slots = __ldcg(r.n_slots), chunks = n_slots * per;
-    if (tid < act_stride / ff_pad) list[tid] = __ldcg(r.expert + tid);   // what is past n_slots is not used
+    const int n_slots = __ldcg(r.n_slots), routed = n_slots * per, chunks = routed + sh.pad / 32;
+    if (tid < slots) list[tid] = __ldcg(r.expert + tid);   // what is past n_slots is not used
     __syncthreads();
     const size_t r_lo = min(row0 + g, W - 1), r_hi = min(row0 + g + 8, W - 1);
     const __nv_bfloat16* x = act + (size_t)(g < T ? g : 0) * act_stride + t * 8;
@@ -371,11 +408,12 @@ moe_down_kernel(const __nv_bfloat16* act, const __nv_bfloat16* __restrict__ w_do
             const int c = c0 + u * 16;
             lo[u] = hi[u] = xv[u] = zero;
             if (c < chunks) {
-                const int slot = c / per, k = (c - slot * per) * 32 + t * 8;
-                const __nv_bfloat16* w = w_down + (size_t)list[slot] * W * ff_pad + k;
-                lo[u] = ldg_stream(w + r_lo * ff_pad);
-                hi[u] = ldg_stream(w + r_hi * ff_pad);
-                if (g < T) xv[u] = ld_act(x + c * 32);
+                const bool own = c < routed;
+                const int slot = own ? c / per : 0, pitch = own ? ff_pad : sh.pad;
+                const __nv_bfloat16* w = own ? w_down + (size_t)list[slot] * W * ff_pad + (c - slot * per) * 32 : sh.down + (c - routed) * 32;
+                lo[u] = ldg_stream(w + r_lo * pitch + t * 8);
+                hi[u] = ldg_stream(w + r_hi * pitch + t * 8);
+                if (g < T) xv[u] = ld_act(x + (own ? c * 32 : slots * ff_pad + (c - routed) * 32));
             }
         }
 #pragma unroll
@@ -398,52 +436,63 @@ moe_down_kernel(const __nv_bfloat16* act, const __nv_bfloat16* __restrict__ w_do
 }
 
 int launch_few(md_ctx* ctx, const md_moe& m, const void* h, size_t rows, const md_moe_buffers& b) {
-    const int T = (int)rows, E = m.experts, slots = T * m.top < E ? T * m.top : E;
+    const int T = (int)rows, E = m.experts, EA = E + (m.shared_pad > 0), slots = T * m.top < E ? T * m.top : E;
     Route r;
     // the ticket first: layers of different sizes share the buffer, and it must stay what the last launch left, zero
     r.ticket = reinterpret_cast<unsigned*>(b.route);
     r.n_slots = reinterpret_cast<int*>(b.route) + 1;
-    r.score = b.route + 8;
-    r.weight = r.score + 8 * (size_t)E;
-    r.expert = reinterpret_cast<int*>(r.weight + 8 * (size_t)E);
+    r.shared = b.route + 8;
+    r.score = r.shared + 8;
+    r.weight = r.score + 8 * (size_t)EA;
+    r.expert = reinterpret_cast<int*>(r.weight + 8 * (size_t)EA);
+    const FewShared sh = {reinterpret_cast<const __nv_bfloat16*>(m.shared_gu), reinterpret_cast<const __nv_bfloat16*>(m.shared_down),
+                          m.shared_pad, m.shared_limit};
     const __nv_bfloat16* x = reinterpret_cast<const __nv_bfloat16*>(h);
     __nv_bfloat16* act = reinterpret_cast<__nv_bfloat16*>(b.act);
-    MD_TRY(md_launch_ex(ctx, moe_route_kernel, dim3((unsigned)((E + 15) / 16)), dim3(512), 16 * (size_t)E * sizeof(float), "moe_route_kernel",
-                        x, reinterpret_cast<const __nv_bfloat16*>(m.router), T, m.width, E, m.top, r));
-    MD_TRY(md_launch_ex(ctx, moe_up_kernel, dim3((unsigned)(m.ff_pad / 8), (unsigned)slots), dim3(256), 0, "moe_up_kernel", x,
-                        reinterpret_cast<const __nv_bfloat16*>(m.w_gu), act, T, m.width, m.ff_pad, m.act, slots * m.ff_pad, r));
+    MD_TRY(md_launch_ex(ctx, moe_route_kernel, dim3((unsigned)((EA + 15) / 16)), dim3(512), 16 * (size_t)EA * sizeof(float), "moe_route_kernel",
+                        x, reinterpret_cast<const __nv_bfloat16*>(m.router), T, m.width, E, EA - E, m.top, m.router_kind, r));
+    MD_TRY(md_launch_ex(ctx, moe_up_kernel, dim3((unsigned)((m.ff_pad > m.shared_pad ? m.ff_pad : m.shared_pad) / 8), (unsigned)(slots + EA - E)),
+                        dim3(256), 0, "moe_up_kernel", x,
+                        reinterpret_cast<const __nv_bfloat16*>(m.w_gu), act, T, m.width, m.ff_pad, m.act, m.limit, m.alpha,
+                        slots, sh, r));
     return md_launch_ex(ctx, moe_down_kernel, dim3((unsigned)((m.width + 15) / 16)), dim3(512), 0, "moe_down_kernel", act,
-                        reinterpret_cast<const __nv_bfloat16*>(m.w_down), b.y_f32, T, m.width, m.ff_pad, slots * m.ff_pad, r);
+                        reinterpret_cast<const __nv_bfloat16*>(m.w_down), b.y_f32, T, m.width, m.ff_pad, slots, sh, r);
 }
 
 template <class T>
 int launch_sorted(md_ctx* ctx, int dtype, const md_moe& m, const void* h, size_t rows, const md_moe_buffers& b) {
+    const int shared = m.shared_pad > 0 ? 1 : 0;
+    const size_t cap = md_moe_sorted_rows(rows, m.experts, m.top);
     MD_CUDA(ctx, cudaMemsetAsync(b.count, 0, m.experts * sizeof(int), ctx->stream));
     if (dtype == MD_DTYPE_BF16 && (m.width % 8) == 0) {
-        const size_t smem = (RW * RT * RE + RT * (size_t)m.experts + m.experts) * sizeof(float);
+        const size_t smem = (RW * RT * RE + RT * (size_t)(m.experts + shared) + m.experts) * sizeof(float);
         if (smem > 48 * 1024)
             MD_CUDA(ctx, cudaFuncSetAttribute(moe_router_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         MD_TRY(md_launch_ex(ctx, moe_router_mma_kernel, dim3((unsigned)((rows + RT - 1) / RT)), dim3(RW * 32), smem, "moe_router_mma_kernel",
                             reinterpret_cast<const __nv_bfloat16*>(h), reinterpret_cast<const __nv_bfloat16*>(m.router), (int)rows,
-                            m.width, m.experts, m.top, b.score, b.sel, b.rank, b.count));
+                            m.width, m.experts, shared, m.top, m.router_kind, b.score, b.sel, b.rank, b.count));
     } else {
         MD_TRY(md_launch_ex(ctx, moe_router_kernel<T>, dim3((unsigned)((rows + 3) / 4)), dim3(128), 0, "moe_router_kernel",
                             reinterpret_cast<const T*>(h), reinterpret_cast<const T*>(m.router), (int)rows, m.width, m.experts,
-                            m.top, b.score, b.sel, b.rank, b.count));
+                            shared, m.top, m.router_kind, b.score, b.sel, b.rank, b.count));
     }
     MD_TRY(md_launch_ex(ctx, moe_permute_kernel<T>, dim3((unsigned)rows), dim3(256), 0, "moe_permute_kernel",
-                        reinterpret_cast<const T*>(h), m.width, m.experts, m.top, b.sel, b.rank, b.count, b.slot,
+                        reinterpret_cast<const T*>(h), m.width, m.experts, shared ? (int)cap : -1, m.top, b.sel, b.rank, b.count, b.slot,
                         b.tile_expert, b.n_blocks, reinterpret_cast<T*>(b.xs)));
-    const size_t cap = md_moe_sorted_rows(rows, m.experts, m.top);
     md_lin up;
-    up.glu = m.act;
+    up.glu = m.act, up.glu_limit = m.limit, up.glu_alpha = m.alpha;
     up.tile_expert = b.tile_expert;
     up.n_blocks = b.n_blocks;
     up.n_experts = m.experts;
     MD_TRY(md_linear(ctx, dtype, b.xs, m.w_gu, b.act, cap, 2 * (size_t)m.ff_pad, m.width, up));
     md_lin down = up;
     down.glu = 0;
-    return md_linear(ctx, dtype, b.act, m.w_down, b.ys, cap, m.width, m.ff_pad, down);
+    MD_TRY(md_linear(ctx, dtype, b.act, m.w_down, b.ys, cap, m.width, m.ff_pad, down));
+    if (!shared) return MD_OK;
+    md_lin own;
+    own.glu = m.act, own.glu_limit = m.shared_limit, own.glu_alpha = m.alpha;
+    MD_TRY(md_linear(ctx, dtype, h, m.shared_gu, b.shared_act, rows, 2 * (size_t)m.shared_pad, m.width, own));
+    return md_linear(ctx, dtype, b.shared_act, m.shared_down, reinterpret_cast<T*>(b.ys) + cap * m.width, rows, m.width, m.shared_pad, md_lin());
 }
 
 }  // namespace

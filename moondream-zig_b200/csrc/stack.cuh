@@ -21,6 +21,7 @@ struct md_lin {
     int sigmoid_from = 1 << 30;      // columns >= sigmoid_from go through the logistic function
     // glu != 0: W's rows are gate and up rows in alternating blocks of 32 (MD_GLU_BLOCK) and C[M, N/2] = act(gate) * up
     int glu = 0;                     // MD_ACT_*
+    float glu_limit = 0.f, glu_alpha = 0.f;   // MD_ACT_CLAMPED (md_gated)
     float* out_f32 = nullptr;        // write f32 sums here instead of T to C
     unsigned long long* amax = nullptr;   // [M] running maximum of md_argmax_key over each row (bfloat16, M <= 8; zero before)
     // rows sorted by expert: row block b (128 rows) belongs to expert tile_expert[b], whose matrix is W + e * N * K;
@@ -80,6 +81,32 @@ struct md_glue {
 };
 int md_launch_glue(md_ctx* ctx, int dtype, const md_glue& g);
 
+// The same place in a layer whose two sublayers read the same residual row (MD_LAYER_PARALLEL).  For every row:
+//   x_out = x + sum_b scale_b * y_b      (b = the sublayers that ran; tokens != null: x = embed[token])
+//   n     = x_out / sqrt(mean(x_out^2) + eps);  out[o] = n * w[o]   for up to two outputs
+struct md_branch {
+    const float* y_f32 = nullptr;           // the sublayer's output, as in md_glue: f32 rows, T rows,
+    const void* y = nullptr;
+    const int* slot = nullptr;              //   or T rows of the expert-sorted buffer: sum_k score[t][k] * y[slot[t][k]]
+    const float* score = nullptr;
+    int top = 0;
+    const float* scale = nullptr;           // [width]
+};
+struct md_parallel_glue {
+    int width = 0, rows = 0;                // rows of all sequences
+    float eps = 0.f;
+    const float* x = nullptr;
+    float* x_out = nullptr;                 // may be x
+    const void* embed = nullptr;
+    const unsigned long long* tokens = nullptr;
+    int vocab = 0;
+    md_branch b[2];
+    const float* w[2] = {};
+    void* out[2] = {};                      // [rows, width] T
+    const int* gather = nullptr;            // as in md_glue
+};
+int md_launch_parallel_glue(md_ctx* ctx, int dtype, const md_parallel_glue& g);
+
 // ---- attention: distance bias, sliding window with kept first keys, values = keys, gated heads -------------
 struct md_win_attn {
     int heads = 0, kv_heads = 0, dim = 0;
@@ -97,6 +124,44 @@ struct md_win_attn {
     int pos0 = 0;                           // prefill: position of row 0
 };
 int md_launch_window_attention(md_ctx* ctx, int dtype, const md_win_attn& a, bool decode);
+
+// ---- latent attention: keys and values of all heads are linear maps of one cached latent per token -----------
+// Per token: cq = rms(in[0 .. q_rank); q_norm), c = rms(in[q_rank .. + kv_rank); kv_norm), kr = rotated in[.. + rot).  Cached:
+// c and kr.  Head h: q = w_uq cq, k = w_uk c, v = w_uv c; score(i, j) = scale * (q . k_j + rotated q . kr_j); softmax whose
+// denominator also holds exp(sink[h]).
+struct md_latent {
+    int heads = 0, dim = 0, rot = 0, vdim = 0, q_rank = 0, kv_rank = 0;
+    float scale = 0.f, eps = 0.f;
+    int window = 0;                         // <= 0: unlimited
+    const float *q_norm = nullptr, *kv_norm = nullptr, *sink = nullptr;
+    const float* rope = nullptr;            // [max_seq][rot / 2] (cos, sin)
+    const void* w_uq = nullptr;             // [heads * (dim + rot), q_rank]: per head [dim | rot]
+    const void* w_ukv = nullptr;            // [heads * dim (keys) + heads * vdim (values), kv_rank]
+    const void* w_ukt = nullptr;            // [heads][kv_rank][dim] (bfloat16 decoding; null: not available)
+    const void* in = nullptr;               // [rows of all sequences, row_stride] T
+    int row_stride = 0;
+    void *cq = nullptr, *q = nullptr;       // [rows, q_rank], [rows, heads * (dim + rot)] T
+    void* out = nullptr;                    // [rows, heads * vdim] T
+    int rows = 0, seqs = 1;                 // rows per sequence
+    size_t max_seq = 0;
+    void* cc[MD_STACK_MAX_SEQS] = {};       // [max_seq][kv_rank] T
+    void* kr[MD_STACK_MAX_SEQS] = {};       // [max_seq][rot] T
+    const int* pos_dev[MD_STACK_MAX_SEQS] = {};   // decode: position of the new token
+    int pos0 = 0;                           // prefill: position of row 0
+    // prompts in bfloat16: keys and values of every visible token, [md_latent_keys(..)][heads * (dim + vdim)]
+    void* kv = nullptr;
+    // bfloat16 decoding: absorbed queries [seqs][heads][kv_rank + rot] and merged latents [seqs][heads][kv_rank]
+    void *qa = nullptr, *ol = nullptr;
+};
+// tokens whose keys a portion of `rows` rows can see (itself included)
+inline size_t md_latent_keys(size_t rows, size_t window, size_t max_seq) {
+    return window > 0 && rows + window - 1 < max_seq ? rows + window - 1 : max_seq;
+}
+// whether a portion of `rows` rows of one sequence takes the tensor-core prompt kernel (and so needs md_latent::kv)
+bool md_latent_expands(int dtype, const md_latent& a);
+int md_launch_latent_attention(md_ctx* ctx, int dtype, const md_latent& a, bool decode);
+// (cos, sin) of pos * base^(-2 i / dims) for pos < rows, i < dims / 2; angles in f64
+int md_launch_rotation_table(md_ctx* ctx, float* table, size_t rows, size_t dims, float base);
 
 // ---- linear attention with per-head decay ----------------------------------------------------------------
 struct md_lightning {
@@ -117,19 +182,29 @@ int md_launch_lightning(md_ctx* ctx, int dtype, const md_lightning& l, bool deco
 
 // ---- mixture of experts --------------------------------------------------------------------------------------
 struct md_moe {
-    int width = 0, experts = 0, top = 0, ff = 0, ff_pad = 0, act = 0;
-    const void *router = nullptr, *w_gu = nullptr, *w_down = nullptr;   // [E, W], [E, 2 ff_pad, W], [E, W, ff_pad]
+    int width = 0, experts = 0, top = 0, ff_pad = 0, act = 0;
+    float limit = 0.f, alpha = 0.f;          // of the activation (md_gated)
+    int router_kind = 0;                     // MD_ROUTER_*
+    const void *router = nullptr, *w_gu = nullptr, *w_down = nullptr;   // [E (+ 1), W], [E, 2 ff_pad, W], [E, W, ff_pad]
+    // shared expert (shared_pad > 0): runs for every token, weighted with the logistic of the router's row E
+    int shared_pad = 0;
+    float shared_limit = 0.f;
+    const void *shared_gu = nullptr, *shared_down = nullptr;            // [2 shared_pad, W], [W, shared_pad]
+    int choices() const { return top + (shared_pad > 0 ? 1 : 0); }      // entries of a token in score and slot
 };
 struct md_moe_buffers {
-    float* score = nullptr;       // [rows, top]
-    int *sel = nullptr, *rank = nullptr, *slot = nullptr;     // [rows, top]
+    float* score = nullptr;       // [rows, choices]
+    int* slot = nullptr;          // [rows, choices]
+    int *sel = nullptr, *rank = nullptr;                      // [rows, top]
     int *count = nullptr;         // [experts]
     int *tile_expert = nullptr, *n_blocks = nullptr;
-    void *xs = nullptr, *act = nullptr, *ys = nullptr;        // sorted rows
+    // sorted rows; act also takes 8 rows of shared_pad, ys also the shared expert's row of every token
+    void *xs = nullptr, *act = nullptr, *ys = nullptr;
+    void* shared_act = nullptr;   // [rows, shared_pad]
     float* y_f32 = nullptr;       // [rows, width], rows <= 8
     float* route = nullptr;       // md_moe_route_floats(experts), zeroed once
 };
-inline size_t md_moe_route_floats(size_t experts) { return 17 * experts + 8; }
+inline size_t md_moe_route_floats(size_t experts) { return 17 * (experts + 1) + 16; }
 size_t md_moe_sorted_rows(size_t rows, int experts, int top);   // capacity of the sorted buffers
 // true: md_launch_moe leaves a token's outputs in the sorted rows (slot, score, ys); false: their sum in y_f32
 bool md_moe_sorted(int dtype, size_t width, size_t rows);
@@ -158,6 +233,15 @@ __device__ __forceinline__ float md_gelu_tanh(float z) {
     return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
 __device__ __forceinline__ float md_act(int act, float z) { return act == MD_ACT_SILU ? md_silu(z) : md_gelu_tanh(z); }
+// gate and up of a gated feed-forward
+__device__ __forceinline__ float md_gated(int act, float limit, float alpha, float g, float u) {
+    if (act == MD_ACT_CLAMPED) {
+        g = fminf(g, limit);
+        u = fminf(fmaxf(u, -limit), limit);
+        return g * md_logistic(alpha * g) * (u + 1.f);
+    }
+    return md_act(act, g) * u;
+}
 // column activation of md_lin
 __device__ __forceinline__ float md_lin_col(float v, int n, int silu_cols, int sigmoid_from) {
     if (n < silu_cols) return md_silu(v);

@@ -6,6 +6,8 @@
 //                            requested before the dependency wait
 //   stack_glue_rows_kernel   rows of a prompt: a row per warp group, its inputs read once into registers
 //   stack_glue_any_kernel    widths that are not a multiple of 4 or too wide for the others
+//   stack_parallel_kernel    the same place in a layer whose two sublayers read the same row (md_parallel_glue): both layer
+//                            scales and sums, one norm, two weighted outputs
 #include "stack.cuh"
 
 namespace {
@@ -528,10 +530,158 @@ int launch_glue(md_ctx* ctx, const md_glue& g) {
                         "stack_glue_kernel", g, R);
 }
 
+// ---- MD_LAYER_PARALLEL: residual update of two sublayers, one norm, up to two weighted outputs
+
+constexpr int PAR_THREADS = 512;
+
+template <class T> __device__ __forceinline__ const T* embed_row(const md_parallel_glue& p, size_t src) {
+    const unsigned long long tok = p.tokens[src];
+    return reinterpret_cast<const T*>(p.embed) + (size_t)(tok < (unsigned long long)p.vocab ? tok : 0ull) * p.width;
+}
+// columns c .. c + V of a sublayer's output for row `src`
+template <class T, int V> __device__ __forceinline__ Vec<V> branch_cols(const md_branch& b, size_t src, int W, int c) {
+    if (b.slot) {
+        Vec<V> v;
+#pragma unroll
+        for (int i = 0; i < V; ++i) v.f[i] = 0.f;
+        for (int k = 0; k < b.top; ++k) {
+            const float s = __ldcg(b.score + src * b.top + k);
+            const Vec<V> e = ldv<T, V>(reinterpret_cast<const T*>(b.y) + (size_t)__ldcg(b.slot + src * b.top + k) * W + c);
+#pragma unroll
+            for (int i = 0; i < V; ++i) v.f[i] = fmaf(s, e.f[i], v.f[i]);
+        }
+        return v;
+    }
+    return b.y_f32 ? ldv<float, V>(b.y_f32 + src * W + c) : ldv<T, V>(reinterpret_cast<const T*>(b.y) + src * W + c);
+}
+
+// GW warps per row, NV vectors of V columns per lane: width <= 32 * V * GW * NV.  All weights are requested before the
+// dependency wait when one group has the whole block (a decode step).
+template <class T, int V, int GW, int NV>
+__global__ void __launch_bounds__(PAR_THREADS)
+stack_parallel_kernel(const __grid_constant__ md_parallel_glue p) {
+    __shared__ float red[PAR_THREADS / 32];
+    constexpr int GROUPS = PAR_THREADS / 32 / GW;
+    constexpr bool EARLY = GW == PAR_THREADS / 32 && NV <= 2;
+    const int W = p.width, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int grp = warp / GW, gl = (warp % GW) * 32 + lane, row = blockIdx.x * GROUPS + grp;
+    const bool live = row < p.rows;
+    md_pdl_launch_dependents();
+    Vec<V> w[2][NV], s[2][NV];
+    if constexpr (EARLY) {
+#pragma unroll
+        for (int n = 0; n < NV; ++n) {
+            const int c = (gl + n * 32 * GW) * V;
+            if (c >= W) continue;
+#pragma unroll
+            for (int o = 0; o < 2; ++o) {
+                if (p.out[o]) w[o][n] = ldv<float, V>(p.w[o] + c);
+                if (p.b[o].scale) s[o][n] = ldv<float, V>(p.b[o].scale + c);
+            }
+        }
+    }
+    md_pdl_wait();
+    const size_t src = live ? (p.gather ? (size_t)p.gather[row] : row) : 0;
+    Vec<V> x[NV];
+    const T* xe = p.tokens ? embed_row<T>(p, src) : nullptr;
+#pragma unroll
+    for (int n = 0; n < NV; ++n) {
+        const int c = (gl + n * 32 * GW) * V;
+#pragma unroll
+        for (int i = 0; i < V; ++i) x[n].f[i] = 0.f;
+        if (live && c < W) x[n] = xe ? ldv<T, V>(xe + c) : ldv<float, V>(p.x + src * W + c);
+    }
+    // The routed sublayer of a prompt gathers its rows by index: the other one first, so that its loads are on their way.
+#pragma unroll
+    for (int b = 0; b < 2; ++b) {
+        if (!p.b[b].y_f32 && !p.b[b].y) continue;
+#pragma unroll
+        for (int n = 0; n < NV; ++n) {
+            const int c = (gl + n * 32 * GW) * V;
+            if (!live || c >= W) continue;
+            const Vec<V> y = branch_cols<T, V>(p.b[b], src, W, c);
+            if (p.b[b].scale) {
+                if constexpr (!EARLY) s[b][n] = ldv<float, V>(p.b[b].scale + c);
+#pragma unroll
+                for (int i = 0; i < V; ++i) x[n].f[i] = fmaf(s[b][n].f[i], y.f[i], x[n].f[i]);
+            } else {
+#pragma unroll
+                for (int i = 0; i < V; ++i) x[n].f[i] += y.f[i];
+            }
+        }
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int n = 0; n < NV; ++n) {
+        const int c = (gl + n * 32 * GW) * V;
+#pragma unroll
+        for (int i = 0; i < V; ++i) ss = fmaf(x[n].f[i], x[n].f[i], ss);
+        if (live && c < W && p.x_out) stv<float, V>(p.x_out + (size_t)row * W + c, x[n]);
+    }
+    ss = warp_sum(ss);
+    if constexpr (GW > 1) {
+        if (lane == 0) red[warp] = ss;
+        __syncthreads();
+        ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < GW; ++i) ss += red[grp * GW + i];
+    }
+    const float inv = 1.f / sqrtf(ss / (float)W + p.eps);
+#pragma unroll
+    for (int o = 0; o < 2; ++o) {
+        if (!p.out[o]) continue;
+        T* out = reinterpret_cast<T*>(p.out[o]) + (size_t)row * W;
+#pragma unroll
+        for (int n = 0; n < NV; ++n) {
+            const int c = (gl + n * 32 * GW) * V;
+            if (!live || c >= W) continue;
+            if constexpr (!EARLY) w[o][n] = ldv<float, V>(p.w[o] + c);
+            Vec<V> v;
+#pragma unroll
+            for (int i = 0; i < V; ++i) v.f[i] = x[n].f[i] * (inv * w[o][n].f[i]);
+            stv<T, V>(out + c, v);
+        }
+    }
+}
+
+template <class T, int V>
+int launch_parallel_v(md_ctx* ctx, const md_parallel_glue& g) {
+    void (*kern)(md_parallel_glue) = nullptr;
+    const int per = 32 * V;   // columns a warp holds in one vector per lane
+    int gw = 16;
+    // few rows: the whole block on one row; many: as few warps per row as four vectors per lane allow
+    if (g.rows <= 296) {
+        kern = g.width <= 16 * per ? stack_parallel_kernel<T, V, 16, 1> : g.width <= 32 * per ? stack_parallel_kernel<T, V, 16, 2>
+             : g.width <= 64 * per ? stack_parallel_kernel<T, V, 16, 4> : stack_parallel_kernel<T, V, 16, 8>;
+    } else if (g.width <= 4 * per) {
+        kern = stack_parallel_kernel<T, V, 1, 4>, gw = 1;
+    } else if (g.width <= 8 * per) {
+        kern = stack_parallel_kernel<T, V, 2, 4>, gw = 2;
+    } else if (g.width <= 16 * per) {
+        kern = stack_parallel_kernel<T, V, 4, 4>, gw = 4;
+    } else if (g.width <= 32 * per) {
+        kern = stack_parallel_kernel<T, V, 8, 4>, gw = 8;
+    } else {
+        kern = g.width <= 64 * per ? stack_parallel_kernel<T, V, 16, 4> : stack_parallel_kernel<T, V, 16, 8>;
+    }
+    if (g.width > 128 * per) return md_fail(ctx, MD_ERR_UNSUPPORTED, "a width of %d exceeds %d", g.width, 128 * per);
+    const int groups = 16 / gw;
+    return md_launch_ex(ctx, kern, dim3((unsigned)((g.rows + groups - 1) / groups)), dim3(PAR_THREADS), 0, "stack_parallel_kernel", g);
+}
+
+template <class T>
+int launch_parallel(md_ctx* ctx, const md_parallel_glue& g) {
+    return (g.width % 4) == 0 ? launch_parallel_v<T, 4>(ctx, g) : launch_parallel_v<T, 1>(ctx, g);
+}
+
 }  // namespace
 
 int md_launch_glue(md_ctx* ctx, int dtype, const md_glue& g) {
     return dtype == MD_DTYPE_F32 ? launch_glue<float>(ctx, g) : launch_glue<__nv_bfloat16>(ctx, g);
+}
+
+int md_launch_parallel_glue(md_ctx* ctx, int dtype, const md_parallel_glue& g) {
+    return dtype == MD_DTYPE_F32 ? launch_parallel<float>(ctx, g) : launch_parallel<__nv_bfloat16>(ctx, g);
 }
 
 int md_launch_argmax_f32(md_ctx* ctx, const float* x, size_t n, size_t stride, size_t rows, unsigned long long* idx_dev) {

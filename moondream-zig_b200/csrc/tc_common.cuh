@@ -239,6 +239,14 @@ __device__ __forceinline__ float fast_gelu_tanh(float z) {   // 0.5 z (1 + tanh 
     return z * fast_logistic(1.5957691216057308f * (z + 0.044715f * z * z * z));
 }
 __device__ __forceinline__ float fast_act(int act, float z) { return act == MD_ACT_SILU ? fast_silu(z) : fast_gelu_tanh(z); }
+// md_gated of an md_lin
+__device__ __forceinline__ float fast_gated(const md_lin& ep, float g, float u) {
+    if (ep.glu == MD_ACT_CLAMPED) {
+        g = fminf(g, ep.glu_limit);
+        return g * fast_logistic(ep.glu_alpha * g) * (fminf(fmaxf(u, -ep.glu_limit), ep.glu_limit) + 1.f);
+    }
+    return fast_act(ep.glu, g) * u;
+}
 
 // md_lin on 8 consecutive output columns of one row: f32 accumulators in, four packed bfloat16 pairs out.  N % 8 == 0.
 __device__ __forceinline__ void lin_glue8(const uint32_t* acc_bits, const md_lin& ep, int cq, int N, uint32_t (&pk)[4]) {
@@ -272,11 +280,11 @@ __device__ __forceinline__ void lin_glue8(const uint32_t* acc_bits, const md_lin
     for (int j = 0; j < 4; ++j) pk[j] = md_pack_bf16(v[2 * j], v[2 * j + 1]);
 }
 // 8 columns of a gated product: gate and up accumulators in
-__device__ __forceinline__ void glu_glue8(const uint32_t* gate, const uint32_t* up, int act, uint32_t (&pk)[4]) {
+__device__ __forceinline__ void glu_glue8(const uint32_t* gate, const uint32_t* up, const md_lin& ep, uint32_t (&pk)[4]) {
 #pragma unroll
     for (int j = 0; j < 4; ++j)
-        pk[j] = md_pack_bf16(fast_act(act, __uint_as_float(gate[2 * j])) * __uint_as_float(up[2 * j]),
-                             fast_act(act, __uint_as_float(gate[2 * j + 1])) * __uint_as_float(up[2 * j + 1]));
+        pk[j] = md_pack_bf16(fast_gated(ep, __uint_as_float(gate[2 * j]), __uint_as_float(up[2 * j])),
+                             fast_gated(ep, __uint_as_float(gate[2 * j + 1]), __uint_as_float(up[2 * j + 1])));
 }
 
 // Shared-memory matrix descriptor (version 1, sm_100) as built by desc_lo / desc_hi:

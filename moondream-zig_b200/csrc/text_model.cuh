@@ -69,6 +69,9 @@ struct PdlScope {
     ~PdlScope() { c->pdl = old; }
 };
 
+// The second stream of a layer that runs as two chains of kernels, and its events (model.cu).
+int md_side_stream(md_ctx* ctx);
+
 // ---- stack.cu ----------------------------------------------------------------------------------------------
 int md_stack_destroy(md_stack* s);
 int md_stack_request_create(md_text_request* req);

@@ -16,27 +16,7 @@ from __future__ import annotations
 import numpy as np
 
 from .models import (ACT_GELU_TANH, ACT_SILU, FF_DENSE, FF_MOE, FF_NONE, MIXER_LIGHTNING, MIXER_WINDOW_ATTENTION,
-                     StackModel, register_model)
-
-GLU_BLOCK = 32
-
-
-def _pad_rows(a: np.ndarray, multiple: int) -> np.ndarray:
-    short = -a.shape[0] % multiple
-    return np.concatenate([a, np.zeros((short,) + a.shape[1:], a.dtype)]) if short else a
-
-
-def gate_up(gate: np.ndarray, up: np.ndarray) -> np.ndarray:
-    """[ff, K] x 2 -> [2 * ff_pad, K]: blocks of 32 gate rows and the 32 up rows beside them."""
-    gate, up = _pad_rows(gate, GLU_BLOCK), _pad_rows(up, GLU_BLOCK)
-    k = gate.shape[1]
-    return np.stack([gate.reshape(-1, GLU_BLOCK, k), up.reshape(-1, GLU_BLOCK, k)], 1).reshape(-1, k)
-
-
-def down(w: np.ndarray) -> np.ndarray:
-    """[width, ff] -> [width, ff_pad]."""
-    return np.ascontiguousarray(_pad_rows(w.T, GLU_BLOCK).T)
-
+                     StackModel, down, gate_up, pad_rows as _pad_rows, register_model)
 
 def _per_head(v, heads: int) -> np.ndarray:
     a = np.asarray(v, np.float32).reshape(-1)

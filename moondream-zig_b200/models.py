@@ -197,9 +197,31 @@ class TextModel:
 # ---------------------------------------------------------------- layer-stack decoders
 
 DTYPES = {"bfloat16": 1, "float32": 2}
-MIXER_WINDOW_ATTENTION, MIXER_LIGHTNING = 1, 2
+MIXER_WINDOW_ATTENTION, MIXER_LIGHTNING, MIXER_LATENT_ATTENTION = 1, 2, 3
 FF_NONE, FF_DENSE, FF_MOE = 0, 1, 2
-ACT_GELU_TANH, ACT_SILU = 1, 2
+ACT_GELU_TANH, ACT_SILU, ACT_CLAMPED = 1, 2, 3
+LAYER_SANDWICH, LAYER_PARALLEL = 0, 1
+ROUTER_LOGISTIC, ROUTER_SOFTMAX = 0, 1
+
+
+GLU_BLOCK = 32
+
+
+def pad_rows(a: np.ndarray, multiple: int) -> np.ndarray:
+    short = -a.shape[0] % multiple
+    return np.concatenate([a, np.zeros((short,) + a.shape[1:], a.dtype)]) if short else a
+
+
+def gate_up(gate: np.ndarray, up: np.ndarray) -> np.ndarray:
+    """[ff, K] x 2 -> [2 * ff_pad, K]: blocks of 32 gate rows and the 32 up rows beside them."""
+    gate, up = pad_rows(gate, GLU_BLOCK), pad_rows(up, GLU_BLOCK)
+    k = gate.shape[1]
+    return np.stack([gate.reshape(-1, GLU_BLOCK, k), up.reshape(-1, GLU_BLOCK, k)], 1).reshape(-1, k)
+
+
+def down(w: np.ndarray) -> np.ndarray:
+    """[width, ff] -> [width, ff_pad]."""
+    return np.ascontiguousarray(pad_rows(w.T, GLU_BLOCK).T)
 
 
 class _StackLayer(C.Structure):
@@ -210,7 +232,12 @@ class _StackLayer(C.Structure):
                 [(n, C.c_void_p) for n in ("w_out", "norm1", "norm1b", "norm2", "norm2b", "conv1", "conv2")] +
                 [("act", C.c_int), ("ff_dim", C.c_size_t), ("ff_pad", C.c_size_t)] +
                 [(n, C.c_void_p) for n in ("w_gate_up", "w_down", "router")] +
-                [("experts", C.c_size_t), ("top", C.c_size_t)])
+                [("experts", C.c_size_t), ("top", C.c_size_t), ("form", C.c_int), ("router_kind", C.c_int), ("ls1", C.c_void_p),
+                 ("ls2", C.c_void_p), ("act_limit", C.c_float), ("act_alpha", C.c_float), ("shared_ff", C.c_size_t),
+                 ("shared_pad", C.c_size_t), ("shared_limit", C.c_float), ("shared_gate_up", C.c_void_p),
+                 ("shared_down", C.c_void_p), ("q_rank", C.c_size_t), ("kv_rank", C.c_size_t), ("rot_dim", C.c_size_t),
+                 ("rope_base", C.c_float)] +
+                [(n, C.c_void_p) for n in ("q_norm", "kv_norm", "sink", "w_uq", "w_ukv", "w_ukt")])
 
 
 class _StackW(C.Structure):
@@ -222,44 +249,60 @@ class _StackW(C.Structure):
 class StackModel(TextModel):
     """A text model described layer by layer (md_stack_model_create).  `layers`: one dict per layer with the fields of
     md_stack_layer; arrays may be numpy (uint16 = bfloat16 bits, or floats) or CUDA torch tensors already of the model's
-    type, which are used in place."""
+    type, which are used in place.  An array that several layers name is uploaded once.  head None: the embedding table."""
     logits_dtype = np.float32
-    VECTORS = ("r1", "r2", "decay", "mix_norm", "b_in", "norm1", "norm1b", "norm2", "norm2b", "conv1", "conv2")
-    MATRICES = ("w_in", "w_out", "w_gate_up", "w_down", "router")
+    VECTORS = ("r1", "r2", "decay", "mix_norm", "b_in", "norm1", "norm1b", "norm2", "norm2b", "conv1", "conv2", "ls1", "ls2",
+               "q_norm", "kv_norm", "sink")
+    MATRICES = ("w_in", "w_out", "w_gate_up", "w_down", "router", "shared_gate_up", "shared_down", "w_uq", "w_ukv", "w_ukt")
+    SIZES = ("kv_heads", "window", "keep_first", "act", "ff_dim", "experts", "top", "form", "router_kind", "shared_ff", "q_rank",
+             "kv_rank", "rot_dim")
+    FLOATS = ("scale", "act_limit", "act_alpha", "shared_limit", "rope_base")
 
-    def __init__(self, ctx, layers: list, embed, head, final_norm, eps: float, residual_mult: float, taps: int,
+    def __init__(self, ctx, layers: list, embed, head, final_norm, eps: float, residual_mult: float = 1.0, taps: int = 1,
                  dtype: str = "bfloat16", max_seq: int = 2048):
         if dtype not in DTYPES:
             raise ValueError(f"dtype {dtype!r}: expected one of {sorted(DTYPES)}")
         self.ctx, self.lib, self.dtype = ctx, ctx.lib, dtype
-        self.dev, self._keep, self._bufs = {}, [], []
+        self.dev, self._keep, self._bufs, self._uploaded = {}, [], [], {}
         table = (_StackLayer * len(layers))()
         for s, d in zip(table, layers):
             for n in ("mixer", "ff", "heads", "dim", "vdim"):
                 setattr(s, n, int(d[n]))
-            for n in ("kv_heads", "window", "keep_first", "act", "ff_dim", "experts", "top"):
+            for n in self.SIZES:
                 setattr(s, n, int(d.get(n) or 0))
-            s.scale = float(d.get("scale") or 0.0)
+            for n in self.FLOATS:
+                setattr(s, n, float(d.get(n) or 0.0))
             s.in_rows = d["w_in"].shape[0]
             if d["ff"] != FF_NONE:
                 s.ff_pad = d["w_down"].shape[-1]
+            if d.get("shared_ff"):
+                s.shared_pad = d["shared_down"].shape[-1]
             for n in self.VECTORS:
                 if d.get(n) is not None:
-                    setattr(s, n, self._vector(d[n].T if n.startswith("conv") else d[n]))
+                    setattr(s, n, self._once(self._vector, d[n], n.startswith("conv")))
             for n in self.MATRICES:
                 if d.get(n) is not None:
-                    setattr(s, n, self._matrix(d[n]))
+                    setattr(s, n, self._once(self._matrix, d[n]))
         w = _StackW()
         w.dtype, w.n_layers, w.width, w.vocab, w.max_seq, w.taps = (DTYPES[dtype], len(layers), embed.shape[1],
                                                                     embed.shape[0], max_seq, taps)
         w.eps, w.residual_mult = eps, residual_mult
         w.layers = C.cast(table, C.c_void_p)
-        w.embed, w.head, w.final_norm = self._matrix(embed), self._matrix(head), self._vector(final_norm)
+        w.embed = self._matrix(embed)
+        w.head, w.final_norm = w.embed if head is None else self._matrix(head), self._vector(final_norm)
         self.s = w
         self.dim, self.vocab, self.n_layers = int(w.width), int(w.vocab), int(w.n_layers)
         h = C.c_void_p()
         ctx._check(self.lib.md_stack_model_create(ctx.h, C.byref(w), C.byref(h)))
         self.h = h
+        self._uploaded = {}
+
+    def _once(self, upload, a, transposed: bool = False):
+        """Device address of an array that several layers may share."""
+        key = (id(a), upload.__name__, transposed)
+        if key not in self._uploaded:
+            self._uploaded[key] = (upload(a.T if transposed else a), a)   # the reference keeps the id in use
+        return self._uploaded[key][0]
 
     @staticmethod
     def widen(a: np.ndarray) -> np.ndarray:
@@ -325,7 +368,7 @@ def register_model(name: str):
 
 def load_model(ctx, folder: str, dtype: str = "bfloat16", max_seq: int = 2048):
     """The text model of a folder: config.json + model.safetensors of a registered architecture, or moondream.bin."""
-    from . import korupel, weights  # noqa: F401  (registers its architecture)
+    from . import korupel, nuvezen, weights  # noqa: F401  (each design registers its architecture)
     path = os.path.join(folder, "config.json")
     if not os.path.exists(path) and os.path.exists(os.path.join(folder, "moondream.bin")):
         return weights.WeightFile(os.path.join(folder, "moondream.bin")).upload(ctx).text_model()
