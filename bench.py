@@ -597,6 +597,11 @@ ONLY_CASES = {
     "korupel_prefill": "layer-stack decoder, width 2048, six layers, 761-token prompt, three passes",
     "korupel_decode": "layer-stack decoder, width 2048, six layers, 761-token prompt then 24 steps",
     "korupel_decode8": "layer-stack decoder, width 2048, six layers, eight requests batched, 761-token prompts then 24 steps",
+    "nuvezen": "layer-stack decoder (Nuvezen design) beside the Korupel design at equal size: prefill and decode",
+    "nuvezen_prefill": "Nuvezen design, width 2048, six layers, 761-token prompt, three passes",
+    "nuvezen_prefill2048": "Nuvezen design, width 2048, six layers, 2048-token prompt, three passes",
+    "nuvezen_decode": "Nuvezen design, width 2048, six layers, 761-token prompt then 24 steps",
+    "nuvezen_decode8": "Nuvezen design, width 2048, six layers, eight requests batched, 761-token prompts then 24 steps",
     "vision1": "vision encode + projection, one crop, three passes",
     "vision13": "vision encode + projection, thirteen crops, three passes",
 }
@@ -667,21 +672,22 @@ def run_only(ctx, torch, stream, case):
             r.close()
         tm.close()
         return out
-    if case == "korupel":
-        return korupel_case(ctx, torch)
-    if case.startswith("korupel_"):
-        m = build_stack_model(ctx, torch, g, STACK_SIZES["2048"], 6)
+    if case in ("korupel", "nuvezen"):
+        return stack_case(ctx, torch, case)
+    if case.startswith(("korupel_", "nuvezen_")):
+        design, what = case.split("_")
+        m = STACK_DESIGNS[design][1](ctx, torch, g, STACK_DESIGNS[design][0]["2048"], 6)
         batch = 8 if case.endswith("8") else 1
         reqs = [m.request() for _ in range(batch)]
-        ids = np.random.default_rng(4100).integers(0, m.vocab, 761)
-        for _ in range(3 if case == "korupel_prefill" else 1):
+        ids = np.random.default_rng(4100).integers(0, m.vocab, 2048 if what.endswith("2048") else 761)
+        for _ in range(3 if what.startswith("prefill") else 1):
             for r in reqs:
                 r.reset()
                 t0 = time.perf_counter()
                 m.step(r, ids, want_token=True)
                 ms = (time.perf_counter() - t0) * 1e3
         out = {"prefill_ms": round(ms, 3)}
-        if case != "korupel_prefill":
+        if not what.startswith("prefill"):
             t0 = time.perf_counter()
             m.generate_batch(reqs, [1] * batch, 24)
             out["us_per_step"] = round((time.perf_counter() - t0) / 24 * 1e6, 1)
@@ -701,8 +707,8 @@ def run_only(ctx, torch, stream, case):
     return {"crops": crops, "encode_ms": round(ms, 3)}
 
 
-# The layer-stack decoder at sizes of a real model's layers.  A layer's active weights equal those of a Phi layer of the
-# same width (12 width^2): 5 width^2 in the mixer, 7 width^2 in the feed-forward (of one token, for experts).
+# The layer-stack decoders at sizes of a real model's layers.  A layer's active weights equal those of a Phi layer of the
+# same width (12 width^2).  Korupel: 5 width^2 in the mixer, 7 width^2 in the feed-forward (of one token, for experts).
 STACK_SIZES = {
     "2048": dict(width=2048, heads=32, kv_heads=8, dim=64, vdim=64, window=1024, keep=4, experts=16, top=2),
     "4096": dict(width=4096, heads=32, kv_heads=8, dim=128, vdim=128, window=1024, keep=4, experts=8, top=2),
@@ -746,9 +752,53 @@ def build_stack_model(ctx, torch, g, z, layers, ff=("dense", "moe"), max_seq=256
                              taps=taps, max_seq=max_seq)
 
 
-def korupel_case(ctx, torch):
-    """Prefill and decode throughput of the layer-stack decoder and of the Phi-style decoder with as many layers of the same
-    width, vocabulary and active weights.  Host wall clock around the library's calls (ids or embeddings copied up, tokens
+# Nuvezen: about 3 (2048) or 2.3 (4096) width^2 in the mixer, the rest in the feed-forward (of one token: the chosen experts
+# and the shared one, all of one size).
+NUVEZEN_SIZES = {
+    "2048": dict(width=2048, heads=16, dim=128, rot=64, vdim=128, q_rank=1024, kv_rank=512, window=1024, experts=16, top=2, ff=6144),
+    "4096": dict(width=4096, heads=32, dim=128, rot=64, vdim=128, q_rank=1536, kv_rank=512, window=1024, experts=8, top=2, ff=13152),
+}
+
+
+def build_nuvezen_model(ctx, torch, g, z, layers, ff=("dense", "moe"), max_seq=2560, vocab=51200):
+    """Random-init Nuvezen-design decoder generated on the device; feed-forwards alternate between dense and mixture of
+    experts with a shared one."""
+    import importlib
+    import __graft_entry__ as entry
+    models = importlib.import_module(entry.PKG_NAME + ".models")
+    W, H, d, rot, e, Q, R = (z[k] for k in ("width", "heads", "dim", "rot", "vdim", "q_rank", "kv_rank"))
+
+    def n(*shape, std=0.02):
+        return (torch.randn(*shape, device="cuda", generator=g) * std).bfloat16()
+
+    def vec(*shape, mean=1.0, std=0.1):
+        return torch.randn(*shape, device="cuda", generator=g) * std + mean
+    out = []
+    for i in range(layers):
+        uk, uv = n(H, d, R), n(H * e, R)
+        s = {"form": models.LAYER_PARALLEL, "mixer": models.MIXER_LATENT_ATTENTION, "norm1": vec(W), "norm2": vec(W),
+             "ls1": vec(W, mean=0.5), "ls2": vec(W, mean=0.5), "heads": H, "dim": d, "vdim": e, "rot_dim": rot, "q_rank": Q,
+             "kv_rank": R, "scale": (d + rot) ** -0.5, "window": z["window"], "rope_base": 10000.0, "w_in": n(Q + R + rot, W),
+             "w_out": n(W, H * e), "w_uq": n(H * (d + rot), Q), "w_ukv": torch.cat([uk.reshape(H * d, R), uv]),
+             "w_ukt": uk.transpose(1, 2).contiguous(), "q_norm": vec(Q), "kv_norm": vec(R), "sink": vec(H, mean=0.0)}
+        if ff[i % len(ff)] == "dense":
+            F = z["ff"]
+            s.update(ff=models.FF_DENSE, act=models.ACT_SILU, ff_dim=F, w_gate_up=n(2 * F, W), w_down=n(W, F))
+        else:
+            E, F = z["experts"], z["ff"] // (z["top"] + 1) // 32 * 32
+            s.update(ff=models.FF_MOE, act=models.ACT_CLAMPED, act_limit=2.0, act_alpha=1.702, ff_dim=F, experts=E, top=z["top"],
+                     router_kind=models.ROUTER_SOFTMAX, router=n(E + 1, W), w_gate_up=n(E, 2 * F, W), w_down=n(E, W, F),
+                     shared_ff=F, shared_limit=1.0, shared_gate_up=n(2 * F, W), shared_down=n(W, F))
+        out.append(s)
+    return models.StackModel(ctx, out, embed=n(vocab, W), head=None, final_norm=vec(W), eps=1e-5, max_seq=max_seq)
+
+
+STACK_DESIGNS = {"korupel": (STACK_SIZES, build_stack_model), "nuvezen": (NUVEZEN_SIZES, build_nuvezen_model)}
+
+
+def stack_case(ctx, torch, design):
+    """Prefill and decode throughput of a layer-stack decoder and of its closest model (the Phi-style decoder, or the Korupel
+    design) with as many layers of the same width, vocabulary and active weights.  Host wall clock around the library's calls (ids or embeddings copied up, tokens
     read back), best of the repetitions that replay recorded graphs."""
     import importlib
     import __graft_entry__ as entry
@@ -764,12 +814,12 @@ def korupel_case(ctx, torch):
         return min(times[2:])
 
     for name, layers in (("2048", 12), ("4096", 6)):
-        z = STACK_SIZES[name]
-        W = z["width"]
+        W = int(name)
         rows = {}
-        for ff in (("dense",), ("moe",)):
+        runs = [(kind, ff) for kind in (["nuvezen", "korupel"] if design == "nuvezen" else ["korupel"]) for ff in (("dense",), ("moe",))]
+        for kind, ff in runs:
             g = torch.Generator(device="cuda").manual_seed(4200)
-            m = build_stack_model(ctx, torch, g, z, layers, ff=ff)
+            m = STACK_DESIGNS[kind][1](ctx, torch, g, STACK_DESIGNS[kind][0][name], layers, ff=ff)
             reqs = [m.request() for _ in range(8)]
             r, res = reqs[0], {}
             for n in (761, 2048):
@@ -788,12 +838,15 @@ def korupel_case(ctx, torch):
                     m.step(q, np.arange(761))
                 return round(batch * 200 / best(fn, 4), 1)
             res["decode_1"], res["decode_8"] = decode(1), decode(8)
-            rows["korupel_" + ff[0]] = res
+            rows[f"{kind}_{ff[0]}"] = res
             for q in reqs:
                 q.close()
             m.close()
             del m, reqs, r
             torch.cuda.empty_cache()
+        if design == "nuvezen":
+            out[f"width_{name}_layers_{layers}"] = rows
+            continue
         g = torch.Generator(device="cuda").manual_seed(4300)
 
         def n(*shape, std=0.02):

@@ -162,3 +162,75 @@ def forward(cfg, w, tokens, want_layers=False):
         streams.append(x)
     logits = rms_norm_zero(x, w["final.norm"], eps) @ embed.T
     return (logits, np.stack(streams)) if want_layers else logits
+
+
+# ---------------------------------------------------------------- synthetic models for the tests
+
+def to_bf16(a):
+    """Round to bfloat16 (nearest even), returned as float32."""
+    u = np.ascontiguousarray(a, np.float32).view(np.uint32)
+    return ((u + 0x7FFF + ((u >> 16) & 1)) & 0xFFFF0000).astype(np.uint32).view(np.float32)
+
+
+def random_weights(cfg, seed):
+    """Random weights for a configuration (bfloat16 values held as float32), sized so that the activations stay of order one,
+    the experts' clamps take part and every mechanism has a visible share of the output.  Which experts a token takes must
+    not hang on rounding: the first channels (one per expert) carry a pattern of the token's own that no sublayer writes to,
+    and the routers read mostly those."""
+    rng = np.random.default_rng(seed)
+    W, V = cfg["width"], cfg["vocab"]
+    w = {}
+
+    def lin(name, n_out, n_in, gain=1.0):
+        w[name] = rng.standard_normal((n_out, n_in)) * (gain / np.sqrt(n_in))
+
+    def vec(name, n, lo, hi):
+        w[name] = rng.uniform(lo, hi, n)
+
+    w["embed"] = 0.4 * rng.standard_normal((V, W))     # also the head: small, or every token would predict itself
+    moes = [l["mlp"] for l in cfg["layers"] if l["mlp"] and l["mlp"]["kind"] == "moe"]
+    R = max((m["router"]["experts"] for m in moes), default=0)
+    if R:   # ranks of the experts per token, in clear steps
+        order = np.argsort(rng.standard_normal((V, R)), axis=1)
+        w["embed"][:, :R] = 1.5 - 3.0 * order / max(R - 1, 1)
+    for i, layer in enumerate(cfg["layers"]):
+        if layer.get("weights_of") is not None:
+            continue
+        p, m, mlp = f"l{i}.", layer["mixer"], layer["mlp"]
+        H, d, r, e = m["heads"], m["dim"], m["rot_dim"], m["vdim"]
+        vec(p + "norm1", W, -0.4, 0.4)
+        vec(p + "ls1", W, 0.5, 1.1)
+        w[p + "ls1"][:R] = 0
+        lin(p + "mix.dq", m["q_rank"], W)
+        lin(p + "mix.dkv", m["kv_rank"] + r, W)
+        w[p + "mix.dkv"][m["kv_rank"]:] *= 1.5
+        vec(p + "mix.dq.norm", m["q_rank"], 0.6, 1.4)
+        vec(p + "mix.dkv.norm", m["kv_rank"], 0.6, 1.4)
+        lin(p + "mix.uq", H * (d + r), m["q_rank"], 1.5)
+        lin(p + "mix.uk", H * d, m["kv_rank"], 1.5)
+        lin(p + "mix.uv", H * e, m["kv_rank"], 1.5)
+        vec(p + "mix.sink", H, -1.0, 2.5)
+        lin(p + "mix.o", W, H * e, 1.5)
+        if mlp is None:
+            continue
+        q = p + "mlp."
+        vec(p + "norm2", W, -0.4, 0.4)
+        w[p + "norm2"][:R] = 0
+        vec(p + "ls2", W, 0.5, 1.1)
+        w[p + "ls2"][:R] = 0
+        if mlp["kind"] == "dense":
+            F = mlp["ff"]
+            lin(q + "gate", F, W); lin(q + "up", F, W); lin(q + "down", W, F, 1.5)
+            continue
+        E = mlp["router"]["experts"]
+        lin(q + "router", E, W, 0.015)
+        w[q + "router"][:, :R] = 2.0 * np.eye(E, R)
+        parts = [(f"e{n}.", mlp["expert"]["ff"]) for n in range(E)]
+        if mlp.get("shared"):
+            parts.append(("shared.", mlp["shared"]["ff"]))
+            lin(q + "shared.sg", 1, W)
+        for n, F in parts:
+            lin(q + n + "gate", F, W, 1.5); lin(q + n + "up", F, W, 1.5); lin(q + n + "down", W, F)
+    vec("final.norm", W, -0.4, 0.4)
+    w["final.norm"][:R] = -1
+    return {k: to_bf16(v) for k, v in w.items()}
