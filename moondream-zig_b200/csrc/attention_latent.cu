@@ -7,11 +7,13 @@
 //   latent_prefill_kernel   bfloat16 prompts: keys and values of the visible tokens come expanded from one product; 64 queries
 //                           x 64 keys per step on tensor cores.  The query's rotation happens on its way to shared memory.
 //                           Weights enter the second product as two bfloat16 terms (mma_bf16.cuh).
-//   latent_heads_kernel     bfloat16, one token per sequence: per-head products (the query into the latent space, the weighted
-//                           latent into the values), weights streamed as in gemv.cu
-//   latent_decode_kernel    bfloat16, one token per sequence: 16 heads share every latent they read; the blocks of a cluster
-//                           take parts of the window and merge through distributed shared memory
+//   latent_query_kernel     bfloat16, one token per sequence: norms, the queries' product and the append to the cache
+//   latent_absorb_kernel    bfloat16, one token per sequence: the query into the latent space, per head
+//   latent_decode_kernel    bfloat16, one token per sequence: 16 heads share every latent they read; blocks take parts of the
+//                           window
+//   latent_value_kernel     bfloat16, one token per sequence: merges the parts (and the sink), the weighted latent into the values
 #include "mma_bf16.cuh"
+#include "tc_common.cuh"
 
 #include <algorithm>
 
@@ -194,7 +196,7 @@ latent_prefill_kernel(const __grid_constant__ md_latent p, int key0) {
     using namespace mb;
     constexpr int KP = DK + 8, VP = DV + 8;
     constexpr bool Q_REGS = DK <= 128;    // longer heads re-read their query fragments from shared memory
-    extern __shared__ __align__(16) unsigned char smem[];
+    extern __shared__ __align__(128) unsigned char smem[];
     __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(smem);    // [BQ][KP]
     __nv_bfloat16* Ks = Qs + BQ * KP;                               // two tiles [BK][KP]
     __nv_bfloat16* Vs = Ks + 2 * BK * KP;                           // two tiles [BK][VP]
@@ -367,225 +369,361 @@ __device__ __forceinline__ uint4 ld_act(const void* p) {
     return v;
 }
 
-// out[s][h][n] = sum_k w[h][n][k] x[s][h][k]; K % 8 == 0.  Strides in elements.
-struct HeadsProduct {
-    const __nv_bfloat16 *w, *x;
-    __nv_bfloat16* out;
-    int N, K, seqs;
-    int x_seq, x_head, out_seq, out_head;
-    // rot > 0: the first block of a head also turns x[s][h][K .. K + rot) into out[s][h][N .. N + rot)
-    int rot;
-    const float* rope;
-    const int* pos[MD_STACK_MAX_SEQS];
-};
-constexpr int HEADS_WARPS = 4, HEADS_UNROLL = 4;
+// The query in the latent space: qa[s][h][r] = sum_d w_ukt[h][r][d] q[s][h][d]; the first block of a head also rotates the rotated
+// part behind it.
+constexpr int HEADS_WARPS = 4;
 
 __global__ void __launch_bounds__(HEADS_WARPS * 32)
-latent_heads_kernel(const __grid_constant__ HeadsProduct p) {
+latent_absorb_kernel(const __grid_constant__ md_latent p) {
     __shared__ float partial[HEADS_WARPS][16][8];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
-    const int row0 = blockIdx.x * 16, h = blockIdx.y;
-    const __nv_bfloat16* w = p.w + (size_t)h * p.N * p.K + t * 8;
-    const __nv_bfloat16 *w_lo = w + (size_t)min(row0 + g, p.N - 1) * p.K, *w_hi = w + (size_t)min(row0 + g + 8, p.N - 1) * p.K;
+    const int R = p.kv_rank, D = p.dim, rot = p.rot, row0 = blockIdx.x * 16, h = blockIdx.y;
+    const __nv_bfloat16* w = reinterpret_cast<const __nv_bfloat16*>(p.w_ukt) + (size_t)h * R * D + t * 8;
+    const __nv_bfloat16 *w_lo = w + (size_t)min(row0 + g, R - 1) * D, *w_hi = w + (size_t)min(row0 + g + 8, R - 1) * D;
     const bool has_x = g < p.seqs;
-    const __nv_bfloat16* x = p.x + (size_t)(has_x ? g : 0) * p.x_seq + (size_t)h * p.x_head + t * 8;
+    const __nv_bfloat16* q = reinterpret_cast<const __nv_bfloat16*>(p.q) + (size_t)h * (D + rot);   // of sequence 0
+    const int q_seq = p.heads * (D + rot);
+    const __nv_bfloat16* x = q + (size_t)(has_x ? g : 0) * q_seq + t * 8;
+    __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(p.qa) + (size_t)h * (R + rot);
+    const int out_seq = p.heads * (R + rot);
     const uint4 zero = make_uint4(0, 0, 0, 0);
     float acc[4] = {0.f, 0.f, 0.f, 0.f};
     md_pdl_launch_dependents();
-    bool waited = false;
-    for (int k0 = warp * 32; k0 < p.K; k0 += HEADS_UNROLL * HEADS_WARPS * 32) {
-        uint4 lo[HEADS_UNROLL], hi[HEADS_UNROLL], xv[HEADS_UNROLL];
+    constexpr int U = 2;               // head sizes up to 256
+    uint4 lo[U], hi[U];
 #pragma unroll
-        for (int u = 0; u < HEADS_UNROLL; ++u) {
-            const int k = k0 + u * HEADS_WARPS * 32;
-            const bool live = k + t * 8 < p.K;
-            lo[u] = live ? ldg_stream(w_lo + k) : zero;
-            hi[u] = live ? ldg_stream(w_hi + k) : zero;
-        }
-        if (!waited) md_pdl_wait();
-        waited = true;
-#pragma unroll
-        for (int u = 0; u < HEADS_UNROLL; ++u) {
-            const int k = k0 + u * HEADS_WARPS * 32;
-            xv[u] = has_x && k + t * 8 < p.K ? ld_act(x + k) : zero;
-        }
-#pragma unroll
-        for (int u = 0; u < HEADS_UNROLL; ++u) {
-            mb::mma(acc, lo[u].x, hi[u].x, lo[u].y, hi[u].y, xv[u].x, xv[u].y);
-            mb::mma(acc, lo[u].z, hi[u].z, lo[u].w, hi[u].w, xv[u].z, xv[u].w);
-        }
+    for (int u = 0; u < U; ++u) {
+        const int k = warp * 32 + u * HEADS_WARPS * 32;
+        const bool live = k + t * 8 < D;
+        lo[u] = live ? ldg_stream(w_lo + k) : zero;
+        hi[u] = live ? ldg_stream(w_hi + k) : zero;
     }
-    if (!waited) md_pdl_wait();
+    md_pdl_wait();
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+        const int k = warp * 32 + u * HEADS_WARPS * 32;
+        const uint4 xv = has_x && k + t * 8 < D ? ld_act(x + k) : zero;
+        mb::mma(acc, lo[u].x, hi[u].x, lo[u].y, hi[u].y, xv.x, xv.y);
+        mb::mma(acc, lo[u].z, hi[u].z, lo[u].w, hi[u].w, xv.z, xv.w);
+    }
     partial[warp][g][2 * t] = acc[0];
     partial[warp][g][2 * t + 1] = acc[1];
     partial[warp][g + 8][2 * t] = acc[2];
     partial[warp][g + 8][2 * t + 1] = acc[3];
     __syncthreads();
     const int m = tid >> 4, e = tid & 15;      // 128 threads: 8 sequences x 16 rows
-    if (m < p.seqs && row0 + e < p.N) {
+    if (m < p.seqs && row0 + e < R) {
         float v = 0.f;
 #pragma unroll
         for (int i = 0; i < HEADS_WARPS; ++i) v += partial[i][e][m];
-        p.out[(size_t)m * p.out_seq + (size_t)h * p.out_head + row0 + e] = __float2bfloat16_rn(v);
+        out[(size_t)m * out_seq + row0 + e] = __float2bfloat16_rn(v);
     }
     if (blockIdx.x == 0)
-        for (int i = tid; i < p.seqs * (p.rot / 2); i += HEADS_WARPS * 32) {
-            const int s = i / (p.rot / 2), c = i % (p.rot / 2);
-            const float2 cs = *reinterpret_cast<const float2*>(p.rope + ((size_t)*p.pos[s] * (p.rot / 2) + c) * 2);
-            const uint32_t uv = __ldcg(reinterpret_cast<const uint32_t*>(p.x + (size_t)s * p.x_seq + (size_t)h * p.x_head + p.K + 2 * c));
+        for (int i = tid; i < p.seqs * (rot / 2); i += HEADS_WARPS * 32) {
+            const int s = i / (rot / 2), c = i % (rot / 2);
+            const float2 cs = *reinterpret_cast<const float2*>(p.rope + ((size_t)*p.pos_dev[s] * (rot / 2) + c) * 2);
+            const uint32_t uv = __ldcg(reinterpret_cast<const uint32_t*>(q + (size_t)s * q_seq + D + 2 * c));
             const float u = __uint_as_float(uv << 16), v = __uint_as_float(uv & 0xffff0000u);
-            *reinterpret_cast<uint32_t*>(p.out + (size_t)s * p.out_seq + (size_t)h * p.out_head + p.N + 2 * c) =
-                md_pack_bf16(u * cs.x - v * cs.y, v * cs.x + u * cs.y);
+            *reinterpret_cast<uint32_t*>(out + (size_t)s * out_seq + R + 2 * c) = md_pack_bf16(u * cs.x - v * cs.y, v * cs.x + u * cs.y);
         }
 }
 
-constexpr int DEC_THREADS = 256, DEC_WARPS = 8, DEC_HEADS = 16, DEC_MAX_SPLITS = 8;
+// The start of a decode step: blocks x < rows / 16 compute q = w_uq cq with cq = rms(in[0 .. q_rank); q_norm) normed on the way
+// (the norm's factor is a number per token, applied to the sums), the last block of a sequence norms and rotates the new token's
+// latent and appends it to the cache.
+constexpr int UQ_WARPS = 8, UQ_UNROLL = 4;
 
-__device__ __forceinline__ void cluster_sync() {
-    asm volatile("barrier.cluster.arrive.release.aligned;\nbarrier.cluster.wait.acquire.aligned;" ::: "memory");
+__global__ void __launch_bounds__(UQ_WARPS * 32)
+latent_query_kernel(const __grid_constant__ md_latent p, int row_blocks) {
+    __shared__ float partial[UQ_WARPS][16][8], red[UQ_WARPS][8];
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+    const int Q = p.q_rank, R = p.kv_rank, rot = p.rot;
+    md_pdl_launch_dependents();
+    if ((int)blockIdx.x >= row_blocks) {
+        const int seq = blockIdx.x - row_blocks, pos = *p.pos_dev[seq];   // written by the kernel that ended the previous step
+        const __nv_bfloat16* in = reinterpret_cast<const __nv_bfloat16*>(p.in) + (size_t)seq * p.row_stride + Q;
+        md_pdl_wait();
+        float ss = 0.f;
+        for (int c = tid * 4; c < R; c += UQ_WARPS * 32 * 4) {
+            float f[4];
+            md_load4<__nv_bfloat16>(in + c, f);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) ss = fmaf(f[i], f[i], ss);
+        }
+        ss = warp_sum(ss);
+        if (lane == 0) red[warp][0] = ss;
+        __syncthreads();
+        ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < UQ_WARPS; ++i) ss += red[i][0];
+        const float inv = 1.f / sqrtf(ss / (float)R + p.eps);
+        __nv_bfloat16* cc = reinterpret_cast<__nv_bfloat16*>(p.cc[seq]) + (size_t)pos * R;
+        for (int c = tid * 4; c < R; c += UQ_WARPS * 32 * 4) {
+            float f[4], w[4];
+            md_load4<__nv_bfloat16>(in + c, f);
+            md_load4<float>(p.kv_norm + c, w);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) f[i] *= inv * w[i];
+            md_store4<__nv_bfloat16>(cc + c, f);
+        }
+        for (int i = tid; i < rot / 2; i += UQ_WARPS * 32) {
+            const float2 cs = *reinterpret_cast<const float2*>(p.rope + ((size_t)pos * (rot / 2) + i) * 2);
+            const uint32_t uv = __ldcg(reinterpret_cast<const uint32_t*>(in + R + 2 * i));
+            const float u = __uint_as_float(uv << 16), v = __uint_as_float(uv & 0xffff0000u);
+            reinterpret_cast<uint32_t*>(reinterpret_cast<__nv_bfloat16*>(p.kr[seq]) + (size_t)pos * rot)[i] =
+                md_pack_bf16(u * cs.x - v * cs.y, v * cs.x + u * cs.y);
+        }
+        return;
+    }
+    const int N = p.heads * (p.dim + rot), row0 = blockIdx.x * 16;
+    const __nv_bfloat16* w = reinterpret_cast<const __nv_bfloat16*>(p.w_uq) + t * 8;
+    const __nv_bfloat16 *w_lo = w + (size_t)min(row0 + g, N - 1) * Q, *w_hi = w + (size_t)min(row0 + g + 8, N - 1) * Q;
+    const bool has_x = g < p.seqs;
+    const __nv_bfloat16* x = reinterpret_cast<const __nv_bfloat16*>(p.in) + (size_t)(has_x ? g : 0) * p.row_stride + t * 8;
+    const float* nw = p.q_norm + t * 8;
+    const uint4 zero = make_uint4(0, 0, 0, 0);
+    float acc[4] = {0.f, 0.f, 0.f, 0.f}, ss = 0.f;
+    bool waited = false;
+    for (int k0 = warp * 32; k0 < Q; k0 += UQ_UNROLL * UQ_WARPS * 32) {
+        uint4 lo[UQ_UNROLL], hi[UQ_UNROLL], xv[UQ_UNROLL];
+        float4 n0[UQ_UNROLL], n1[UQ_UNROLL];
+#pragma unroll
+        for (int u = 0; u < UQ_UNROLL; ++u) {
+            const int k = k0 + u * UQ_WARPS * 32;
+            const bool live = k + t * 8 < Q;
+            lo[u] = live ? ldg_stream(w_lo + k) : zero;
+            hi[u] = live ? ldg_stream(w_hi + k) : zero;
+            n0[u] = n1[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (live) {
+                n0[u] = __ldg(reinterpret_cast<const float4*>(nw + k));
+                n1[u] = __ldg(reinterpret_cast<const float4*>(nw + k) + 1);
+            }
+        }
+        if (!waited) md_pdl_wait();
+        waited = true;
+#pragma unroll
+        for (int u = 0; u < UQ_UNROLL; ++u) {
+            const int k = k0 + u * UQ_WARPS * 32;
+            xv[u] = has_x && k + t * 8 < Q ? ld_act(x + k) : zero;
+        }
+#pragma unroll
+        for (int u = 0; u < UQ_UNROLL; ++u) {
+            const uint32_t v[4] = {xv[u].x, xv[u].y, xv[u].z, xv[u].w};
+            const float f[8] = {n0[u].x, n0[u].y, n0[u].z, n0[u].w, n1[u].x, n1[u].y, n1[u].z, n1[u].w};
+            uint32_t b[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const float a0 = __uint_as_float(v[i] << 16), a1 = __uint_as_float(v[i] & 0xffff0000u);
+                ss = fmaf(a0, a0, fmaf(a1, a1, ss));
+                b[i] = md_pack_bf16(a0 * f[2 * i], a1 * f[2 * i + 1]);
+            }
+            mb::mma(acc, lo[u].x, hi[u].x, lo[u].y, hi[u].y, b[0], b[1]);
+            mb::mma(acc, lo[u].z, hi[u].z, lo[u].w, hi[u].w, b[2], b[3]);
+        }
+    }
+    if (!waited) md_pdl_wait();
+    ss += __shfl_xor_sync(0xffffffffu, ss, 1);
+    ss += __shfl_xor_sync(0xffffffffu, ss, 2);
+    if (t == 0) red[warp][g] = ss;
+    partial[warp][g][2 * t] = acc[0];
+    partial[warp][g][2 * t + 1] = acc[1];
+    partial[warp][g + 8][2 * t] = acc[2];
+    partial[warp][g + 8][2 * t + 1] = acc[3];
+    __syncthreads();
+    const int m = tid >> 4, e = tid & 15;
+    if (tid < 128 && m < p.seqs && row0 + e < N) {
+        float v = 0.f, s2 = 0.f;
+#pragma unroll
+        for (int i = 0; i < UQ_WARPS; ++i) v += partial[i][e][m], s2 += red[i][m];
+        reinterpret_cast<__nv_bfloat16*>(p.q)[(size_t)m * N + row0 + e] = __float2bfloat16_rn(v / sqrtf(s2 / (float)Q + p.eps));
+    }
 }
-// f32 at this block's shared-memory address `addr`, of the cluster's block `rank`
-__device__ __forceinline__ float ld_peer(uint32_t addr, int rank) {
-    uint32_t a;
-    float v;
-    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(a) : "r"(addr), "r"(rank));
-    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(a) : "memory");
-    return v;
+
+constexpr int DEC_THREADS = 256, DEC_WARPS = 8, DEC_HEADS = 16, DEC_MAX_SPLITS = 32;
+
+__device__ __forceinline__ void bulk_load(uint32_t dst, const void* src, uint32_t bytes, uint32_t bar) {
+    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst), "l"(src),
+                 "r"(bytes), "r"(bar)
+                 : "memory");
 }
-__device__ __forceinline__ float2 ld_peer2(uint32_t addr, int rank) {
-    uint32_t a;
-    float2 v;
-    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(a) : "r"(addr), "r"(rank));
-    asm volatile("ld.shared::cluster.v2.f32 {%0, %1}, [%2];" : "=f"(v.x), "=f"(v.y) : "r"(a) : "memory");
-    return v;
+
+// What the blocks of a window leave for latent_value_kernel: unnormalised sums and their (maximum, sum of weights).
+struct LatentParts {
+    float* o;        // [seqs][heads][splits][kv_rank]
+    float2* ml;      // [seqs][heads][splits]
+    int splits;      // blocks a window is dealt to; those past its last tile leave nothing
+    int tile;        // latents per tile
+    int buffers;     // 2 if a block may have more than one tile
+};
+__device__ __forceinline__ int visible_tiles(int pos, int window, int tile) {
+    return (window > 0 ? min(pos, window - 1) : pos) / tile + 1;
 }
 
 __host__ __device__ constexpr int dec_pitch(int kv_rank, int rot) { return (kv_rank + rot + 31) / 32 * 32 + 8; }
-template <int TK> constexpr size_t dec_smem(int kv_rank, int rot) {
-    return ((size_t)(DEC_HEADS + 2 * TK) * dec_pitch(kv_rank, rot) + 2 * DEC_HEADS * (TK + 8)) * 2 +
-           (2 * DEC_WARPS * DEC_HEADS + 2 * DEC_HEADS + DEC_MAX_SPLITS * DEC_HEADS) * sizeof(float);
+template <int TK> constexpr size_t dec_smem(int kv_rank, int rot, int buffers) {
+    return ((size_t)(DEC_HEADS + buffers * TK) * dec_pitch(kv_rank, rot) + 2 * DEC_HEADS * (TK + 8)) * 2 +
+           (size_t)(DEC_WARPS * 32 / TK) * DEC_HEADS * (TK + 8) * sizeof(float);
 }
 
-// Grid (splits, groups of 16 heads, sequences), clusters of all splits.  A split takes every tile of TK visible latents that is
-// congruent to it.  NT: output tiles of 8 latent values per warp, 64 * NT >= kv_rank.
+// Grid (splits, groups of 16 heads, sequences).  Split i takes the tiles i, i + splits, .. of TK visible latents.  NT: output
+// tiles of 8 latent values per warp, 64 * NT >= kv_rank.  Latents arrive by bulk copies into padded rows; those of earlier
+// steps are requested before the dependency wait.
 template <int TK, int NT>
 __global__ void __launch_bounds__(DEC_THREADS)
-latent_decode_kernel(const __grid_constant__ md_latent p) {
+latent_decode_kernel(const __grid_constant__ md_latent p, const LatentParts parts, md_devflags* flags) {
     using namespace mb;
-    constexpr int PP = TK + 8;
-    extern __shared__ __align__(16) unsigned char smem[];
-    const int R = p.kv_rank, rot = p.rot, pitch = dec_pitch(R, rot), steps = (pitch - 8) / 32;
-    __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(smem);       // [16][pitch]
-    __nv_bfloat16* Ks = Qs + DEC_HEADS * pitch;                        // two tiles [TK][pitch]; afterwards [16][R] f32
-    __nv_bfloat16* Ps = Ks + 2 * TK * pitch;                           // [2][16][PP]: weights as two terms
-    float* mxs = reinterpret_cast<float*>(Ps + 2 * DEC_HEADS * PP);    // [8][16] maxima
-    float* sms = mxs + DEC_WARPS * DEC_HEADS;                          // [8][16] sums
-    float* ml = sms + DEC_WARPS * DEC_HEADS;                           // [2][16] this block's maximum and sum
-    float* fac = ml + 2 * DEC_HEADS;                                   // [8][16] factors of the cluster's blocks
+    // scores: warps are GROUPS groups of 32 keys x SLICES slices of the latent
+    constexpr int PP = TK + 8, GROUPS = TK / 32, SLICES = DEC_WARPS / GROUPS, KPL = TK / 16;
+    extern __shared__ __align__(128) unsigned char smem[];
+    __shared__ __align__(8) unsigned long long bars[3];               // two tiles, the queries
+    __shared__ float corr_s[DEC_HEADS];
+    __shared__ int abort_s;
+    const int R = p.kv_rank, rot = p.rot, pitch = dec_pitch(R, rot), steps = (pitch - 8) / 16;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
-    const int split = blockIdx.x, splits = gridDim.x, h0 = blockIdx.y * DEC_HEADS, seq = blockIdx.z;
+    const int split = blockIdx.x, splits = parts.splits, h0 = blockIdx.y * DEC_HEADS, seq = blockIdx.z;
     const int heads = min(DEC_HEADS, p.heads - h0);
+    __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(smem);       // [16][pitch]
+    __nv_bfloat16* Ks = Qs + DEC_HEADS * pitch;                        // [buffers][TK][pitch]
+    __nv_bfloat16* Ps = Ks + (size_t)parts.buffers * TK * pitch;       // [2][16][PP]: weights as two terms
+    float* Sx = reinterpret_cast<float*>(Ps + 2 * DEC_HEADS * PP);     // [SLICES][16][PP]: partial scores
     const int pos = *p.pos_dev[seq];      // written by the kernel that ended the previous step
-    const int first = p.window > 0 ? max(0, pos - p.window + 1) : 0;
-    const int tiles = (pos - first) / TK + 1, mine = split < tiles ? (tiles - split - 1) / splits + 1 : 0;
+    const int first = p.window > 0 ? max(0, pos - p.window + 1) : 0, tiles = visible_tiles(pos, p.window, TK);
+    md_pdl_launch_dependents();
+    if (split >= tiles) return;
+    const int mine = (tiles - split - 1) / splits + 1;
+    const uint32_t bar = smem_u32(bars), row_bytes = (uint32_t)(R + rot) * 2;
     const __nv_bfloat16* cc = reinterpret_cast<const __nv_bfloat16*>(p.cc[seq]);
     const __nv_bfloat16* kr = reinterpret_cast<const __nv_bfloat16*>(p.kr[seq]);
-    const int ch = (pitch - 8) / 8, cr = R / 8, crot = (R + rot) / 8;
-    md_pdl_launch_dependents();
-    // keys [lo, hi) of tile `i` of this split; the other rows of the tile and its pad become zero with `fill`
-    auto load_tile = [&](int i, int lo, int hi, bool fill) {
-        const int k0 = first + (split + i * splits) * TK;
-        __nv_bfloat16* K = Ks + (size_t)(i & 1) * TK * pitch;
-        for (int j = tid; j < TK * ch; j += DEC_THREADS) {
-            const int r = j / ch, c = j % ch, key = k0 + r;
-            __nv_bfloat16* dst = K + r * pitch + c * 8;
-            if (key >= lo && key < hi && c < crot)
-                cp_async16(smem_u32(dst), c < cr ? cc + (size_t)key * R + c * 8 : kr + (size_t)key * rot + (c - cr) * 8);
-            else if (fill && (key > pos || c >= crot))
-                *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
-        }
+    auto tile_key = [&](int i) { return first + (split + i * splits) * TK; };
+    auto load_row = [&](int i, int r) {
+        const size_t key = tile_key(i) + r;
+        const uint32_t dst = smem_u32(Ks + ((size_t)(i & 1) * TK + r) * pitch), b = bar + 8 * (i & 1);
+        bulk_load(dst, cc + key * R, R * 2, b);
+        if (rot) bulk_load(dst + R * 2, kr + key * rot, rot * 2, b);
     };
-    // the cached latents of earlier steps are requested before the wait for this step's
-    if (mine > 0) load_tile(0, 0, pos, true);
-    cp_async_commit();
-    md_pdl_wait();
-    if (mine == 1) load_tile(0, pos, pos + 1, false);
-    const __nv_bfloat16* qa = reinterpret_cast<const __nv_bfloat16*>(p.qa) + ((size_t)seq * p.heads + h0) * (R + rot);
-    for (int j = tid; j < DEC_HEADS * ch; j += DEC_THREADS) {
-        const int r = j / ch, c = j % ch;
-        *reinterpret_cast<uint4*>(Qs + r * pitch + c * 8) =
-            r < heads && c < crot ? ld_act(qa + (size_t)r * (R + rot) + c * 8) : make_uint4(0, 0, 0, 0);
+    // by warp 0: the rows of tile i below key `end` (the barrier counts all of the tile's)
+    auto load_tile = [&](int i, int end) {
+        const int n = min(TK, pos + 1 - tile_key(i));
+        if (lane == 0) tc::mbar_expect_tx(bar + 8 * (i & 1), n * row_bytes);
+        __syncwarp();
+        for (int r = lane; r < min(n, end - tile_key(i)); r += 32) load_row(i, r);
+    };
+    if (warp == 0) {
+        if (lane == 0) {
+            abort_s = 0;
+            for (int i = 0; i < 3; ++i) tc::mbar_init(bar + 8 * i, 1);
+            asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+        }
+        __syncwarp();
+        for (int i = 0; i < min(mine, 2); ++i) load_tile(i, pos);
+        if (lane == 0) tc::mbar_expect_tx(bar + 16, heads * row_bytes);
+        md_pdl_wait();
+        // this step's latent, if one of the first tiles holds it, and the queries
+        for (int i = 0; i < min(mine, 2); ++i)
+            if (lane == 0 && pos - tile_key(i) < TK) load_row(i, pos - tile_key(i));
+        if (lane < heads)
+            bulk_load(smem_u32(Qs + lane * pitch),
+                      reinterpret_cast<const __nv_bfloat16*>(p.qa) + ((size_t)seq * p.heads + h0 + lane) * (R + rot), row_bytes, bar + 16);
+    } else {
+        // what no copy fills: the pad of every row, heads and keys that are not there
+        const uint4 zero = make_uint4(0, 0, 0, 0);
+        const int pad0 = (R + rot) / 8, ch = (pitch - 8) / 8;
+        for (int r = warp - 1; r < DEC_HEADS + min(mine, 2) * TK; r += DEC_WARPS - 1) {
+            const int i = (r - DEC_HEADS) / TK;     // (rows of the queries: r < 16)
+            const bool there = r < DEC_HEADS ? r < heads : tile_key(i) + (r - DEC_HEADS) % TK <= pos;
+            for (int c = (there ? pad0 : 0) + lane; c < ch; c += 32) *reinterpret_cast<uint4*>(Qs + r * pitch + c * 8) = zero;
+        }
     }
-    cp_async_commit();
+    __syncthreads();
 
     const float scale = p.scale * LOG2E;
     float o[NT][4];
 #pragma unroll
     for (int i = 0; i < NT; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
-    float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};   // heads g and g + 8; sums over this thread's keys only
-    constexpr int S_WARPS = TK / 8;      // warps that take a tile of 8 keys each
+    float m_run = -INFINITY, l_run = 0.f;      // of head 2 * warp + (lane >> 4); the sum over this lane's keys only
     const int a_row = (lane & 7) + ((lane >> 3) & 1) * 8, a_col = (lane >> 4) * 8;
+    const int b_row = (lane & 7) + (lane >> 4) * 8, b_col = ((lane >> 3) & 1) * 8;
+    const int grp = warp % GROUPS, slice = warp / GROUPS, per = (steps + SLICES - 1) / SLICES;
+    const int s_lo = slice * per, s_hi = min(steps, s_lo + per);
+    const int sh = 2 * warp + (lane >> 4), sk = (lane & 15) * KPL;    // softmax: this lane's head and first key
+    bool ok = tc::mbar_wait(bar + 16, 0, &abort_s, flags, 61);
     for (int it = 0; it < mine; ++it) {
-        cp_async_wait<0>();
-        __syncthreads();                 // tile `it` is there, and nobody reads the other buffer or the weights any more
-        if (it + 1 < mine) load_tile(it + 1, 0, pos + 1, true);
-        cp_async_commit();
+        ok = tc::mbar_wait(bar + 8 * (it & 1), (it >> 1) & 1, &abort_s, flags, 62) && ok;
         const __nv_bfloat16* K = Ks + (size_t)(it & 1) * TK * pitch;
-        const int k0 = first + (split + it * splits) * TK;
-        float s[4] = {0.f, 0.f, 0.f, 0.f};
-        if (warp < S_WARPS) {
-            float s2[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll 4
-            for (int ks = 0; ks < steps; ++ks) {
-                uint32_t a0[4], a1[4], b[4];
-                ldsm_x4(smem_u32(K + (warp * 8 + (lane & 7)) * pitch + ks * 32 + (lane >> 3) * 8), b);
-                ldsm_x4(smem_u32(Qs + a_row * pitch + ks * 32 + a_col), a0);
-                ldsm_x4(smem_u32(Qs + a_row * pitch + ks * 32 + 16 + a_col), a1);
-                mma(s, a0[0], a0[1], a0[2], a0[3], b[0], b[1]);
-                mma(s2, a1[0], a1[1], a1[2], a1[3], b[2], b[3]);
-            }
-            float mx[2] = {-INFINITY, -INFINITY};
+        {
+            float s[4][4];
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {      // head g + 8 (e >> 1), key 2 t + (e & 1)
-                s[e] = k0 + warp * 8 + 2 * t + (e & 1) <= pos ? (s[e] + s2[e]) * scale : -INFINITY;
-                mx[e >> 1] = fmaxf(mx[e >> 1], s[e]);
+            for (int i = 0; i < 4; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
+            const uint32_t qa = smem_u32(Qs + a_row * pitch + a_col), kb = smem_u32(K + (grp * 32 + b_row) * pitch + b_col);
+#pragma unroll 3
+            for (int ks = s_lo; ks < s_hi; ++ks) {
+                uint32_t a[4], b0[4], b1[4];
+                ldsm_x4(qa + ks * 32, a);
+                ldsm_x4(kb + ks * 32, b0);
+                ldsm_x4(kb + 32 * pitch + ks * 32, b1);
+                mma(s[0], a[0], a[1], a[2], a[3], b0[0], b0[1]);
+                mma(s[1], a[0], a[1], a[2], a[3], b0[2], b0[3]);
+                mma(s[2], a[0], a[1], a[2], a[3], b1[0], b1[1]);
+                mma(s[3], a[0], a[1], a[2], a[3], b1[2], b1[3]);
             }
+            float* dst = Sx + (slice * DEC_HEADS + g) * PP + grp * 32 + 2 * t;
 #pragma unroll
-            for (int rr = 0; rr < 2; ++rr) {
-                mx[rr] = fmaxf(mx[rr], __shfl_xor_sync(0xffffffffu, mx[rr], 1));
-                mx[rr] = fmaxf(mx[rr], __shfl_xor_sync(0xffffffffu, mx[rr], 2));
-                if (t == 0) mxs[warp * DEC_HEADS + g + 8 * rr] = mx[rr];
+            for (int i = 0; i < 4; ++i) {
+                *reinterpret_cast<float2*>(dst + i * 8) = make_float2(s[i][0], s[i][1]);
+                *reinterpret_cast<float2*>(dst + 8 * PP + i * 8) = make_float2(s[i][2], s[i][3]);
             }
         }
-        __syncthreads();
-        float corr[2];
-#pragma unroll
-        for (int rr = 0; rr < 2; ++rr) {
-            float mn = m_run[rr];        // every tile holds a visible key: finite from here on
-#pragma unroll
-            for (int i = 0; i < S_WARPS; ++i) mn = fmaxf(mn, mxs[i * DEC_HEADS + g + 8 * rr]);
-            corr[rr] = m_run[rr] == -INFINITY ? 0.f : ex2(m_run[rr] - mn);
-            m_run[rr] = mn;
-            l_run[rr] *= corr[rr];
+        __syncthreads();        // the scores are there, and nobody reads the previous tile any more
+        if (it + 1 >= 2 && it + 1 < mine && warp == 0) {
+            tc::fence_async_smem();
+            load_tile(it + 1, pos + 1);
         }
-        if (warp < S_WARPS) {
+        {
+            float v[KPL];
 #pragma unroll
-            for (int rr = 0; rr < 2; ++rr) {
-                const float w0 = ex2(s[2 * rr] - m_run[rr]), w1 = ex2(s[2 * rr + 1] - m_run[rr]);
-                l_run[rr] += w0 + w1;
+            for (int i = 0; i < KPL; ++i) v[i] = 0.f;
+#pragma unroll
+            for (int c = 0; c < SLICES; ++c) {
+                const float* src = Sx + (c * DEC_HEADS + sh) * PP + sk;
+#pragma unroll
+                for (int i = 0; i < KPL; i += 2) {
+                    const float2 x = *reinterpret_cast<const float2*>(src + i);
+                    v[i] += x.x;
+                    v[i + 1] += x.y;
+                }
+            }
+            float mx = -INFINITY;
+#pragma unroll
+            for (int i = 0; i < KPL; ++i) {
+                v[i] = tile_key(it) + sk + i <= pos ? v[i] * scale : -INFINITY;
+                mx = fmaxf(mx, v[i]);
+            }
+#pragma unroll
+            for (int x = 8; x; x >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, x));
+            const float mn = fmaxf(m_run, mx);       // every tile holds a visible key: finite
+            const float corr = m_run == -INFINITY ? 0.f : ex2(m_run - mn);
+            m_run = mn;
+            l_run *= corr;
+#pragma unroll
+            for (int i = 0; i < KPL; i += 2) {
+                const float w0 = ex2(v[i] - mn), w1 = ex2(v[i + 1] - mn);
+                l_run += w0 + w1;
                 uint32_t hi, lo;
                 split2(w0, w1, hi, lo);
-                __nv_bfloat16* dst = Ps + (g + 8 * rr) * PP + warp * 8 + 2 * t;
-                *reinterpret_cast<uint32_t*>(dst) = hi;
-                *reinterpret_cast<uint32_t*>(dst + DEC_HEADS * PP) = lo;
+                *reinterpret_cast<uint32_t*>(Ps + sh * PP + sk + i) = hi;
+                *reinterpret_cast<uint32_t*>(Ps + (DEC_HEADS + sh) * PP + sk + i) = lo;
             }
-        }
-#pragma unroll
-        for (int i = 0; i < NT; ++i) {
-            o[i][0] *= corr[0]; o[i][1] *= corr[0];
-            o[i][2] *= corr[1]; o[i][3] *= corr[1];
+            if ((lane & 15) == 0) corr_s[sh] = corr;
         }
         __syncthreads();
+        if (it > 0) {
+            const float c0 = corr_s[g], c1 = corr_s[g + 8];
+#pragma unroll
+            for (int i = 0; i < NT; ++i) {
+                o[i][0] *= c0; o[i][1] *= c0;
+                o[i][2] *= c1; o[i][3] *= c1;
+            }
+        }
 #pragma unroll
         for (int kk = 0; kk < TK / 16; ++kk) {
             uint32_t hi[4], lo[4];
@@ -596,7 +734,7 @@ latent_decode_kernel(const __grid_constant__ md_latent p) {
                 const int col = (warp * NT + 2 * np) * 8;
                 if (col >= R) break;
                 uint32_t b[4];
-                ldsm_x4_t(smem_u32(K + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * pitch + col + (lane >> 4) * 8), b);
+                ldsm_x4_t(smem_u32(K + (kk * 16 + a_row) * pitch + col + a_col), b);
                 mma(o[2 * np], hi[0], hi[1], hi[2], hi[3], b[0], b[1]);
                 mma(o[2 * np + 1], hi[0], hi[1], hi[2], hi[3], b[2], b[3]);
                 mma(o[2 * np], lo[0], lo[1], lo[2], lo[3], b[0], b[1]);
@@ -604,68 +742,99 @@ latent_decode_kernel(const __grid_constant__ md_latent p) {
             }
         }
     }
-    cp_async_wait<0>();
+    if (!ok) return;                          // a copy did not arrive within the wait's limit: reported through `flags`
 #pragma unroll
-    for (int rr = 0; rr < 2; ++rr) {
-        l_run[rr] += __shfl_xor_sync(0xffffffffu, l_run[rr], 1);
-        l_run[rr] += __shfl_xor_sync(0xffffffffu, l_run[rr], 2);
-        if (t == 0) sms[warp * DEC_HEADS + g + 8 * rr] = l_run[rr];
-        if (t == 0 && warp == 0) ml[g + 8 * rr] = m_run[rr];
+    for (int x = 8; x; x >>= 1) l_run += __shfl_xor_sync(0xffffffffu, l_run, x);
+    const size_t slot = ((size_t)seq * p.heads + h0) * splits + split;   // + head * splits
+    if ((lane & 15) == 0 && sh < heads) parts.ml[slot + (size_t)sh * splits] = make_float2(m_run, l_run);
+    float* out = parts.o + (slot + (size_t)g * splits) * R;
+#pragma unroll
+    for (int i = 0; i < NT; ++i) {
+        const int col = (warp * NT + i) * 8 + 2 * t;
+        if (col >= R) break;
+        if (g < heads) *reinterpret_cast<float2*>(out + col) = make_float2(o[i][0], o[i][1]);
+        if (g + 8 < heads) *reinterpret_cast<float2*>(out + 8 * (size_t)splits * R + col) = make_float2(o[i][2], o[i][3]);
     }
-    __syncthreads();                     // all reads of the tiles are over
-    float* Of = reinterpret_cast<float*>(Ks);
-    if (mine > 0) {
+}
+
+// out[s][h][e] = sum_r w[h][e][r] o[s][h][r] with o merged from the window's parts, the sink in its denominator.  Block: 32 rows
+// of a head, all sequences; 4 warps split the latent.
+constexpr int VAL_THREADS = 256, VAL_UNROLL = 4, VAL_MAX_RANK = 1024;
+
+__global__ void __launch_bounds__(VAL_THREADS)
+latent_value_kernel(const __grid_constant__ md_latent p, const LatentParts parts) {
+    __shared__ __align__(16) __nv_bfloat16 xs[MD_STACK_MAX_SEQS][VAL_MAX_RANK + 8];
+    __shared__ float fac[MD_STACK_MAX_SEQS][DEC_MAX_SPLITS];
+    __shared__ int used[MD_STACK_MAX_SEQS];
+    __shared__ float partial[4][32][9];
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+    const int R = p.kv_rank, E = p.vdim, h = blockIdx.y, row0 = blockIdx.x * 32 + (warp & 1) * 16, slice = warp >> 1;
+    const __nv_bfloat16* w = reinterpret_cast<const __nv_bfloat16*>(p.w_ukv) + ((size_t)p.heads * p.dim + (size_t)h * E) * R + t * 8;
+    const __nv_bfloat16 *w_lo = w + (size_t)min(row0 + g, E - 1) * R, *w_hi = w + (size_t)min(row0 + g + 8, E - 1) * R;
+    const uint4 zero = make_uint4(0, 0, 0, 0);
+    md_pdl_launch_dependents();
+    uint4 lo[VAL_UNROLL], hi[VAL_UNROLL];
+    auto weights = [&](int k0) {
 #pragma unroll
-        for (int i = 0; i < NT; ++i) {
-            const int col = (warp * NT + i) * 8 + 2 * t;
-            if (col >= R) break;
-            *reinterpret_cast<float2*>(Of + g * R + col) = make_float2(o[i][0], o[i][1]);
-            *reinterpret_cast<float2*>(Of + (g + 8) * R + col) = make_float2(o[i][2], o[i][3]);
+        for (int u = 0; u < VAL_UNROLL; ++u) {
+            const int k = k0 + u * 128;
+            const bool live = k + t * 8 < R;
+            lo[u] = live ? ldg_stream(w_lo + k) : zero;
+            hi[u] = live ? ldg_stream(w_hi + k) : zero;
         }
-    }
-    if (tid < DEC_HEADS) {
-        float l = 0.f;
+    };
+    weights(slice * 32);
+    if (warp < p.seqs && lane == 0) used[warp] = min(parts.splits, visible_tiles(*p.pos_dev[warp], p.window, parts.tile));
+    __syncwarp();
+    md_pdl_wait();
+    if (warp < p.seqs) {         // a warp per sequence, a lane per part
+        const bool live = lane < used[warp];
+        const float2 v = live ? __ldcg(parts.ml + ((size_t)warp * p.heads + h) * parts.splits + lane) : make_float2(-INFINITY, 0.f);
+        const float sink = p.sink[h] * LOG2E;
+        float m = fmaxf(v.x, sink);
 #pragma unroll
-        for (int i = 0; i < DEC_WARPS; ++i) l += sms[i * DEC_HEADS + tid];
-        ml[DEC_HEADS + tid] = l;
-    }
-    cluster_sync();
-    if (tid < DEC_HEADS) {
-        const uint32_t at = smem_u32(ml + tid);
-        const float sink = p.sink[h0 + min(tid, heads - 1)] * LOG2E;
-        float m = sink, pm[DEC_MAX_SPLITS], l;
-#pragma unroll
-        for (int i = 0; i < DEC_MAX_SPLITS; ++i) {
-            pm[i] = i < splits ? ld_peer(at, i) : -INFINITY;
-            m = fmaxf(m, pm[i]);
-        }
-        l = ex2(sink - m);
-#pragma unroll
-        for (int i = 0; i < DEC_MAX_SPLITS; ++i) {
-            pm[i] = pm[i] == -INFINITY ? 0.f : ex2(pm[i] - m);
-            if (i < splits) l = fmaf(ld_peer(at + DEC_HEADS * sizeof(float), i), pm[i], l);
-        }
-#pragma unroll
-        for (int i = 0; i < DEC_MAX_SPLITS; ++i) fac[i * DEC_HEADS + tid] = pm[i] / l;
+        for (int x = 16; x; x >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, x));
+        const float f = live ? ex2(v.x - m) : 0.f, l = warp_sum(v.y * f) + ex2(sink - m);
+        fac[warp][lane] = f / l;
     }
     __syncthreads();
-    __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(p.ol) + ((size_t)seq * p.heads + h0) * R;
-    const int used = min(splits, tiles);
-    for (int i = (split * DEC_THREADS + tid) * 2; i < heads * R; i += splits * DEC_THREADS * 2) {
-        const int hh = i / R;
-        const uint32_t at = smem_u32(Of + i);
-        float2 a = make_float2(0.f, 0.f);
-#pragma unroll
-        for (int j = 0; j < DEC_MAX_SPLITS; ++j) {
-            if (j >= used) break;
-            const float2 v = ld_peer2(at, j);
-            const float f = fac[j * DEC_HEADS + hh];
-            a.x = fmaf(v.x, f, a.x);
-            a.y = fmaf(v.y, f, a.y);
+    const int quads = R / 4;
+    for (int i = tid; i < p.seqs * quads; i += VAL_THREADS) {
+        const int s = i / quads, c = (i - s * quads) * 4, n = used[s];
+        const float* src = parts.o + ((size_t)s * p.heads + h) * parts.splits * R + c;
+        float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+        for (int j = 0; j < n; ++j) {
+            const float4 v = __ldcg(reinterpret_cast<const float4*>(src + (size_t)j * R));
+            const float f = fac[s][j];
+            a.x = fmaf(v.x, f, a.x); a.y = fmaf(v.y, f, a.y);
+            a.z = fmaf(v.z, f, a.z); a.w = fmaf(v.w, f, a.w);
         }
-        *reinterpret_cast<uint32_t*>(out + i) = md_pack_bf16(a.x, a.y);
+        *reinterpret_cast<uint2*>(&xs[s][c]) = make_uint2(md_pack_bf16(a.x, a.y), md_pack_bf16(a.z, a.w));
     }
-    cluster_sync();                      // the peers' shared memory stays until all have read it
+    __syncthreads();
+    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+    const bool has_x = g < p.seqs;
+    for (int k0 = slice * 32; k0 < R; k0 += VAL_UNROLL * 128) {
+        if (k0 != slice * 32) weights(k0);
+#pragma unroll
+        for (int u = 0; u < VAL_UNROLL; ++u) {
+            const int k = k0 + u * 128 + t * 8;
+            const uint4 x = has_x && k < R ? *reinterpret_cast<const uint4*>(&xs[has_x ? g : 0][k]) : zero;
+            mb::mma(acc, lo[u].x, hi[u].x, lo[u].y, hi[u].y, x.x, x.y);
+            mb::mma(acc, lo[u].z, hi[u].z, lo[u].w, hi[u].w, x.z, x.w);
+        }
+    }
+    float (*dst)[9] = partial[slice] + (warp & 1) * 16;
+    dst[g][2 * t] = acc[0];
+    dst[g][2 * t + 1] = acc[1];
+    dst[g + 8][2 * t] = acc[2];
+    dst[g + 8][2 * t + 1] = acc[3];
+    __syncthreads();
+    const int s = tid >> 5, e = blockIdx.x * 32 + lane;
+    if (s < p.seqs && e < E)
+        reinterpret_cast<__nv_bfloat16*>(p.out)[((size_t)s * p.heads + h) * E + e] =
+            __float2bfloat16_rn(partial[0][lane][s] + partial[1][lane][s] + partial[2][lane][s] + partial[3][lane][s]);
 }
 
 bool eights(std::initializer_list<int> v) {
@@ -721,57 +890,36 @@ int launch_prefill(md_ctx* ctx, const md_latent& a) {
     return launch_prefill_as<256, 256>(ctx, a, key0);
 }
 
-int launch_heads(md_ctx* ctx, const HeadsProduct& h, int heads) {
-    return md_launch_ex(ctx, latent_heads_kernel, dim3((unsigned)((h.N + 15) / 16), (unsigned)heads), dim3(HEADS_WARPS * 32), 0,
-                        "latent_heads_kernel", h);
-}
-
 template <int TK, int NT>
 int launch_decode_as(md_ctx* ctx, const md_latent& a) {
     const size_t most = md_latent_keys(1, a.window > 0 ? a.window : 0, a.max_seq), tiles = (most + TK - 1) / TK;
-    const unsigned splits = (unsigned)std::min<size_t>(DEC_MAX_SPLITS, tiles);
-    const size_t smem = dec_smem<TK>(a.kv_rank, a.rot);
+    const size_t groups = (a.heads + DEC_HEADS - 1) / DEC_HEADS, rows = (size_t)a.seqs * a.heads;
+    // a block per SM where the windows are long enough
+    const size_t splits = std::max<size_t>(1, std::min<size_t>({DEC_MAX_SPLITS, tiles, ctx->sm_count / (a.seqs * groups)}));
+    LatentParts parts;
+    parts.splits = (int)splits, parts.tile = TK, parts.buffers = tiles > splits ? 2 : 1;
+    void* scratch = nullptr;
+    MD_TRY(md_scratch(ctx, rows * splits * (a.kv_rank * sizeof(float) + sizeof(float2)), &scratch));
+    parts.o = reinterpret_cast<float*>(scratch);
+    parts.ml = reinterpret_cast<float2*>(parts.o + rows * splits * a.kv_rank);
+    const size_t smem = dec_smem<TK>(a.kv_rank, a.rot, parts.buffers);
     auto kern = latent_decode_kernel<TK, NT>;
     MD_CUDA(ctx, cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    cudaLaunchConfig_t cfg = {};
-    cfg.gridDim = dim3(splits, (unsigned)((a.heads + DEC_HEADS - 1) / DEC_HEADS), (unsigned)a.seqs);
-    cfg.blockDim = dim3(DEC_THREADS);
-    cfg.dynamicSmemBytes = smem;
-    cfg.stream = ctx->stream;
-    cudaLaunchAttribute attr[2];
-    attr[0].id = cudaLaunchAttributeClusterDimension;
-    attr[0].val.clusterDim.x = splits;
-    attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
-    attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    attr[1].val.programmaticStreamSerializationAllowed = 1;
-    cfg.attrs = attr;
-    cfg.numAttrs = ctx->pdl ? 2 : 1;
-    const cudaError_t e = cudaLaunchKernelEx(&cfg, kern, a);
-    if (e != cudaSuccess) return md_fail(ctx, MD_ERR_CUDA, "launch of latent_decode_kernel failed: %s", cudaGetErrorString(e));
-    ctx->launches++;
-    return MD_OK;
+    MD_TRY(md_launch_ex(ctx, kern, dim3((unsigned)splits, (unsigned)groups, (unsigned)a.seqs), dim3(DEC_THREADS), smem, "latent_decode_kernel",
+                        a, parts, ctx->flags));
+    return md_launch_ex(ctx, latent_value_kernel, dim3((unsigned)((a.vdim + 31) / 32), (unsigned)a.heads), dim3(VAL_THREADS), 0,
+                        "latent_value_kernel", a, parts);
 }
 
 int launch_decode(md_ctx* ctx, const md_latent& a) {
     const int D = a.dim, R = a.kv_rank, rot = a.rot, H = a.heads;
-    const __nv_bfloat16* ukv = reinterpret_cast<const __nv_bfloat16*>(a.w_ukv);
-    HeadsProduct q = {};
-    q.w = reinterpret_cast<const __nv_bfloat16*>(a.w_ukt), q.x = reinterpret_cast<const __nv_bfloat16*>(a.q);
-    q.out = reinterpret_cast<__nv_bfloat16*>(a.qa);
-    q.N = R, q.K = D, q.seqs = a.seqs;
-    q.x_seq = H * (D + rot), q.x_head = D + rot, q.out_seq = H * (R + rot), q.out_head = R + rot;
-    q.rot = rot, q.rope = a.rope;
-    for (int i = 0; i < a.seqs; ++i) q.pos[i] = a.pos_dev[i];
-    MD_TRY(launch_heads(ctx, q, H));
-    if (R <= 128) MD_TRY((launch_decode_as<64, 2>(ctx, a)));
-    else if (R <= 256) MD_TRY((launch_decode_as<64, 4>(ctx, a)));
-    else if (R <= 512) MD_TRY((launch_decode_as<64, 8>(ctx, a)));
-    else MD_TRY((launch_decode_as<32, 16>(ctx, a)));
-    HeadsProduct v = {};
-    v.w = ukv + (size_t)H * D * R, v.x = reinterpret_cast<const __nv_bfloat16*>(a.ol), v.out = reinterpret_cast<__nv_bfloat16*>(a.out);
-    v.N = a.vdim, v.K = R, v.seqs = a.seqs;
-    v.x_seq = H * R, v.x_head = R, v.out_seq = H * a.vdim, v.out_head = a.vdim;
-    return launch_heads(ctx, v, H);
+    const int row_blocks = (H * (D + rot) + 15) / 16;
+    MD_TRY(md_launch_ex(ctx, latent_query_kernel, dim3((unsigned)(row_blocks + a.seqs)), dim3(UQ_WARPS * 32), 0, "latent_query_kernel", a, row_blocks));
+    MD_TRY(md_launch_ex(ctx, latent_absorb_kernel, dim3((unsigned)((R + 15) / 16), (unsigned)H), dim3(HEADS_WARPS * 32), 0, "latent_absorb_kernel", a));
+    if (R <= 128) return launch_decode_as<64, 2>(ctx, a);
+    if (R <= 256) return launch_decode_as<64, 4>(ctx, a);
+    if (R <= 512) return launch_decode_as<64, 8>(ctx, a);
+    return launch_decode_as<32, 16>(ctx, a);
 }
 
 }  // namespace
@@ -788,10 +936,10 @@ int md_launch_rotation_table(md_ctx* ctx, float* table, size_t rows, size_t dims
 
 int md_launch_latent_attention(md_ctx* ctx, int dtype, const md_latent& a, bool decode) {
     const bool f32 = dtype == MD_DTYPE_F32;
+    if (!f32 && decode && a.rows == 1 && decode_ok(a)) return launch_decode(ctx, a);
     MD_TRY(f32 ? launch_norm<float>(ctx, a) : launch_norm<__nv_bfloat16>(ctx, a));
     const size_t rows = (size_t)a.rows * a.seqs;
     MD_TRY(md_linear(ctx, dtype, a.cq, a.w_uq, a.q, rows, (size_t)a.heads * (a.dim + a.rot), a.q_rank, md_lin()));
     if (md_latent_expands(dtype, a) && !decode) return launch_prefill(ctx, a);
-    if (!f32 && decode && a.rows == 1 && decode_ok(a)) return launch_decode(ctx, a);
     return f32 ? launch_plain<float>(ctx, a) : launch_plain<__nv_bfloat16>(ctx, a);
 }

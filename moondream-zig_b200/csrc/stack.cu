@@ -13,7 +13,7 @@ struct md_stack {
     size_t elem = 2;                 // bytes of T
     bool parallel = false;           // MD_LAYER_PARALLEL
     size_t max_in = 0, max_o = 0, max_ff = 0, max_ssq = 0, max_top = 0, max_choices = 0, max_experts = 0, max_moe_ff = 0, max_shared = 0;
-    size_t max_cq = 0, max_q = 0, max_qa = 0, max_ol = 0;   // latent attention, per row
+    size_t max_cq = 0, max_q = 0, max_qa = 0;   // latent attention, per row
     size_t kv_bytes = 0;             // key caches of one request
     size_t state_floats = 0;         // recurrent states and convolution tails of one request
     std::vector<size_t> kv_off, rec_off, conv1_off, conv2_off;   // per layer; bytes / floats
@@ -29,7 +29,7 @@ struct md_stack_request {
     DevPtr state;     // all f32 states, zeroed by a reset
     DevPtr x[2], h, in, o, y, ff, ssq;
     DevPtr h2, y2;              // parallel layers: the feed-forward's input and output
-    DevPtr cq, q, qa, ol;       // latent attention
+    DevPtr cq, q, qa;           // latent attention
     DevPtr route, score, sel, rank, slot, count, tile_expert, n_blocks, xs, act, ys;
     DevPtr trace;     // [layers][rows][width] when stack_trace is set
     size_t cap_rows = 0, trace_rows = 0;
@@ -182,7 +182,6 @@ extern "C" int md_stack_model_create(md_ctx* ctx, const md_stack_weights* w, md_
             s.max_cq = std::max(s.max_cq, l.q_rank);
             s.max_q = std::max(s.max_q, l.heads * (l.dim + l.rot_dim));
             s.max_qa = std::max(s.max_qa, l.heads * (l.kv_rank + l.rot_dim));
-            s.max_ol = std::max(s.max_ol, l.heads * l.kv_rank);
             MD_TRY(add_rotation(ctx, s, l.rot_dim, l.rope_base));
         } else {
             s.rope.push_back(nullptr);
@@ -277,7 +276,6 @@ int md_stack_reserve(md_text_request* req, size_t rows) {
         MD_TRY(r->cq.ensure(ctx, rows * s.max_cq * E));
         MD_TRY(r->q.ensure(ctx, rows * s.max_q * E));
         MD_TRY(r->qa.ensure(ctx, MD_STACK_MAX_SEQS * s.max_qa * E));
-        MD_TRY(r->ol.ensure(ctx, MD_STACK_MAX_SEQS * s.max_ol * E));
     }
     if (s.max_ssq) MD_TRY(r->ssq.ensure(ctx, rows * s.max_ssq * sizeof(float)));
     if (s.max_experts) {
@@ -356,7 +354,7 @@ int latent_mixer(const Pass& p, size_t i) {
     a.q_norm = l.q_norm, a.kv_norm = l.kv_norm, a.sink = l.sink, a.rope = p.s.rope[i];
     a.w_uq = l.w_uq, a.w_ukv = l.w_ukv, a.w_ukt = l.w_ukt;
     a.in = b->in.p, a.row_stride = (int)l.in_rows;
-    a.cq = b->cq.p, a.q = b->q.p, a.qa = b->qa.p, a.ol = b->ol.p, a.out = b->o.p;
+    a.cq = b->cq.p, a.q = b->q.p, a.qa = b->qa.p, a.out = b->o.p;
     a.rows = (int)p.rows, a.seqs = (int)p.seqs, a.max_seq = p.s.w.max_seq, a.pos0 = (int)p.pos0;
     for (size_t q = 0; q < p.seqs; ++q) {
         char* at = p.reqs[q]->stack->keys.as<char>() + p.s.kv_off[i];

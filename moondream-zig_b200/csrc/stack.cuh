@@ -150,8 +150,7 @@ struct md_latent {
     int pos0 = 0;                           // prefill: position of row 0
     // prompts in bfloat16: keys and values of every visible token, [md_latent_keys(..)][heads * (dim + vdim)]
     void* kv = nullptr;
-    // bfloat16 decoding: absorbed queries [seqs][heads][kv_rank + rot] and merged latents [seqs][heads][kv_rank]
-    void *qa = nullptr, *ol = nullptr;
+    void* qa = nullptr;                     // bfloat16 decoding: queries in the latent space [seqs][heads][kv_rank + rot]
 };
 // tokens whose keys a portion of `rows` rows can see (itself included)
 inline size_t md_latent_keys(size_t rows, size_t window, size_t max_seq) {
