@@ -4,9 +4,10 @@
 //   latent_norm_kernel      norms of the two latents, rotation of the shared key part, append to the cache
 //   latent_plain_kernel     any element type and size, prompts and decoding: a block per (token, head) that takes the query
 //                           into the latent space (q_h W_uk_h), so that scores and weighted sums run on the cached latents
-//   latent_prefill_kernel   bfloat16 prompts: keys and values of the visible tokens come expanded from one product; 64 queries
-//                           x 64 keys per step on tensor cores.  The query's rotation happens on its way to shared memory.
-//                           Weights enter the second product as two bfloat16 terms (mma_bf16.cuh).
+//   latent_prefill_kernel   bfloat16 prompts whose head sizes the tcgen05 kernel (attention_latent_tc.cu) cannot hold: keys and
+//                           values of the visible tokens come expanded from one product; 64 queries x 64 keys per step on
+//                           mma.sync.  The query's rotation happens on its way to shared memory.  Weights enter the second
+//                           product as two bfloat16 terms (mma_bf16.cuh).
 //   latent_query_kernel     bfloat16, one token per sequence: norms, the queries' product and the append to the cache
 //   latent_absorb_kernel    bfloat16, one token per sequence: the query into the latent space, per head
 //   latent_decode_kernel    bfloat16, one token per sequence: 16 heads share every latent they read; blocks take parts of the
@@ -758,17 +759,18 @@ latent_decode_kernel(const __grid_constant__ md_latent p, const LatentParts part
 }
 
 // out[s][h][e] = sum_r w[h][e][r] o[s][h][r] with o merged from the window's parts, the sink in its denominator.  Block: 32 rows
-// of a head, all sequences; 4 warps split the latent.
-constexpr int VAL_THREADS = 256, VAL_UNROLL = 4, VAL_MAX_RANK = 1024;
+// of a head, four sequences; 4 warps split the latent.
+constexpr int VAL_THREADS = 256, VAL_UNROLL = 4, VAL_MAX_RANK = 1024, VAL_SEQS = 4;
 
 __global__ void __launch_bounds__(VAL_THREADS)
 latent_value_kernel(const __grid_constant__ md_latent p, const LatentParts parts) {
-    __shared__ __align__(16) __nv_bfloat16 xs[MD_STACK_MAX_SEQS][VAL_MAX_RANK + 8];
-    __shared__ float fac[MD_STACK_MAX_SEQS][DEC_MAX_SPLITS];
-    __shared__ int used[MD_STACK_MAX_SEQS];
+    __shared__ __align__(16) __nv_bfloat16 xs[VAL_SEQS][VAL_MAX_RANK + 8];
+    __shared__ float fac[VAL_SEQS][DEC_MAX_SPLITS];
+    __shared__ int used[VAL_SEQS];
     __shared__ float partial[4][32][9];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
     const int R = p.kv_rank, E = p.vdim, h = blockIdx.y, row0 = blockIdx.x * 32 + (warp & 1) * 16, slice = warp >> 1;
+    const int seq0 = blockIdx.z * VAL_SEQS, seqs = min(VAL_SEQS, p.seqs - seq0);
     const __nv_bfloat16* w = reinterpret_cast<const __nv_bfloat16*>(p.w_ukv) + ((size_t)p.heads * p.dim + (size_t)h * E) * R + t * 8;
     const __nv_bfloat16 *w_lo = w + (size_t)min(row0 + g, E - 1) * R, *w_hi = w + (size_t)min(row0 + g + 8, E - 1) * R;
     const uint4 zero = make_uint4(0, 0, 0, 0);
@@ -784,12 +786,12 @@ latent_value_kernel(const __grid_constant__ md_latent p, const LatentParts parts
         }
     };
     weights(slice * 32);
-    if (warp < p.seqs && lane == 0) used[warp] = min(parts.splits, visible_tiles(*p.pos_dev[warp], p.window, parts.tile));
+    if (warp < seqs && lane == 0) used[warp] = min(parts.splits, visible_tiles(*p.pos_dev[seq0 + warp], p.window, parts.tile));
     __syncwarp();
     md_pdl_wait();
-    if (warp < p.seqs) {         // a warp per sequence, a lane per part
+    if (warp < seqs) {           // a warp per sequence, a lane per part
         const bool live = lane < used[warp];
-        const float2 v = live ? __ldcg(parts.ml + ((size_t)warp * p.heads + h) * parts.splits + lane) : make_float2(-INFINITY, 0.f);
+        const float2 v = live ? __ldcg(parts.ml + ((size_t)(seq0 + warp) * p.heads + h) * parts.splits + lane) : make_float2(-INFINITY, 0.f);
         const float sink = p.sink[h] * LOG2E;
         float m = fmaxf(v.x, sink);
 #pragma unroll
@@ -799,9 +801,9 @@ latent_value_kernel(const __grid_constant__ md_latent p, const LatentParts parts
     }
     __syncthreads();
     const int quads = R / 4;
-    for (int i = tid; i < p.seqs * quads; i += VAL_THREADS) {
+    for (int i = tid; i < seqs * quads; i += VAL_THREADS) {
         const int s = i / quads, c = (i - s * quads) * 4, n = used[s];
-        const float* src = parts.o + ((size_t)s * p.heads + h) * parts.splits * R + c;
+        const float* src = parts.o + ((size_t)(seq0 + s) * p.heads + h) * parts.splits * R + c;
         float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll 8
         for (int j = 0; j < n; ++j) {
@@ -814,7 +816,7 @@ latent_value_kernel(const __grid_constant__ md_latent p, const LatentParts parts
     }
     __syncthreads();
     float acc[4] = {0.f, 0.f, 0.f, 0.f};
-    const bool has_x = g < p.seqs;
+    const bool has_x = g < seqs;
     for (int k0 = slice * 32; k0 < R; k0 += VAL_UNROLL * 128) {
         if (k0 != slice * 32) weights(k0);
 #pragma unroll
@@ -832,8 +834,8 @@ latent_value_kernel(const __grid_constant__ md_latent p, const LatentParts parts
     dst[g + 8][2 * t + 1] = acc[3];
     __syncthreads();
     const int s = tid >> 5, e = blockIdx.x * 32 + lane;
-    if (s < p.seqs && e < E)
-        reinterpret_cast<__nv_bfloat16*>(p.out)[((size_t)s * p.heads + h) * E + e] =
+    if (s < seqs && e < E)
+        reinterpret_cast<__nv_bfloat16*>(p.out)[((size_t)(seq0 + s) * p.heads + h) * E + e] =
             __float2bfloat16_rn(partial[0][lane][s] + partial[1][lane][s] + partial[2][lane][s] + partial[3][lane][s]);
 }
 
@@ -881,12 +883,8 @@ int launch_prefill(md_ctx* ctx, const md_latent& a) {
     const size_t R = a.kv_rank;
     MD_TRY(md_linear(ctx, MD_DTYPE_BF16, reinterpret_cast<const __nv_bfloat16*>(a.cc[0]) + key0 * R, a.w_ukv, a.kv, keys,
                      (size_t)a.heads * (a.dim + a.vdim), R, md_lin()));
-    const int dk = a.dim + a.rot, dv = a.vdim;
-    if (dk <= 64 && dv <= 64) return launch_prefill_as<64, 64>(ctx, a, key0);
-    if (dk <= 96 && dv <= 64) return launch_prefill_as<96, 64>(ctx, a, key0);
-    if (dk <= 128 && dv <= 64) return launch_prefill_as<128, 64>(ctx, a, key0);
-    if (dk <= 128 && dv <= 128) return launch_prefill_as<128, 128>(ctx, a, key0);
-    if (dk <= 192 && dv <= 128) return launch_prefill_as<192, 128>(ctx, a, key0);
+    if (ctx->attn_tc != 0 && md_latent_tc_supported(a)) return md_launch_latent_tc(ctx, a, key0);
+    if (a.dim + a.rot <= 128 && a.vdim <= 128) return launch_prefill_as<128, 128>(ctx, a, key0);
     return launch_prefill_as<256, 256>(ctx, a, key0);
 }
 
@@ -907,7 +905,7 @@ int launch_decode_as(md_ctx* ctx, const md_latent& a) {
     MD_CUDA(ctx, cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     MD_TRY(md_launch_ex(ctx, kern, dim3((unsigned)splits, (unsigned)groups, (unsigned)a.seqs), dim3(DEC_THREADS), smem, "latent_decode_kernel",
                         a, parts, ctx->flags));
-    return md_launch_ex(ctx, latent_value_kernel, dim3((unsigned)((a.vdim + 31) / 32), (unsigned)a.heads), dim3(VAL_THREADS), 0,
+    return md_launch_ex(ctx, latent_value_kernel, dim3((unsigned)((a.vdim + 31) / 32), (unsigned)a.heads, (unsigned)((a.seqs + VAL_SEQS - 1) / VAL_SEQS)), dim3(VAL_THREADS), 0,
                         "latent_value_kernel", a, parts);
 }
 

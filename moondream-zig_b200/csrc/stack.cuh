@@ -159,6 +159,9 @@ inline size_t md_latent_keys(size_t rows, size_t window, size_t max_seq) {
 // whether a portion of `rows` rows of one sequence takes the tensor-core prompt kernel (and so needs md_latent::kv)
 bool md_latent_expands(int dtype, const md_latent& a);
 int md_launch_latent_attention(md_ctx* ctx, int dtype, const md_latent& a, bool decode);
+// the prompt kernel on tcgen05 (bfloat16; head sizes it cannot hold take latent_prefill_kernel)
+bool md_latent_tc_supported(const md_latent& a);
+int md_launch_latent_tc(md_ctx* ctx, const md_latent& a, int key0);
 // (cos, sin) of pos * base^(-2 i / dims) for pos < rows, i < dims / 2; angles in f64
 int md_launch_rotation_table(md_ctx* ctx, float* table, size_t rows, size_t dims, float base);
 

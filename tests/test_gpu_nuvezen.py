@@ -174,6 +174,23 @@ def test_token_by_token_equals_the_prompt(ctx, mods, name, dtype):
         r.close()
 
 
+@pytest.mark.parametrize("name", ["even", "wide", "long"])
+def test_both_prompt_kernels(ctx, mods, name):
+    """The tcgen05 kernel and the one that takes the head sizes it cannot hold."""
+    toks, want = expected(name, 300)
+    try:
+        for option in (1, 0):
+            ctx.set_option("attn_tc", option)
+            with model(ctx, mods, name, "bfloat16") as m:
+                r = m.request()
+                for cuts in ((), (5, 130, 133, 270)):
+                    r.reset()
+                    nu.assert_logits(run(m, r, toks, cuts), want, "bfloat16", f"{name}, attn_tc {option}, cuts {cuts}")
+                r.close()
+    finally:
+        ctx.set_option("attn_tc", -1)
+
+
 PORTIONS = [tuple(range(2, 300, 2)), tuple(range(3, 300, 7)), (1, 3, 66, 69, 133, 135, 136, 200, 263, 266), tuple(range(64, 300, 64)),
             tuple(range(8, 300, 9)), (299,)]
 
