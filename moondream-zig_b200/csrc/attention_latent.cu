@@ -45,61 +45,98 @@ __global__ void rotation_table_kernel(float* table, int rows, int half, double b
 }
 
 template <class T, int V> __device__ __forceinline__ void load_v(const T* p, float (&f)[V]) {
-    if constexpr (V == 4) md_load4<T>(p, f);
-    else f[0] = md_elem<T>::get(*p);
+    if constexpr (V == 8) {
+        const uint4 u = __ldcg(reinterpret_cast<const uint4*>(p));
+        const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i) f[2 * i] = __uint_as_float(w[i] << 16), f[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
+    } else if constexpr (V == 4) {
+        md_load4<T>(p, f);
+    } else {
+        f[0] = md_elem<T>::get(*p);
+    }
+}
+template <int V> __device__ __forceinline__ void load_weight(const float* p, float (&f)[V]) {
+    if constexpr (V == 1) {
+        f[0] = __ldg(p);
+    } else {
+#pragma unroll
+        for (int i = 0; i < V; i += 4) {
+            const float4 v = __ldg(reinterpret_cast<const float4*>(p + i));
+            f[i] = v.x, f[i + 1] = v.y, f[i + 2] = v.z, f[i + 3] = v.w;
+        }
+    }
 }
 template <class T, int V> __device__ __forceinline__ void store_v(T* p, const float (&f)[V]) {
-    if constexpr (V == 4) md_store4<T>(p, f);
-    else *p = md_elem<T>::put(f[0]);
+    if constexpr (V == 8) {
+        *reinterpret_cast<uint4*>(p) = make_uint4(md_pack_bf16(f[0], f[1]), md_pack_bf16(f[2], f[3]), md_pack_bf16(f[4], f[5]), md_pack_bf16(f[6], f[7]));
+    } else if constexpr (V == 4) {
+        md_store4<T>(p, f);
+    } else {
+        *p = md_elem<T>::put(f[0]);
+    }
 }
 
-constexpr int NORM_THREADS = 256;
+constexpr int NORM_WARPS = 4;
 
-// block = (row, sequence); V = 4: every size a multiple of 4
+// a warp per row, y = sequence; V divides every size
 template <class T, int V>
-__global__ void __launch_bounds__(NORM_THREADS)
+__global__ void __launch_bounds__(NORM_WARPS * 32)
 latent_norm_kernel(const __grid_constant__ md_latent p) {
-    extern __shared__ __align__(16) float xs[];   // the row
-    __shared__ float red[2][NORM_THREADS / 32];
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, t = blockIdx.x, seq = blockIdx.y;
-    const int Q = p.q_rank, R = p.kv_rank, n = Q + R + p.rot;
+    const int lane = threadIdx.x & 31, t = blockIdx.x * NORM_WARPS + (threadIdx.x >> 5), seq = blockIdx.y;
+    const int Q = p.q_rank, R = p.kv_rank;
     md_pdl_launch_dependents();
     md_pdl_wait();
+    if (t >= p.rows) return;
     const int pos = (p.pos_dev[seq] ? *p.pos_dev[seq] : p.pos0) + t;
     const size_t row = (size_t)seq * p.rows + t;
     const T* in = reinterpret_cast<const T*>(p.in) + row * p.row_stride;
-    float sq = 0.f, sc = 0.f;
-    for (int c = tid * V; c < n; c += NORM_THREADS * V) {
-        float f[V];
-        load_v<T, V>(in + c, f);
+    constexpr int KEEP = 48 / V;     // vectors of a latent that stay in registers; the second pass finds the others in L2
+    float q[KEEP][V], k[KEEP][V];
+    auto load = [&](const T* src, int n, float (&f)[KEEP][V]) {
 #pragma unroll
-        for (int i = 0; i < V; ++i) {
-            xs[c + i] = f[i];
-            if (c < Q) sq = fmaf(f[i], f[i], sq);
-            else if (c < Q + R) sc = fmaf(f[i], f[i], sc);
+        for (int j = 0; j < KEEP; ++j)
+            if ((lane + 32 * j) * V < n) load_v<T, V>(src + (lane + 32 * j) * V, f[j]);
+    };
+    auto norm = [&](const T* src, int n, const float* w, T* dst, float (&f)[KEEP][V]) {
+        float ss = 0.f;
+#pragma unroll
+        for (int j = 0; j < KEEP; ++j) {
+#pragma unroll
+            for (int i = 0; i < V; ++i)
+                if ((lane + 32 * j) * V < n) ss = fmaf(f[j][i], f[j][i], ss);
         }
-    }
-    sq = warp_sum(sq);
-    sc = warp_sum(sc);
-    if (lane == 0) red[0][warp] = sq, red[1][warp] = sc;
-    __syncthreads();
-    sq = sc = 0.f;
+        for (int c = (lane + 32 * KEEP) * V; c < n; c += 32 * V) {
+            float x[V];
+            load_v<T, V>(src + c, x);
 #pragma unroll
-    for (int i = 0; i < NORM_THREADS / 32; ++i) sq += red[0][i], sc += red[1][i];
-    const float iq = 1.f / sqrtf(sq / (float)Q + p.eps), ic = 1.f / sqrtf(sc / (float)R + p.eps);
-    T* cq = reinterpret_cast<T*>(p.cq) + row * Q;
-    T* cc = reinterpret_cast<T*>(p.cc[seq]) + (size_t)pos * R;
+            for (int i = 0; i < V; ++i) ss = fmaf(x[i], x[i], ss);
+        }
+        const float inv = 1.f / sqrtf(warp_sum(ss) / (float)n + p.eps);
+        auto put = [&](int c, float (&x)[V]) {
+            float g[V];
+            load_weight<V>(w + c, g);
+#pragma unroll
+            for (int i = 0; i < V; ++i) x[i] *= inv * g[i];
+            store_v<T, V>(dst + c, x);
+        };
+#pragma unroll
+        for (int j = 0; j < KEEP; ++j)
+            if ((lane + 32 * j) * V < n) put((lane + 32 * j) * V, f[j]);
+        for (int c = (lane + 32 * KEEP) * V; c < n; c += 32 * V) {
+            float x[V];
+            load_v<T, V>(src + c, x);
+            put(c, x);
+        }
+    };
+    load(in, Q, q);
+    load(in + Q, R, k);
+    norm(in, Q, p.q_norm, reinterpret_cast<T*>(p.cq) + row * Q, q);
+    norm(in + Q, R, p.kv_norm, reinterpret_cast<T*>(p.cc[seq]) + (size_t)pos * R, k);
     T* kr = reinterpret_cast<T*>(p.kr[seq]) + (size_t)pos * p.rot;
-    for (int c = tid * V; c < Q + R; c += NORM_THREADS * V) {
-        float w[V], f[V];
-        load_v<float, V>(c < Q ? p.q_norm + c : p.kv_norm + (c - Q), w);
-#pragma unroll
-        for (int i = 0; i < V; ++i) f[i] = xs[c + i] * (c < Q ? iq : ic) * w[i];
-        store_v<T, V>(c < Q ? cq + c : cc + (c - Q), f);
-    }
-    for (int i = tid; i < p.rot / 2; i += NORM_THREADS) {
+    for (int i = lane; i < p.rot / 2; i += 32) {
         const float2 cs = *reinterpret_cast<const float2*>(p.rope + ((size_t)pos * (p.rot / 2) + i) * 2);
-        const float u = xs[Q + R + 2 * i], v = xs[Q + R + 2 * i + 1];
+        const float u = md_elem<T>::get(in[Q + R + 2 * i]), v = md_elem<T>::get(in[Q + R + 2 * i + 1]);
         kr[2 * i] = md_elem<T>::put(u * cs.x - v * cs.y);
         kr[2 * i + 1] = md_elem<T>::put(v * cs.x + u * cs.y);
     }
@@ -851,12 +888,10 @@ bool decode_ok(const md_latent& a) { return vector_ok(a) && a.kv_rank <= 1024 &&
 
 template <class T>
 int launch_norm(md_ctx* ctx, const md_latent& a) {
-    const size_t smem = (size_t)(a.q_rank + a.kv_rank + a.rot) * sizeof(float);
-    if (smem > 200 * 1024) return md_fail(ctx, MD_ERR_UNSUPPORTED, "latent attention: latents of %d and %d values", a.q_rank, a.kv_rank);
-    const bool v4 = ((a.q_rank | a.kv_rank | a.rot | a.row_stride) % 4) == 0;
-    auto kern = v4 ? latent_norm_kernel<T, 4> : latent_norm_kernel<T, 1>;
-    if (smem > 47 * 1024) MD_CUDA(ctx, cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
-    return md_launch_ex(ctx, kern, dim3((unsigned)a.rows, (unsigned)a.seqs), dim3(NORM_THREADS), smem, "latent_norm_kernel", a);
+    constexpr int V = 16 / sizeof(T);
+    auto kern = ((a.q_rank | a.kv_rank | a.row_stride) % V) == 0 ? latent_norm_kernel<T, V> : latent_norm_kernel<T, 1>;
+    return md_launch_ex(ctx, kern, dim3((unsigned)((a.rows + NORM_WARPS - 1) / NORM_WARPS), (unsigned)a.seqs), dim3(NORM_WARPS * 32), 0,
+                        "latent_norm_kernel", a);
 }
 
 template <class T>

@@ -4,14 +4,15 @@
 // The division of work is that of attn_tc_kernel (attention_tc.cu): a work item = 128 queries of one head, key tiles of 64, a
 // persistent CTA per SM, and per CTA
 //   warp 0      TMA producer: an item's Q, K tiles through a ring of three stages, V tiles through a ring of two
-//   warp 1      issues S = Q K^T into one of two S buffers in tensor memory;  warp 6 issues O += P V
+//   warp 1      issues S = Q K^T into one of four S buffers in tensor memory;  warp 6 issues O += P V
 //   warps 2..5  one thread per query row: its row of Q into tensor memory (the rotated part turned on the way), then per tile its
 //               row of S, the softmax, P back over the S buffer.
 // What differs: a row of K is two pieces from two tensors, so Q and K travel as 64-dim atoms of the plain part followed by atoms
 // of the rotated part (zero filled past either), and the k-steps walk both.  P goes back as two bfloat16 terms, 32 columns each,
 // which together fill the S buffer they came from; V is multiplied by both, so the weights keep about 2^-17.  The row sum
 // starts at the sink's weight, which is also the first exponent reference: every row has a finite reference from the start.
-// Tiles run from the first key of the item's window.
+// Tiles run from the first key of the item's window.  With two S buffers the tile period was the chain PV(j-1) -> S(j+1) ->
+// softmax(j+1) (2000 cycles at head sizes 128 + 64, 128); with four it is the longer of the softmax and the products.
 //
 // Numerics: scores, sums and the output accumulate in f32, one rounding to bfloat16 at the end.  Every mbarrier wait is bounded
 // (tc_common.cuh); a wait that gives up is reported through the context's error word and the kernel still runs to its end and
@@ -32,7 +33,7 @@ using namespace tc;
 constexpr int LBQ = 128, LBK = 64, LAT_THREADS = 224;
 constexpr int K_STAGES = 3, V_STAGES = 2, MAX_ATOMS = 4, MAX_V_ATOMS = 2;
 constexpr uint32_t Q_ATOM = LBQ * 128, K_ATOM = LBK * 128;    // bytes of a 64-dim atom
-constexpr uint32_t LAT_TMEM = 512, LT_O = 128, LT_Q = 256;    // two S buffers, O (up to 128), Q (up to 128)
+constexpr uint32_t LAT_TMEM = 512, LT_O = 256, LT_Q = 384;    // four S buffers of 64, O (up to 128), Q (up to 128)
 constexpr float LAT_LOG2E = 1.4426950408889634f, LAT_RESCALE = 8.0f;   // see RESCALE_THRESHOLD of attention_tc.cu
 
 struct LatTcParams {
@@ -78,15 +79,14 @@ latent_tc_kernel(const __grid_constant__ LatTcMaps tm, const LatTcParams p, md_d
     uint8_t* out_ptr = base_ptr + (sm_out - base);
     const uint32_t bars = sm_out + (uint32_t)(LBQ * p.vdim * 2);
     uint8_t* bars_ptr = base_ptr + (bars - base);
-    const uint32_t b_qfull = bars, b_kfull = bars + 8, b_kempty = b_kfull + 8 * K_STAGES, b_vfull = b_kempty + 8 * K_STAGES;
-    const uint32_t b_vempty = b_vfull + 8 * V_STAGES;
-    const uint32_t b_sfull = b_vempty + 8 * V_STAGES;   // S(j) is in tensor memory
-    const uint32_t b_pfull = b_sfull + 16;              // the softmax warps have written P(j) over it
-    const uint32_t b_pvdone = b_pfull + 16;             // PV(j) has completed: O is current, the S / P buffer is free
-    const uint32_t b_qcopied = b_pvdone + 16;           // the softmax warps have moved Q from shared to tensor memory
+    const uint32_t b_qfull = bars, b_kfull = bars + 8, b_vfull = b_kfull + 8 * K_STAGES;
+    const uint32_t b_sfull = b_vfull + 8 * V_STAGES;    // S(j) is in tensor memory: its K stage is free too
+    const uint32_t b_pfull = b_sfull + 32;              // the softmax warps have written P(j) over it
+    const uint32_t b_pvdone = b_pfull + 32;             // PV(j) has completed: O is current, the S / P buffer and the V stage are free
+    const uint32_t b_qcopied = b_pvdone + 32;           // the softmax warps have moved Q from shared to tensor memory
     const uint32_t b_oempty = b_qcopied + 8;            // ... and have read an item's O out of tensor memory
-    volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(bars_ptr + 176);
-    volatile int* abort_flag = reinterpret_cast<volatile int*>(bars_ptr + 180);
+    volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(bars_ptr + 240);
+    volatile int* abort_flag = reinterpret_cast<volatile int*>(bars_ptr + 244);
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     md_pdl_launch_dependents();
@@ -100,15 +100,9 @@ latent_tc_kernel(const __grid_constant__ LatTcMaps tm, const LatTcParams p, md_d
         mbar_init(b_qfull, 1);
         mbar_init(b_qcopied, 4);
         mbar_init(b_oempty, 4);
-        for (int s = 0; s < K_STAGES; ++s) {
-            mbar_init(b_kfull + 8 * s, 1);
-            mbar_init(b_kempty + 8 * s, 1);
-        }
-        for (int s = 0; s < V_STAGES; ++s) {
-            mbar_init(b_vfull + 8 * s, 1);
-            mbar_init(b_vempty + 8 * s, 1);
-        }
-        for (int b = 0; b < 2; ++b) {
+        for (int s = 0; s < K_STAGES; ++s) mbar_init(b_kfull + 8 * s, 1);
+        for (int s = 0; s < V_STAGES; ++s) mbar_init(b_vfull + 8 * s, 1);
+        for (int b = 0; b < 4; ++b) {
             mbar_init(b_sfull + 8 * b, 1);
             mbar_init(b_pfull + 8 * b, 4);
             mbar_init(b_pvdone + 8 * b, 1);
@@ -134,19 +128,21 @@ latent_tc_kernel(const __grid_constant__ LatTcMaps tm, const LatTcParams p, md_d
     if (warp == 0) {
         // ------------------------------------------------------------------ TMA producer
         if (lane == 0) {
-            uint32_t kst = 0, kpar = 1, vst = 0, vpar = 1;  // ring slots and the parities that say "slot free"
+            uint32_t kst = 0, vst = 0;       // ring slots
+            uint32_t gk = 0, gv = 0;         // K and V tiles loaded so far
             int it = 0;
             for (int w; (w = lat_walk(p, it)) >= 0; ++it) {
                 const LatItem i = lat_item(p, w);
                 auto load_k = [&](int j) {
                     const int key = i.start + j * LBK;
-                    mbar_wait(b_kempty + 8 * kst, kpar, abort_flag, flags, 71);
+                    if (gk >= K_STAGES) mbar_wait(b_sfull + 8 * ((gk - K_STAGES) & 3u), ((gk - K_STAGES) >> 2) & 1u, abort_flag, flags, 71);
                     const uint32_t kfull = b_kfull + 8 * kst;
                     uint32_t dst = sm_k + kst * k_bytes;
                     mbar_expect_tx(kfull, k_bytes);
                     for (int a = 0; a < p.atoms_n; ++a, dst += K_ATOM) tma_load_4d(dst, &tm.kn, kfull, a * 64, i.head, key - p.key0, 0);
                     for (int a = 0; a < p.atoms_r; ++a, dst += K_ATOM) tma_load_4d(dst, &tm.kr, kfull, a * 64, key, 0, 0);
-                    if (++kst == K_STAGES) { kst = 0; kpar ^= 1u; }
+                    if (++kst == K_STAGES) kst = 0;
+                    ++gk;
                 };
                 if (it > 0) mbar_wait(b_qcopied, (uint32_t)((it - 1) & 1), abort_flag, flags, 72);
                 mbar_expect_tx(b_qfull, q_bytes);
@@ -157,12 +153,13 @@ latent_tc_kernel(const __grid_constant__ LatTcMaps tm, const LatTcParams p, md_d
                 load_k(0);
                 for (int j = 0; j < i.nt; ++j) {
                     if (j + 1 < i.nt) load_k(j + 1);
-                    mbar_wait(b_vempty + 8 * vst, vpar, abort_flag, flags, 73);
+                    if (gv >= V_STAGES) mbar_wait(b_pvdone + 8 * ((gv - V_STAGES) & 3u), ((gv - V_STAGES) >> 2) & 1u, abort_flag, flags, 73);
                     const uint32_t vfull = b_vfull + 8 * vst, vdst = sm_v + vst * V_BYTES;
                     mbar_expect_tx(vfull, V_BYTES);
 #pragma unroll
                     for (int a = 0; a < NV; ++a) tma_load_4d(vdst + a * K_ATOM, &tm.v, vfull, a * 64, i.head, i.start + j * LBK - p.key0, 0);
-                    if (++vst == V_STAGES) { vst = 0; vpar ^= 1u; }
+                    if (++vst == V_STAGES) vst = 0;
+                    ++gv;
                 }
             }
             if (*abort_flag) {  // let copies in flight land before the CTA's shared memory is released
@@ -182,27 +179,31 @@ latent_tc_kernel(const __grid_constant__ LatTcMaps tm, const LatTcParams p, md_d
                 const int nt = lat_item(p, w).nt;
                 mbar_wait(b_qcopied, (uint32_t)(it & 1), abort_flag, flags, 74);
                 for (int j = 0; j < nt; ++j) {
-                    const uint32_t gj = g + (uint32_t)j, sb = gj & 1u;
+                    const uint32_t gj = g + (uint32_t)j, sb = gj & 3u;
                     mbar_wait(b_kfull + 8 * st, par, abort_flag, flags, 75);
-                    // the buffer still holds P of two tiles back until that PV product has completed
-                    mbar_wait(b_pvdone + 8 * sb, ((gj >> 1) & 1u) ^ 1u, abort_flag, flags, 76);
+                    // the buffer still holds P of four tiles back until that PV product has completed
+                    mbar_wait(b_pvdone + 8 * sb, ((gj >> 2) & 1u) ^ 1u, abort_flag, flags, 76);
                     tc_fence_after();
                     const uint32_t t_s = tmem_base + sb * 64u;
-                    // a k-step of 16 dims: 8 columns of Q, 32 bytes within an atom of K
+                    // a k-step of 16 dims: 8 columns of Q, 32 bytes within an atom of K.  What the issuing thread does between
+                    // two MMAs is tensor-pipe idle time, so whole atoms are unrolled.
                     uint32_t k_lo = k_lo0 + st * stage16, t_q = tmem_base + LT_Q;
-                    auto part = [&](int steps, bool first) {
-                        for (int ks = 0; ks < steps; ++ks) {
-                            const uint32_t lo = k_lo + (uint32_t)(ks >> 2) * (K_ATOM >> 4) + (uint32_t)(ks & 3) * 2;
-                            if (first && ks == 0) tc_mma_f16_ts<false>(t_s, t_q, lo, hi128, idesc_s);
-                            else tc_mma_f16_ts<true>(t_s, t_q + ks * 8, lo, hi128, idesc_s);
+                    tc_mma_f16_ts<false>(t_s, t_q, k_lo, hi128, idesc_s);
+                    int skip = 1;
+                    auto part = [&](int steps) {
+                        for (; steps > 0; steps -= 4, k_lo += K_ATOM >> 4, t_q += 32, skip = 0) {
+                            if (!skip) tc_mma_f16_ts<true>(t_s, t_q, k_lo, hi128, idesc_s);
+                            if (steps >= 4) {
+#pragma unroll
+                                for (int ks = 1; ks < 4; ++ks) tc_mma_f16_ts<true>(t_s, t_q + ks * 8, k_lo + ks * 2, hi128, idesc_s);
+                            } else {
+                                for (int ks = 1; ks < steps; ++ks) tc_mma_f16_ts<true>(t_s, t_q + ks * 8, k_lo + ks * 2, hi128, idesc_s);
+                            }
                         }
                     };
-                    part(p.steps_n, true);
-                    k_lo += (uint32_t)p.atoms_n * (K_ATOM >> 4);
-                    t_q += (uint32_t)p.atoms_n * 32u;
-                    part(p.steps_r, false);
+                    part(p.steps_n);
+                    part(p.steps_r);
                     tc_commit(b_sfull + 8 * sb);
-                    tc_commit(b_kempty + 8 * st);
                     if (++st == K_STAGES) { st = 0; par ^= 1u; }
                 }
                 g += (uint32_t)nt;
@@ -221,9 +222,9 @@ latent_tc_kernel(const __grid_constant__ LatTcMaps tm, const LatTcParams p, md_d
             for (int w; (w = lat_walk(p, it)) >= 0; ++it) {
                 const int nt = lat_item(p, w).nt;
                 for (int j = 0; j < nt; ++j) {
-                    const uint32_t gj = g + (uint32_t)j, pb = gj & 1u;
+                    const uint32_t gj = g + (uint32_t)j, pb = gj & 3u;
                     mbar_wait(b_vfull + 8 * st, par, abort_flag, flags, 77);
-                    mbar_wait(b_pfull + 8 * pb, (gj >> 1) & 1u, abort_flag, flags, 78);
+                    mbar_wait(b_pfull + 8 * pb, (gj >> 2) & 1u, abort_flag, flags, 78);
                     // the first product of an item overwrites O: the previous item's output must have left tensor memory
                     if (j == 0 && it > 0) mbar_wait(b_oempty, (uint32_t)((it - 1) & 1), abort_flag, flags, 79);
                     tc_fence_after();
@@ -238,7 +239,6 @@ latent_tc_kernel(const __grid_constant__ LatTcMaps tm, const LatTcParams p, md_d
                         tc_mma_f16_ts<true>(tmem_base + LT_O, t_p + 32 + ks * 8, v_lo + ks * 128, hi128, idesc_pv);
                     }
                     tc_commit(b_pvdone + 8 * pb);
-                    tc_commit(b_vempty + 8 * st);
                     if (++st == V_STAGES) { st = 0; par ^= 1u; }
                 }
                 g += (uint32_t)nt;
@@ -306,8 +306,8 @@ latent_tc_kernel(const __grid_constant__ LatTcMaps tm, const LatTcParams p, md_d
 
             for (int j = 0; j < nt; ++j) {
                 const uint32_t gj = g + (uint32_t)j;
-                const int sb = (int)(gj & 1u), k0 = i.start + j * LBK;
-                mbar_wait(b_sfull + 8 * sb, (gj >> 1) & 1u, abort_flag, flags, 81);
+                const int sb = (int)(gj & 3u), k0 = i.start + j * LBK;
+                mbar_wait(b_sfull + 8 * sb, (gj >> 2) & 1u, abort_flag, flags, 81);
                 tc_fence_after();
                 uint32_t s0[32], s1[32];
                 tc_ld_32x32(t_lane + (uint32_t)(sb * 64), s0);
@@ -347,7 +347,7 @@ latent_tc_kernel(const __grid_constant__ LatTcMaps tm, const LatTcParams p, md_d
                     const float m_new = fmaxf(m_run, mt), corr = ex2_fast(m_run - m_new);
                     l_run *= corr;
                     m_run = m_new;
-                    mbar_wait(b_pvdone + 8 * ((gj - 1) & 1u), ((gj - 1) >> 1) & 1u, abort_flag, flags, 82);
+                    mbar_wait(b_pvdone + 8 * ((gj - 1) & 3u), ((gj - 1) >> 2) & 1u, abort_flag, flags, 82);
                     tc_fence_after();
 #pragma unroll
                     for (int c = 0; c < NV * 4; ++c) {
@@ -392,7 +392,7 @@ latent_tc_kernel(const __grid_constant__ LatTcMaps tm, const LatTcParams p, md_d
             // its Q goes into tensor memory now, so its first S product runs while this item's output is converted and stored.
             uint32_t o[NV * 4][16];
             const uint32_t gl = g + (uint32_t)nt - 1u;
-            mbar_wait(b_pvdone + 8 * (gl & 1u), (gl >> 1) & 1u, abort_flag, flags, 83);
+            mbar_wait(b_pvdone + 8 * (gl & 3u), (gl >> 2) & 1u, abort_flag, flags, 83);
             tc_fence_after();
 #pragma unroll
             for (int c = 0; c < NV * 4; ++c) {

@@ -530,7 +530,7 @@ int launch_glue(md_ctx* ctx, const md_glue& g) {
                         "stack_glue_kernel", g, R);
 }
 
-// ---- MD_LAYER_PARALLEL: residual update of two sublayers, one norm, up to two weighted outputs
+// ---- MD_LAYER_PARALLEL: residual update of two sublayers (the second may be a routed one), one norm, up to two weighted outputs
 
 constexpr int PAR_THREADS = 512;
 
@@ -538,135 +538,146 @@ template <class T> __device__ __forceinline__ const T* embed_row(const md_parall
     const unsigned long long tok = p.tokens[src];
     return reinterpret_cast<const T*>(p.embed) + (size_t)(tok < (unsigned long long)p.vocab ? tok : 0ull) * p.width;
 }
-// columns c .. c + V of a sublayer's output for row `src`
-template <class T, int V> __device__ __forceinline__ Vec<V> branch_cols(const md_branch& b, size_t src, int W, int c) {
-    if (b.slot) {
-        Vec<V> v;
+// the first choices of a routed row, requested ahead of everything that does not depend on them
+struct Choices { int slot[4]; float score[4]; };
+__device__ __forceinline__ Choices first_choices(const md_branch& b, size_t src) {
+    Choices c = {};
+    if (!b.slot) return c;
 #pragma unroll
-        for (int i = 0; i < V; ++i) v.f[i] = 0.f;
-        for (int k = 0; k < b.top; ++k) {
-            const float s = __ldcg(b.score + src * b.top + k);
-            const Vec<V> e = ldv<T, V>(reinterpret_cast<const T*>(b.y) + (size_t)__ldcg(b.slot + src * b.top + k) * W + c);
-#pragma unroll
-            for (int i = 0; i < V; ++i) v.f[i] = fmaf(s, e.f[i], v.f[i]);
-        }
-        return v;
+    for (int k = 0; k < 4; ++k) {
+        c.slot[k] = k < b.top ? __ldcg(b.slot + src * b.top + k) : 0;
+        c.score[k] = k < b.top ? __ldcg(b.score + src * b.top + k) : 0.f;
     }
-    return b.y_f32 ? ldv<float, V>(b.y_f32 + src * W + c) : ldv<T, V>(reinterpret_cast<const T*>(b.y) + src * W + c);
+    return c;
+}
+// A thread's vectors (every `step` columns from c0) of a sublayer's output for row `src`, all requested before one is used.
+template <class T, int V, int NV>
+__device__ __forceinline__ void branch_row(const md_branch& b, const Choices& ch, size_t src, int W, int c0, int step, Vec<V> (&y)[NV]) {
+#pragma unroll
+    for (int n = 0; n < NV; ++n) {
+#pragma unroll
+        for (int i = 0; i < V; ++i) y[n].f[i] = 0.f;
+    }
+    if (b.slot) {
+        auto take = [&](int slot, float s) {
+            const T* e = reinterpret_cast<const T*>(b.y) + (size_t)slot * W;
+#pragma unroll
+            for (int n = 0; n < NV; ++n) {
+                if (c0 + n * step >= W) continue;
+                const Vec<V> v = ldv<T, V>(e + c0 + n * step);
+#pragma unroll
+                for (int i = 0; i < V; ++i) y[n].f[i] = fmaf(s, v.f[i], y[n].f[i]);
+            }
+        };
+#pragma unroll
+        for (int k = 0; k < 4; ++k)
+            if (k < b.top) take(ch.slot[k], ch.score[k]);
+        for (int k = 4; k < b.top; ++k) take(__ldcg(b.slot + src * b.top + k), __ldcg(b.score + src * b.top + k));
+        return;
+    }
+#pragma unroll
+    for (int n = 0; n < NV; ++n) {
+        const int c = c0 + n * step;
+        if (c >= W) continue;
+        y[n] = b.y_f32 ? ldv<float, V>(b.y_f32 + src * W + c) : ldv<T, V>(reinterpret_cast<const T*>(b.y) + src * W + c);
+    }
 }
 
-// GW warps per row, NV vectors of V columns per lane: width <= 32 * V * GW * NV.  All weights are requested before the
-// dependency wait when one group has the whole block (a decode step).
+// GW warps per row, NV vectors of V columns per lane: width <= 32 * V * GW * NV.  A block walks over rows and keeps its columns'
+// weights and scales in registers, requested before the dependency wait.
 template <class T, int V, int GW, int NV>
-__global__ void __launch_bounds__(PAR_THREADS)
+__global__ void __launch_bounds__(PAR_THREADS, NV == 1 ? 2 : 1)
 stack_parallel_kernel(const __grid_constant__ md_parallel_glue p) {
-    __shared__ float red[PAR_THREADS / 32];
+    __shared__ float red[2][PAR_THREADS / 32];
     constexpr int GROUPS = PAR_THREADS / 32 / GW;
-    constexpr bool EARLY = GW == PAR_THREADS / 32 && NV <= 2;
     const int W = p.width, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int grp = warp / GW, gl = (warp % GW) * 32 + lane, row = blockIdx.x * GROUPS + grp;
-    const bool live = row < p.rows;
+    const int grp = warp / GW, c0 = ((warp % GW) * 32 + lane) * V, step = 32 * GW * V;
     md_pdl_launch_dependents();
     Vec<V> w[2][NV], s[2][NV];
-    if constexpr (EARLY) {
 #pragma unroll
-        for (int n = 0; n < NV; ++n) {
-            const int c = (gl + n * 32 * GW) * V;
-            if (c >= W) continue;
+    for (int n = 0; n < NV; ++n) {
+        const int c = c0 + n * step;
 #pragma unroll
-            for (int o = 0; o < 2; ++o) {
-                if (p.out[o]) w[o][n] = ldv<float, V>(p.w[o] + c);
-                if (p.b[o].scale) s[o][n] = ldv<float, V>(p.b[o].scale + c);
-            }
+        for (int o = 0; o < 2; ++o) {
+#pragma unroll
+            for (int i = 0; i < V; ++i) w[o][n].f[i] = 0.f, s[o][n].f[i] = 1.f;
+            if (c < W && p.out[o]) w[o][n] = ldv<float, V>(p.w[o] + c);
+            if (c < W && p.b[o].scale) s[o][n] = ldv<float, V>(p.b[o].scale + c);
         }
     }
     md_pdl_wait();
-    const size_t src = live ? (p.gather ? (size_t)p.gather[row] : row) : 0;
-    Vec<V> x[NV];
-    const T* xe = p.tokens ? embed_row<T>(p, src) : nullptr;
-#pragma unroll
-    for (int n = 0; n < NV; ++n) {
-        const int c = (gl + n * 32 * GW) * V;
-#pragma unroll
-        for (int i = 0; i < V; ++i) x[n].f[i] = 0.f;
-        if (live && c < W) x[n] = xe ? ldv<T, V>(xe + c) : ldv<float, V>(p.x + src * W + c);
-    }
-    // The routed sublayer of a prompt gathers its rows by index: the other one first, so that its loads are on their way.
-#pragma unroll
-    for (int b = 0; b < 2; ++b) {
-        if (!p.b[b].y_f32 && !p.b[b].y) continue;
+    int turn = 0;
+    for (int row0 = blockIdx.x * GROUPS; row0 < p.rows; row0 += gridDim.x * GROUPS, turn ^= 1) {
+        const int row = row0 + grp;
+        const bool live = row < p.rows;
+        const size_t src = live ? (p.gather ? (size_t)p.gather[row] : row) : 0;
+        Vec<V> x[NV];
+        const Choices ch = first_choices(p.b[1], src);
+        const T* xe = p.tokens ? embed_row<T>(p, src) : nullptr;
 #pragma unroll
         for (int n = 0; n < NV; ++n) {
-            const int c = (gl + n * 32 * GW) * V;
-            if (!live || c >= W) continue;
-            const Vec<V> y = branch_cols<T, V>(p.b[b], src, W, c);
-            if (p.b[b].scale) {
-                if constexpr (!EARLY) s[b][n] = ldv<float, V>(p.b[b].scale + c);
+            const int c = c0 + n * step;
 #pragma unroll
-                for (int i = 0; i < V; ++i) x[n].f[i] = fmaf(s[b][n].f[i], y.f[i], x[n].f[i]);
-            } else {
+            for (int i = 0; i < V; ++i) x[n].f[i] = 0.f;
+            if (live && c < W) x[n] = xe ? ldv<T, V>(xe + c) : ldv<float, V>(p.x + src * W + c);
+        }
 #pragma unroll
-                for (int i = 0; i < V; ++i) x[n].f[i] += y.f[i];
+        for (int b = 0; b < 2; ++b) {
+            if ((!p.b[b].y_f32 && !p.b[b].y) || !live) continue;
+            Vec<V> y[NV];
+            branch_row<T, V, NV>(p.b[b], ch, src, W, c0, step, y);
+#pragma unroll
+            for (int n = 0; n < NV; ++n) {
+#pragma unroll
+                for (int i = 0; i < V; ++i) x[n].f[i] = fmaf(s[b][n].f[i], y[n].f[i], x[n].f[i]);
             }
         }
-    }
-    float ss = 0.f;
-#pragma unroll
-    for (int n = 0; n < NV; ++n) {
-        const int c = (gl + n * 32 * GW) * V;
-#pragma unroll
-        for (int i = 0; i < V; ++i) ss = fmaf(x[n].f[i], x[n].f[i], ss);
-        if (live && c < W && p.x_out) stv<float, V>(p.x_out + (size_t)row * W + c, x[n]);
-    }
-    ss = warp_sum(ss);
-    if constexpr (GW > 1) {
-        if (lane == 0) red[warp] = ss;
-        __syncthreads();
-        ss = 0.f;
-#pragma unroll
-        for (int i = 0; i < GW; ++i) ss += red[grp * GW + i];
-    }
-    const float inv = 1.f / sqrtf(ss / (float)W + p.eps);
-#pragma unroll
-    for (int o = 0; o < 2; ++o) {
-        if (!p.out[o]) continue;
-        T* out = reinterpret_cast<T*>(p.out[o]) + (size_t)row * W;
+        float ss = 0.f;
 #pragma unroll
         for (int n = 0; n < NV; ++n) {
-            const int c = (gl + n * 32 * GW) * V;
-            if (!live || c >= W) continue;
-            if constexpr (!EARLY) w[o][n] = ldv<float, V>(p.w[o] + c);
-            Vec<V> v;
+            const int c = c0 + n * step;
 #pragma unroll
-            for (int i = 0; i < V; ++i) v.f[i] = x[n].f[i] * (inv * w[o][n].f[i]);
-            stv<T, V>(out + c, v);
+            for (int i = 0; i < V; ++i) ss = fmaf(x[n].f[i], x[n].f[i], ss);
+            if (live && c < W && p.x_out) stv<float, V>(p.x_out + (size_t)row * W + c, x[n]);
+        }
+        ss = warp_sum(ss);
+        if constexpr (GW > 1) {
+            if (lane == 0) red[turn][warp] = ss;
+            __syncthreads();
+            ss = 0.f;
+#pragma unroll
+            for (int i = 0; i < GW; ++i) ss += red[turn][grp * GW + i];
+        }
+        const float inv = 1.f / sqrtf(ss / (float)W + p.eps);
+#pragma unroll
+        for (int o = 0; o < 2; ++o) {
+            if (!p.out[o]) continue;
+            T* out = reinterpret_cast<T*>(p.out[o]) + (size_t)row * W;
+#pragma unroll
+            for (int n = 0; n < NV; ++n) {
+                const int c = c0 + n * step;
+                if (!live || c >= W) continue;
+                Vec<V> v;
+#pragma unroll
+                for (int i = 0; i < V; ++i) v.f[i] = x[n].f[i] * (inv * w[o][n].f[i]);
+                stv<T, V>(out + c, v);
+            }
         }
     }
 }
 
 template <class T, int V>
 int launch_parallel_v(md_ctx* ctx, const md_parallel_glue& g) {
-    void (*kern)(md_parallel_glue) = nullptr;
     const int per = 32 * V;   // columns a warp holds in one vector per lane
-    int gw = 16;
-    // few rows: the whole block on one row; many: as few warps per row as four vectors per lane allow
-    if (g.rows <= 296) {
-        kern = g.width <= 16 * per ? stack_parallel_kernel<T, V, 16, 1> : g.width <= 32 * per ? stack_parallel_kernel<T, V, 16, 2>
-             : g.width <= 64 * per ? stack_parallel_kernel<T, V, 16, 4> : stack_parallel_kernel<T, V, 16, 8>;
-    } else if (g.width <= 4 * per) {
-        kern = stack_parallel_kernel<T, V, 1, 4>, gw = 1;
-    } else if (g.width <= 8 * per) {
-        kern = stack_parallel_kernel<T, V, 2, 4>, gw = 2;
-    } else if (g.width <= 16 * per) {
-        kern = stack_parallel_kernel<T, V, 4, 4>, gw = 4;
-    } else if (g.width <= 32 * per) {
-        kern = stack_parallel_kernel<T, V, 8, 4>, gw = 8;
-    } else {
-        kern = g.width <= 64 * per ? stack_parallel_kernel<T, V, 16, 4> : stack_parallel_kernel<T, V, 16, 8>;
-    }
     if (g.width > 128 * per) return md_fail(ctx, MD_ERR_UNSUPPORTED, "a width of %d exceeds %d", g.width, 128 * per);
-    const int groups = 16 / gw;
-    return md_launch_ex(ctx, kern, dim3((unsigned)((g.rows + groups - 1) / groups)), dim3(PAR_THREADS), 0, "stack_parallel_kernel", g);
+    const int vectors = (g.width + per - 1) / per;
+    void (*kern)(md_parallel_glue) = vectors <= 1 ? stack_parallel_kernel<T, V, 1, 1> : vectors <= 2 ? stack_parallel_kernel<T, V, 2, 1>
+                                   : vectors <= 4 ? stack_parallel_kernel<T, V, 4, 1> : vectors <= 8 ? stack_parallel_kernel<T, V, 8, 1>
+                                   : vectors <= 16 ? stack_parallel_kernel<T, V, 16, 1> : vectors <= 32 ? stack_parallel_kernel<T, V, 16, 2>
+                                   : vectors <= 64 ? stack_parallel_kernel<T, V, 16, 4> : stack_parallel_kernel<T, V, 16, 8>;
+    const int groups = vectors <= 1 ? 16 : vectors <= 2 ? 8 : vectors <= 4 ? 4 : vectors <= 8 ? 2 : 1, blocks = (g.rows + groups - 1) / groups;
+    const int most = ctx->sm_count * (vectors <= 16 ? 2 : 1);
+    return md_launch_ex(ctx, kern, dim3((unsigned)(blocks < most ? blocks : most)), dim3(PAR_THREADS), 0, "stack_parallel_kernel", g);
 }
 
 template <class T>
